@@ -75,7 +75,7 @@ _SIGNATURES = {
     "illm_model_files_read": [S, S, P, LL], "illm_write_safetensors": [S, S, P, S],
     "illm_pool_create": [I, S, PP], "illm_pool_free_handle": [P], "illm_pool_alloc": [P, I, PI],
     "illm_pool_release": [P, PI, I], "illm_pool_check": [P], "illm_pool_stats": [P, PI, PI], "illm_pool_is_held": [P, I],
-    "illm_ledger_create": [I, I, I, I, PP], "illm_ledger_free_handle": [P], "illm_ledger_pages_needed": [P, I, LL],
+    "illm_ledger_create": [I, I, I, I, I, PP], "illm_ledger_free_handle": [P], "illm_ledger_pages_needed": [P, I, LL],
     "illm_ledger_reserve": [P, I, LL], "illm_ledger_release_outside_window": [P, I, LL], "illm_ledger_release_all": [P, I],
     "illm_ledger_release_beyond": [P, I, LL], "illm_ledger_row": [P, I, I, PI], "illm_ledger_check": [P],
     "illm_ledger_pool": [P], "illm_ledger_pages": [P, I, PI, PI, I],

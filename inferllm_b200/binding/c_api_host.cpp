@@ -242,8 +242,8 @@ ILLM_API int illm_pool_stats(void* p, int* n_free, int* n_held) {
 }
 ILLM_API int illm_pool_is_held(void* p, int i) { return ((IndexPool*)p)->is_held(i) ? 1 : 0; }
 
-ILLM_API int illm_ledger_create(int num_pages, int page_size, int num_slots, int window, void** out) {
-    return guard([&] { *out = new PageLedger(num_pages, page_size, num_slots, window); });
+ILLM_API int illm_ledger_create(int num_pages, int page_size, int num_slots, int window, int chunk, void** out) {
+    return guard([&] { *out = new PageLedger(num_pages, page_size, num_slots, window, chunk); });
 }
 ILLM_API void illm_ledger_free_handle(void* p) { delete (PageLedger*)p; }
 ILLM_API int illm_ledger_pages_needed(void* p, int slot, long long new_len) { return ((PageLedger*)p)->pages_needed(slot, new_len); }

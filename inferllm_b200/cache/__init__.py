@@ -16,18 +16,21 @@ from ..binding import CacheError, CacheFull   # noqa: F401
 
 @dataclass(frozen=True)
 class PagedKV:
-    """Keys and values of every position (or of the last `window` positions) of a sequence; `keys_only`: one row
-    per position that serves as key and as value (a shared latent), no value pages."""
+    """Keys and values of every position (or of the last `window` positions, or of the query's own `chunk` of positions) of a
+    sequence; `keys_only`: one row per position that serves as key and as value (a shared latent), no value pages."""
 
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     keys_only: bool = False
+    chunk: Optional[int] = None
 
     def to_json(self):
         j = {"kind": "kv", "n_kv_heads": self.n_kv_heads, "head_dim": self.head_dim, "window": self.window}
         if self.keys_only:
             j["keys_only"] = True
+        if self.chunk:
+            j["chunk"] = self.chunk
         return j
 
 
@@ -81,9 +84,9 @@ class IndexPool:
 
 
 class PageLedger:
-    def __init__(self, num_pages: int, page_size: int, num_slots: int, window=None):
+    def __init__(self, num_pages: int, page_size: int, num_slots: int, window=None, chunk=None):
         out = ctypes.c_void_p()
-        _b.check(_b.lib().illm_ledger_create(num_pages, page_size, num_slots, int(window or 0), ctypes.byref(out)))
+        _b.check(_b.lib().illm_ledger_create(num_pages, page_size, num_slots, int(window or 0), int(chunk or 0), ctypes.byref(out)))
         self._ptr = out
         self.num_slots = num_slots
         self.pool = IndexPool(num_pages, "page", _ptr=ctypes.c_void_p(_b.lib().illm_ledger_pool(out)), _owner=self)

@@ -32,7 +32,7 @@ CacheRequest CacheRequest::state(std::vector<long long> shape, DType dtype) {
     return r;
 }
 bool CacheRequest::operator==(const CacheRequest& o) const {
-    return kind == o.kind && n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && v_head_dim == o.v_head_dim && window == o.window &&
+    return kind == o.kind && n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && v_head_dim == o.v_head_dim && window == o.window && chunk == o.chunk &&
            keys_only == o.keys_only && shape == o.shape &&
            (kind != FixedState || dtype == o.dtype);
 }
@@ -46,6 +46,7 @@ Json CacheRequest::to_json() const {
         if (v_head_dim != head_dim) j.set("v_head_dim", v_head_dim);
         if (keys_only) j.set("keys_only", true);
         j.set("window", window ? Json(window) : Json());
+        if (chunk) j.set("chunk", chunk);
     } else {
         j.set("kind", "state");
         Json s = Json::array();
@@ -58,13 +59,16 @@ Json CacheRequest::to_json() const {
 CacheRequest CacheRequest::from_json(const Json& j) {
     if (j.is_null()) return CacheRequest();
     const std::string kind = j.at("kind").is_string() ? j.at("kind").as_string() : "";
+    const int chunk = j.has("chunk") && j.at("chunk").is_int() ? (int)j.at("chunk").as_int() : 0;
+    if (chunk < 0 || (chunk > 0 && j.has("window") && j.at("window").is_int() && j.at("window").as_int() > 0))
+        throw CacheError("a cache request has a window or a chunk, not both, and neither is negative");
     if (kind == "kv" && j.has("keys_only") && j.at("keys_only").is_bool() && j.at("keys_only").as_bool())
         return paged_keys_only((int)j.at("n_kv_heads").as_int(), (int)j.at("head_dim").as_int(),
-                               j.at("window").is_int() ? (int)j.at("window").as_int() : 0);
+                               j.at("window").is_int() ? (int)j.at("window").as_int() : 0).in_chunks(chunk);
     if (kind == "kv")
         return paged((int)j.at("n_kv_heads").as_int(), (int)j.at("head_dim").as_int(),
                      j.at("window").is_int() ? (int)j.at("window").as_int() : 0,
-                     j.has("v_head_dim") && j.at("v_head_dim").is_int() ? (int)j.at("v_head_dim").as_int() : 0);
+                     j.has("v_head_dim") && j.at("v_head_dim").is_int() ? (int)j.at("v_head_dim").as_int() : 0).in_chunks(chunk);
     if (kind == "state") {
         std::vector<long long> shape;
         for (const Json& d : j.at("shape").items()) shape.push_back(d.as_int());
@@ -116,8 +120,8 @@ void IndexPool::check() const {
 
 // ---- PageLedger
 
-PageLedger::PageLedger(int num_pages, int page_size_, int num_slots, int window_)
-        : pool(num_pages, "page"), page_size(page_size_), window(window_), pages((size_t)num_slots), n_logical((size_t)num_slots, 0) {}
+PageLedger::PageLedger(int num_pages, int page_size_, int num_slots, int window_, int chunk_)
+        : pool(num_pages, "page"), page_size(page_size_), window(window_), chunk(chunk_), pages((size_t)num_slots), n_logical((size_t)num_slots, 0) {}
 
 static long long ceil_div(long long a, long long b) { return (a + b - 1) / b; }
 
@@ -134,8 +138,9 @@ void PageLedger::reserve(int slot, long long new_len) {
 }
 std::vector<int> PageLedger::release_outside_window(int slot, long long seq_len) {
     std::vector<int> gone;
-    if (window <= 0) return gone;
-    const long long first_needed_pos = seq_len - window + 1;     // oldest key the next token may see
+    if (window <= 0 && chunk <= 0) return gone;
+    // oldest key the next token (at position seq_len) may see
+    const long long first_needed_pos = chunk > 0 ? seq_len / chunk * chunk : seq_len - window + 1;
     if (first_needed_pos <= 0) return gone;
     const int first_page = (int)(first_needed_pos / page_size);
     auto& have = pages[slot];
@@ -212,7 +217,7 @@ SequenceCache::SequenceCache(const std::map<int, CacheRequest>& requests, int nu
             if (gi < 0) {
                 PagedGroup g;
                 g.request = req;
-                g.ledger.reset(new PageLedger(num_pages, page_size, num_slots, req.window));
+                g.ledger.reset(new PageLedger(num_pages, page_size, num_slots, req.window, req.chunk));
                 paged.push_back(std::move(g));
                 gi = (int)paged.size() - 1;
             }
@@ -406,6 +411,7 @@ KVView SequenceCache::kv_view(int entry, const int* table_dev) const {
     v.num_pages = num_pages;
     v.page_size = page_size;
     v.window = g.request.window;
+    v.chunk = g.request.chunk;
     v.n_kv_heads = g.request.n_kv_heads;
     v.head_dim = g.request.head_dim;
     v.v_head_dim = g.request.v_head_dim;

@@ -2,7 +2,7 @@
 // per-sequence state of fixed size.
 //
 // Layers ask for storage through their mixer's cache_request(): PagedKV(kv heads, head size,
-// window) or FixedState(shape, dtype).  Cache entries (one per writing entry of the model's
+// window or chunk) or FixedState(shape, dtype).  Cache entries (one per writing entry of the model's
 // schedule) with equal requests form a group; every group has storage, a page pool and page tables
 // of its own, so groups with different needs (all keys, a window of them, another head size) live
 // side by side.  Device storage of a paged group: k : [entries, pages, kv heads, page_size,
@@ -37,6 +37,9 @@ struct CacheRequest {
     // PagedKV: keys and values of every position (window 0) or of the last `window` positions
     // (value rows of v_head_dim elements; equal to head_dim unless the mixer says otherwise)
     int n_kv_heads = 0, head_dim = 0, window = 0, v_head_dim = 0;
+    // PagedKV with chunk c > 0: a query sees the earlier positions of its own chunk of c positions, floor(j / c) ==
+    // floor(i / c), counted from the sequence's start (not together with a window)
+    int chunk = 0;
     // PagedKV with keys_only: one row per position that serves as key and as value (a shared latent); no value
     // pages are kept, and a view's `v` is its `k`
     bool keys_only = false;
@@ -46,6 +49,7 @@ struct CacheRequest {
 
     static CacheRequest paged(int n_kv_heads, int head_dim, int window = 0, int v_head_dim = 0);
     static CacheRequest paged_keys_only(int n_kv_heads, int head_dim, int window = 0);
+    CacheRequest in_chunks(int size) const { CacheRequest r = *this; r.chunk = size; return r; }
     static CacheRequest state(std::vector<long long> shape, DType dtype = DType::F32);
     long long elements() const { long long n = 1; for (long long s : shape) n *= s; return n; }
     bool operator==(const CacheRequest& o) const;
@@ -74,10 +78,10 @@ private:
 
 // The pages of one group of layers: a pool and, per slot, the pages it holds by logical page number.
 // A windowed group gives pages back once every position in them has left the window of all future
-// queries; their logical entry then reads -1.
+// queries, a chunked group once every position in them lies in a finished chunk; their logical entry then reads -1.
 class PageLedger {
 public:
-    PageLedger(int num_pages, int page_size, int num_slots, int window = 0);
+    PageLedger(int num_pages, int page_size, int num_slots, int window = 0, int chunk = 0);
     int pages_needed(int slot, long long new_len) const;
     void reserve(int slot, long long new_len);                        // pages for positions 0..new_len-1 (those not yet released)
     std::vector<int> release_outside_window(int slot, long long seq_len);   // after a step; returns the pages given back
@@ -86,7 +90,7 @@ public:
     void row(int slot, int width, int* out) const;                    // logical -> physical table, -1 = no page
     void check() const;
     IndexPool pool;
-    int page_size, window;
+    int page_size, window, chunk;
     std::vector<std::map<int, int>> pages;     // per slot: logical page -> physical page
     std::vector<int> n_logical;                // logical pages ever reserved by the slot's sequence
 };
@@ -104,6 +108,10 @@ struct KVView {
     const int* block_table = nullptr;   // int32 [B, width] on the device, rows in the order of the step's sequences
     int width = 0, num_pages = 0, page_size = 0, window = 0, n_kv_heads = 0, head_dim = 0;
     int v_head_dim = 0;         // v: [pages, kv heads, page_size, v_head_dim]
+    int chunk = 0;              // see CacheRequest::chunk
+    // Which earlier positions a query sees, as the one number the attention kernels take (first_visible, csrc/common.cuh):
+    // 0 all, w > 0 the last w, -c < 0 those of its own chunk of c.
+    int span() const { return chunk > 0 ? -chunk : window; }
     DType dtype = DType::BF16;
     bool writes = true;
 };

@@ -233,8 +233,16 @@ class TukulornConfig(LibraryConfig):
     architecture = "Tukulorn"
 
 
+class FifotarConfig(LibraryConfig):
+    """The Fifotar decoder (`config/fifotar.h`): `layers` (a list of {type: "delta" | "latent_attention" | "attention",
+    mixer: {...}, mlp: {kind: "dense", ff, limit} | None}), `width`, `vocab`, `norm` ({eps}), `embedding` ({scale}),
+    `residual_mult`, `logit_softcap`, optionally `max_positions`.  The dictionary names the class under `architecture`."""
+
+    architecture = "Fifotar"
+
+
 _PY_CLASSES: Dict[str, type] = {"LlamaForCausalLM": LlamaConfig, "Vokelix": VokelixConfig, "Vizosun": VizosunConfig, "Kudonex": KudonexConfig,
-                                "Tukulorn": TukulornConfig}
+                                "Tukulorn": TukulornConfig, "Fifotar": FifotarConfig}
 _CALLBACKS = {}      # name -> (ctypes callback, holder of the last returned text): kept alive while registered
 
 
@@ -277,7 +285,7 @@ def register_architecture(name: str, config_cls: type, aliases=()):
 def unregister_architecture(name: str):
     _b.check(_b.lib().illm_unregister_architecture(name.encode()))
     _CALLBACKS.pop(name, None)
-    if _PY_CLASSES.get(name) not in (LlamaConfig, VokelixConfig, VizosunConfig, KudonexConfig, TukulornConfig):
+    if _PY_CLASSES.get(name) not in (LlamaConfig, VokelixConfig, VizosunConfig, KudonexConfig, TukulornConfig, FifotarConfig):
         _PY_CLASSES.pop(name, None)
 
 

@@ -214,6 +214,7 @@ void register_vokelix_architecture();   // config/vokelix.cpp
 void register_vizosun_architecture();   // config/vizosun.cpp
 void register_kudonex_architecture();   // config/kudonex.cpp
 void register_tukulorn_architecture();  // config/tukulorn.cpp
+void register_fifotar_architecture();   // config/fifotar.cpp
 
 static void ensure_builtin() {
     static bool done = false;
@@ -224,6 +225,7 @@ static void ensure_builtin() {
         register_vizosun_architecture();
         register_kudonex_architecture();
         register_tukulorn_architecture();
+        register_fifotar_architecture();
     }
 }
 

@@ -147,16 +147,19 @@ __device__ __forceinline__ void rd_encoded_chunk(const RdRope& rp, const bf16* _
 
 // What mixers beyond the plain attention add: `sinks` (float32 [nh]: one more term exp(sink) of the
 // softmax denominator, without a value), `gate` (float32, gate[t * gate_stride + h]: the head's output
-// is multiplied by its sigmoid).  WIDE: the softmax weights enter the product with V as two bfloat16
+// is multiplied by its sigmoid; with gate_wide gate[t * gate_stride + h * D + c], one per channel), `softcap` (> 0: the scaled
+// scores s become softcap * tanh(s / softcap); softcap_x is 2 scale log2(e) / softcap).  WIDE: the softmax weights enter the product with V as two bfloat16
 // terms (P1 = P rounded, P2 = P - P1 rounded), sixteen bits of their mantissa instead of eight.
 struct RdExtras {
     const float* sinks;
     const float* gate;
     int gate_stride;
+    int gate_wide;
+    float softcap, softcap_x;
 };
 
 // num / den of a head with the sink's term added (m and the sink in units of log2) and the gate applied
-__device__ __forceinline__ float rd_finish(float num, float den, float m, const RdExtras& ex, int t, int h) {
+__device__ __forceinline__ float rd_finish(float num, float den, float m, const RdExtras& ex, int t, int h, int d, int c) {
     if (ex.sinks) {
         const float s2 = ex.sinks[h] * 1.4426950408889634f;
         if (s2 <= m) {
@@ -168,7 +171,7 @@ __device__ __forceinline__ float rd_finish(float num, float den, float m, const 
         }
     }
     float r = num / den;
-    if (ex.gate) r *= 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.gate_stride + h]));
+    if (ex.gate) r *= 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.gate_stride + (ex.gate_wide ? (size_t)h * d + c : h)]));
     return r;
 }
 
@@ -178,7 +181,7 @@ attention_decode_ring_kernel(const __grid_constant__ CUtensorMap map_k, const __
                              const bf16* __restrict__ q, int q_stride, const int* __restrict__ block_table,
                              int max_pages, const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                              float* __restrict__ part_acc, float* __restrict__ part_ml, bf16* __restrict__ out,
-                             int n_splits, int nh, int nkv, int G, int page_size, int window, float scale_log2e,
+                             int n_splits, int nh, int nkv, int G, int page_size, int span, float scale_log2e,
                              int* __restrict__ err, const RdRope rp, const RdExtras ex) {
     constexpr int STAGES = 384 / D;
     constexpr int CH = D / 8, KS = D / 16, NT_D = D / 8;
@@ -215,7 +218,7 @@ attention_decode_ring_kernel(const __grid_constant__ CUtensorMap map_k, const __
 
     const int split = blockIdx.x, hk = blockIdx.y, t = blockIdx.z;
     const int p = token_pos[t];
-    const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+    const int lo = first_visible(p, span);
     const int tile_lo = lo / RD_BN, tile_hi = p / RD_BN;
     const int n_tiles = tile_hi - tile_lo + 1;
     const int n_my = split < n_tiles ? (n_tiles - split + n_splits - 1) / n_splits : 0;
@@ -371,7 +374,9 @@ attention_decode_ring_kernel(const __grid_constant__ CUtensorMap map_k, const __
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int key = key0 + nt * 8 + t4 * 2 + (e & 1);
-                    const float v = (key > p || key < lo) ? -INFINITY : (sa[nt][e] + sb[nt][e]) * scale_log2e;
+                    float v = (sa[nt][e] + sb[nt][e]) * scale_log2e;
+                    if (WIDE && ex.softcap > 0.f) v = 1.4426950408889634f * soft_cap_fast(sa[nt][e] + sb[nt][e], ex.softcap, ex.softcap_x);
+                    if (key > p || key < lo) v = -INFINITY;
                     sc[nt][e] = v;
                     mx[e >> 1] = fmaxf(mx[e >> 1], v);
                 }
@@ -476,7 +481,7 @@ attention_decode_ring_kernel(const __grid_constant__ CUtensorMap map_k, const __
         }
         const size_t head = (size_t)t * nh + hk * G + r;
         if (n_splits == 1) {
-            out[head * D + c] = __float2bfloat16_rn(rd_finish(num, den, M, ex, t, hk * G + r));
+            out[head * D + c] = __float2bfloat16_rn(rd_finish(num, den, M, ex, t, hk * G + r, D, c));
         } else {
             const size_t oidx = head * n_splits + split;
             part_acc[oidx * D + c] = num;
@@ -507,7 +512,7 @@ __global__ void attention_decode_ring_merge_kernel(const float* __restrict__ par
         den += part_ml[(o + s) * 2 + 1] * w;
         num += part_acc[(o + s) * D + c] * w;
     }
-    out[((size_t)t * nh + h) * D + c] = __float2bfloat16_rn(rd_finish(num, den, M, ex, t, h));
+    out[((size_t)t * nh + h) * D + c] = __float2bfloat16_rn(rd_finish(num, den, M, ex, t, h, D, c));
 }
 
 // ---- host side
@@ -607,14 +612,16 @@ extern "C" int illm_attention_decode_ring(const void* q, int q_stride, const voi
                   nh, nkv, d, page_size, window, scale, n_splits, err, stream, nullptr);
 }
 
-// The same with sinks, gates (either may be nullptr) and, with wide_p, two-term softmax weights.
+// The same with sinks, gates (either may be nullptr), a soft cap (0: none; needs wide_p) and, with wide_p, two-term softmax
+// weights; `window` is a span (first_visible): a window, or chunks if it is negative.
 extern "C" int illm_attention_decode_ring_ex(const void* q, int q_stride, const void* kc, const void* vc,
                                              long long n_pages, const int* block_table, int max_pages,
                                              const int* token_pos, const int* token_seq, float* part_acc,
                                              float* part_ml, void* out, int T, int nh, int nkv, int d, int page_size,
                                              int window, float scale, int n_splits, int* err, int wide_p, const float* sinks,
-                                             const float* gate, int gate_stride, void* stream) {
-    RdExtras ex{sinks, gate, gate_stride};
+                                             const float* gate, int gate_stride, int gate_wide, float softcap, void* stream) {
+    if (softcap > 0.f && !wide_p) return ILLM_ERR_BAD_ARG;
+    RdExtras ex{sinks, gate, gate_stride, gate_wide, softcap, softcap > 0.f ? 2.0f * scale * 1.4426950408889634f / softcap : 0.f};
     return rd_run(q, q_stride, kc, vc, n_pages, block_table, max_pages, token_pos, token_seq, part_acc, part_ml, out, T,
                   nh, nkv, d, page_size, window, scale, n_splits, err, stream, nullptr, &ex, wide_p != 0);
 }

@@ -13,12 +13,13 @@
 // (a key per lane for the scores, a channel per lane for the values) with a running maximum
 // and sum, and are merged in a fixed order.  The split of the keys depends only on the
 // token's own position and window, so its result does not depend on the step it is part of.
-//   score = (q . k) * scale;  keys lo..p with lo = max(0, p - window + 1) (window 0 = all)
+//   score = (q . k) * scale;  keys lo..p with lo = first_visible(p, span): all, a window or a chunk
 //
-// Three options for mixers that are more than the plain softmax attention: values of another head
+// Four options for mixers that are more than the plain softmax attention: values of another head
 // size than the keys (dv); a sink, one learned number per head whose exponential joins the
-// softmax denominator as one more term without a value (sinks[h], not scaled); and an output gate,
-// sigmoid(gate[t * gate_stride + h]) multiplied into the head's output.
+// softmax denominator as one more term without a value (sinks[h], not scaled); an output gate,
+// sigmoid(gate[t * gate_stride + h]) multiplied into the head's output (or, wide, one per value channel:
+// sigmoid(gate[t * gate_stride + h * dv + c])); and a soft cap, score <- cap * tanh(score / cap).
 #include <math.h>
 
 #include "common.cuh"
@@ -32,8 +33,8 @@ attention_generic_kernel(const TA* __restrict__ q, int q_stride, const TA* __res
                          const TA* __restrict__ vc, const int* __restrict__ block_table,
                          int max_pages, const int* __restrict__ token_pos,
                          const int* __restrict__ token_seq, TA* __restrict__ out, int nh, int nkv,
-                         int d, int page_size, int window, float scale, int dv,
-                         const float* __restrict__ sinks, const float* __restrict__ gate, int gate_stride) {
+                         int d, int page_size, int span, float scale, int dv,
+                         const float* __restrict__ sinks, const float* __restrict__ gate, int gate_stride, int gate_wide, float softcap) {
     pdl_grid_sync();
     extern __shared__ float smem[];
     float* qs = smem;                 // [d]
@@ -44,7 +45,7 @@ attention_generic_kernel(const TA* __restrict__ q, int q_stride, const TA* __res
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int hk = h / (nh / nkv);
     const int p = token_pos[t];
-    const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+    const int lo = first_visible(p, span);
     const int* bt = block_table + (size_t)token_seq[t] * max_pages;
 
     const TA* qrow = q + (size_t)t * q_stride + (size_t)h * d;
@@ -79,6 +80,7 @@ attention_generic_kernel(const TA* __restrict__ q, int q_stride, const TA* __res
                 for (int c = 0; c < d; c++) dot = fmaf(qs[c], to_f32(kr[c]), dot);
             }
             s = dot * scale;
+            if (softcap > 0.f) s = softcap * tanhf(s / softcap);
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float pe = valid ? expf(s - m_new) : 0.f;
@@ -126,22 +128,25 @@ attention_generic_kernel(const TA* __restrict__ q, int q_stride, const TA* __res
         den += l_s[w] * wgt[w];
     }
     float inv = 1.0f / den;
-    if (gate) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_stride + h]));
+    if (gate && !gate_wide) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_stride + h]));
     TA* o = out + ((size_t)t * nh + h) * dv;
     for (int c = threadIdx.x; c < dv; c += blockDim.x) {
         float num = 0.f;
 #pragma unroll
         for (int w = 0; w < AG_WARPS; w++) num += acc_s[w * dv + c] * wgt[w];
-        o[c] = from_f32<TA>(num * inv);
+        float r = num * inv;
+        if (gate && gate_wide) r *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_stride + (size_t)h * dv + c]));
+        o[c] = from_f32<TA>(r);
     }
 }
 
-extern "C" int illm_attention_generic(const void* q, int q_stride, const void* kc, const void* vc,
-                                      const int* block_table, int max_pages, const int* token_pos,
-                                      const int* token_seq, void* out, int act_dtype, int T, int nh,
-                                      int nkv, int d, int page_size, int window, float scale,
-                                      int dv, const float* sinks, const float* gate, int gate_stride,
-                                      void* stream) {
+// span: see first_visible; gate_wide: a gate per value channel; softcap 0: none
+extern "C" int illm_attention_generic_ex(const void* q, int q_stride, const void* kc, const void* vc,
+                                         const int* block_table, int max_pages, const int* token_pos,
+                                         const int* token_seq, void* out, int act_dtype, int T, int nh,
+                                         int nkv, int d, int page_size, int span, float scale,
+                                         int dv, const float* sinks, const float* gate, int gate_stride,
+                                         int gate_wide, float softcap, void* stream) {
     if (T <= 0) return 0;
     if (dv <= 0) dv = d;
     if (d <= 0 || d > AG_MAX_D || dv > AG_MAX_D || nkv <= 0 || nh % nkv || nh > 65535) return ILLM_ERR_BAD_ARG;
@@ -151,12 +156,20 @@ extern "C" int illm_attention_generic(const void* q, int q_stride, const void* k
     if (act_dtype == ILLM_BF16)
         illm_launch(attention_generic_kernel<bf16>, dim3(grid), dim3(AG_WARPS * 32), smem, s, 
             (const bf16*)q, q_stride, (const bf16*)kc, (const bf16*)vc, block_table, max_pages,
-            token_pos, token_seq, (bf16*)out, nh, nkv, d, page_size, window, scale, dv, sinks, gate, gate_stride);
+            token_pos, token_seq, (bf16*)out, nh, nkv, d, page_size, span, scale, dv, sinks, gate, gate_stride, gate_wide, softcap);
     else if (act_dtype == ILLM_F32)
         illm_launch(attention_generic_kernel<float>, dim3(grid), dim3(AG_WARPS * 32), smem, s, 
             (const float*)q, q_stride, (const float*)kc, (const float*)vc, block_table, max_pages,
-            token_pos, token_seq, (float*)out, nh, nkv, d, page_size, window, scale, dv, sinks, gate, gate_stride);
+            token_pos, token_seq, (float*)out, nh, nkv, d, page_size, span, scale, dv, sinks, gate, gate_stride, gate_wide, softcap);
     else
         return ILLM_ERR_BAD_ARG;
     return illm_launch_status();
+}
+
+extern "C" int illm_attention_generic(const void* q, int q_stride, const void* kc, const void* vc, const int* block_table, int max_pages,
+                                      const int* token_pos, const int* token_seq, void* out, int act_dtype, int T, int nh, int nkv, int d,
+                                      int page_size, int window, float scale, int dv, const float* sinks, const float* gate, int gate_stride,
+                                      void* stream) {
+    return illm_attention_generic_ex(q, q_stride, kc, vc, block_table, max_pages, token_pos, token_seq, out, act_dtype, T, nh, nkv, d, page_size,
+                                     window, scale, dv, sinks, gate, gate_stride, 0, 0.f, stream);
 }

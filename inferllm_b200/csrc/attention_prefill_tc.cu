@@ -26,7 +26,7 @@
 // which materialises S in float32 and runs four launches over it
 // (src/kern/gpu/kernel_gpu.cu:576-609, :504-536, :78-125).
 // Takes head sizes 64 and 128 and page sizes that are multiples of 64; any number of heads and
-// groups; prompts that start at 0 or continue a sequence; an optional window.  Every wait is
+// groups; prompts that start at 0 or continue a sequence; an optional window or chunks (first_visible).  Every wait is
 // bounded and raises the error word instead of hanging.
 #include <cuda.h>
 #include <math.h>
@@ -185,15 +185,17 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
 // the S block's columns and P V is issued once more with it.  For mixers whose softmax weights are to
 // stay float32; the plain attention passes false and is compiled as before.  `sinks` (float32 [nh]):
 // one more term exp(sink) of the row's denominator, without a value; `gate` (float32,
-// gate[row * gate_stride + head]): the head's output is multiplied by its sigmoid.  Either may be nullptr.
-template <int D, bool WIDE_P>
+// gate[row * gate_stride + head], or with gate_wide gate[row * gate_stride + head * D + channel]): the output is multiplied by
+// its sigmoid.  Either may be nullptr.  CAP: the scaled scores s become cap * tanh(s / cap) before the mask; the kernel
+// then works on capped scores and its scale is log2(e) (cap, and 2 scale log2(e) / cap as cap_x).
+template <int D, bool WIDE_P, bool CAP>
 __global__ void __launch_bounds__(FT_THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table,
                             int max_pages, const int* __restrict__ cu_q, const int* __restrict__ seq_lens,
-                            bf16* __restrict__ out, int nh, int nkv, int page_size, int window,
+                            bf16* __restrict__ out, int nh, int nkv, int page_size, int span,
                             float scale_log2e, int* __restrict__ err, const float* __restrict__ sinks,
-                            const float* __restrict__ gate, int gate_stride) {
+                            const float* __restrict__ gate, int gate_stride, int gate_wide, float cap, float cap_x) {
     constexpr int FT_MMA_WARP = 4, FT_TMA_WARP = 5;
     constexpr int NA = D / 64;                            // 64-channel atoms of the head
     constexpr unsigned Q_TILE = FT_BM * D * 2;            // the query tile: [NA][128 rows][128 B]
@@ -266,7 +268,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int rows = tile < 0 ? 0 : ((qlen - row0 < FT_BM) ? qlen - row0 : FT_BM);   // 0: nothing to do
     const bool has_rows = rows > 0;
     const int first_pos = past + row0, last_pos = first_pos + rows - 1;
-    const int lo_key = (window > 0 && first_pos - window + 1 > 0) ? first_pos - window + 1 : 0;
+    const int lo_key = first_visible(first_pos, span);
     const int jb0 = lo_key / FT_BN;                                        // first key block
     const int n_blocks = has_rows ? last_pos / FT_BN - jb0 + 1 : 0;
     const int* bt = block_table + (size_t)b * max_pages;
@@ -354,6 +356,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int r = threadIdx.x & 127;
         const unsigned lane_addr = tmem + ((unsigned)(warp * 32) << 16);
         const int pos = (r < rows) ? first_pos + r : last_pos;
+        const int lo_pos = first_visible(pos, span);
         float m_ref = -INFINITY, l_run = 0.f;
         bool alive = has_rows;
         for (int i = 0; i < n_blocks && alive; i++) {
@@ -368,12 +371,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tmem_ld32_issue(s_addr, sr);
             tmem_ld32_issue(s_addr + 32, sr + 32);
             tmem_wait_ld<FT_BN>(sr);
-            const bool need_mask = (key0 + FT_BN - 1 > first_pos) || (window > 0);
+            if (CAP) {
+#pragma unroll
+                for (int c = 0; c < FT_BN; c++) sr[c] = __float_as_uint(soft_cap_fast(__uint_as_float(sr[c]), cap, cap_x));
+            }
+            const bool need_mask = (key0 + FT_BN - 1 > first_pos) || (span != 0);
             if (need_mask) {
 #pragma unroll
                 for (int c = 0; c < FT_BN; c++) {
                     const int key = key0 + c;
-                    const bool hide = key > pos || (window > 0 && key < pos - window + 1);
+                    const bool hide = key > pos || key < lo_pos;
                     if (hide) sr[c] = 0xff800000u;      // -inf
                 }
             }
@@ -488,7 +495,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             } else {
                 inv = 1.0f / l_run;
             }
-            if (gate && r < rows) inv *= 1.0f / (1.0f + expf(-gate[(size_t)(q0 + row0 + r) * gate_stride + h]));
+            if (gate && !gate_wide && r < rows) inv *= 1.0f / (1.0f + expf(-gate[(size_t)(q0 + row0 + r) * gate_stride + h]));
             bf16* dst = out + ((size_t)(q0 + row0 + r) * nh + h) * D;
 #pragma unroll 1
             for (int c0 = 0; c0 < D; c0 += 32) {
@@ -501,6 +508,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                         float f[8];
 #pragma unroll
                         for (int e = 0; e < 8; e++) f[e] = __uint_as_float(orr[c + e]) * inv;
+                        if (gate && gate_wide) {
+                            const float* gr = gate + (size_t)(q0 + row0 + r) * gate_stride + (size_t)h * D + c0 + c;
+#pragma unroll
+                            for (int e = 0; e < 8; e++) f[e] *= 1.0f / (1.0f + expf(-gr[e]));
+                        }
                         store8(dst + c0 + c, f);
                     }
                 }
@@ -547,11 +559,11 @@ static int ft_make_map(CUtensorMap* map, const void* ptr, long long rows, long l
     return r == CUDA_SUCCESS ? 0 : ILLM_ERR_BAD_ARG;
 }
 
-template <int D, bool WIDE_P>
+template <int D, bool WIDE_P, bool CAP>
 static int ft_launch(const void* q, int q_stride, int T, const void* kc, const void* vc, long long n_pages,
                      const int* block_table, int max_pages, const int* cu_q, const int* seq_lens, void* out, int B,
-                     int max_q, int nh, int nkv, int page_size, int window, float scale, int* err, const float* sinks,
-                     const float* gate, int gate_stride, cudaStream_t s) {
+                     int max_q, int nh, int nkv, int page_size, int span, float scale, int* err, const float* sinks,
+                     const float* gate, int gate_stride, int gate_wide, float softcap, cudaStream_t s) {
     CUtensorMap mq, mk, mv;
     int rc;
     if ((rc = ft_make_map(&mq, q, T, (long long)nh * D, q_stride, FT_BM)) != 0) return rc;
@@ -560,32 +572,37 @@ static int ft_launch(const void* q, int q_stride, int T, const void* kc, const v
     if ((rc = ft_make_map(&mv, vc, kv_rows, D, D, FT_BN)) != 0) return rc;
     const size_t smem = (size_t)FT_BM * D * 2 + (size_t)(FT_KSTAGES + FT_VSTAGES) * FT_BN * D * 2 +
                         256;   // + barriers and the tensor-memory address
-    auto kern = attention_prefill_tc_kernel<D, WIDE_P>;
+    auto kern = attention_prefill_tc_kernel<D, WIDE_P, CAP>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     dim3 grid(nh, (max_q + FT_BM - 1) / FT_BM, B);
     illm_launch(kern, grid, dim3(FT_THREADS), smem, s, mq, mk, mv, block_table, max_pages, cu_q, seq_lens,
-                (bf16*)out, nh, nkv, page_size, window, scale * 1.4426950408889634f, err, sinks, gate, gate_stride);
+                (bf16*)out, nh, nkv, page_size, span, (CAP ? 1.0f : scale) * 1.4426950408889634f, err, sinks, gate, gate_stride, gate_wide, softcap,
+                CAP ? 2.0f * scale * 1.4426950408889634f / softcap : 0.f);
     return illm_launch_status();
 }
 
 // q: the packed projection [T, q_stride] whose first nh*d columns are the query heads;
-// kc, vc: one cache entry [n_pages, nkv, page_size, d].  wide_p, sinks, gate: see the kernel.
+// kc, vc: one cache entry [n_pages, nkv, page_size, d].  wide_p, sinks, gate, gate_wide, softcap (0: none; needs wide_p): see
+// the kernel; span: see first_visible.
 extern "C" int illm_attention_prefill_tc_ex(const void* q, int q_stride, int T, const void* kc, const void* vc,
                                             long long n_pages, const int* block_table, int max_pages,
                                             const int* cu_q, const int* seq_lens, void* out, int B, int max_q, int nh,
-                                            int nkv, int d, int page_size, int window, float scale, int* err,
-                                            int wide_p, const float* sinks, const float* gate, int gate_stride, void* stream) {
+                                            int nkv, int d, int page_size, int span, float scale, int* err,
+                                            int wide_p, const float* sinks, const float* gate, int gate_stride, int gate_wide,
+                                            float softcap, void* stream) {
     if (B <= 0 || max_q <= 0) return 0;
     if (nkv <= 0 || nh % nkv || max_q > 65535 * FT_BM || B > 65535 || (q_stride & 7) || page_size % 64 ||
         ((uintptr_t)q & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15))
         return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
-#define FT_CASE(DD, WW)                                                                                                   \
-    if (d == DD && (wide_p != 0) == WW)                                                                                   \
-        return ft_launch<DD, WW>(q, q_stride, T, kc, vc, n_pages, block_table, max_pages, cu_q, seq_lens, out, B, max_q, \
-                                 nh, nkv, page_size, window, scale, err, sinks, gate, gate_stride, s);
-    FT_CASE(128, false) FT_CASE(64, false) FT_CASE(128, true) FT_CASE(64, true)
+    if (softcap > 0.f && !wide_p) return ILLM_ERR_BAD_ARG;
+#define FT_CASE(DD, WW, CC)                                                                                                   \
+    if (d == DD && (wide_p != 0) == WW && (softcap > 0.f) == CC)                                                              \
+        return ft_launch<DD, WW, CC>(q, q_stride, T, kc, vc, n_pages, block_table, max_pages, cu_q, seq_lens, out, B, max_q, \
+                                     nh, nkv, page_size, span, scale, err, sinks, gate, gate_stride, gate_wide, softcap, s);
+    FT_CASE(128, false, false) FT_CASE(64, false, false) FT_CASE(128, true, false) FT_CASE(64, true, false)
+    FT_CASE(128, true, true) FT_CASE(64, true, true)
 #undef FT_CASE
     return ILLM_ERR_BAD_ARG;
 }
@@ -596,5 +613,5 @@ extern "C" int illm_attention_prefill_tc(const void* q, int q_stride, int T, con
                                          int nkv, int d, int page_size, int window, float scale, int* err,
                                          void* stream) {
     return illm_attention_prefill_tc_ex(q, q_stride, T, kc, vc, n_pages, block_table, max_pages, cu_q, seq_lens, out, B, max_q, nh, nkv, d,
-                                        page_size, window, scale, err, 0, nullptr, nullptr, 0, stream);
+                                        page_size, window, scale, err, 0, nullptr, nullptr, 0, 0, 0.f, stream);
 }

@@ -44,6 +44,22 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
     return warp_sum(t);
 }
 
+// The first position that the query at position p sees, for a layer whose `span` is 0 (all earlier positions), w > 0
+// (the last w, its own included) or -c < 0 (those of its own chunk of c positions, counted from the sequence's start).
+__device__ __forceinline__ int first_visible(int p, int span) {
+    if (span < 0) return p - p % (-span);
+    return (span > 0 && p - span + 1 > 0) ? p - span + 1 : 0;
+}
+
+// cap * tanh(s / cap) by the special-function unit, for scores that a kernel of the bfloat16 mode made: tanh x =
+// 1 - 2 / (1 + e^(2x)), absolute error a few 2^-23 of the cap.  two_log2e_over_cap = 2 log2(e) / cap.
+__device__ __forceinline__ float soft_cap_fast(float s, float cap, float two_log2e_over_cap) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * two_log2e_over_cap));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return fmaf(-2.0f * cap, r, cap);
+}
+
 // 16-byte loads of 8 bf16 or 4 float into float registers.
 __device__ __forceinline__ void load8(const bf16* p, float* f) {
     uint4 u = *reinterpret_cast<const uint4*>(p);

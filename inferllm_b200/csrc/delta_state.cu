@@ -1,4 +1,4 @@
-// The gated delta rule with a decay per head and key channel, over per-sequence state.
+// The gated delta rule with a decay per head and key channel, or one per head, over per-sequence state.
 //
 // Per head, with the state S [d, dv] float32 (zero when a sequence starts), for every token in order:
 //     S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
@@ -7,7 +7,7 @@
 //                                           tap the token's own, zeros before the sequence's start
 //     q, k     = x / sqrt(sum(x^2) + 1e-6) per head;  q also times q_scale
 //     beta     = sigmoid(b)                 one per head
-//     g        = exp(-exp(A_log_h) * softplus(a + dt_bias))      one per head and key channel
+//     g        = exp(-exp(A_log_h) * softplus(a + dt_bias))      one per head and key channel, or one per head
 // Query/key head of value head h: h / (heads / kv_heads).  The last taps - 1 rows of the raw q, k, v projections
 // are per-sequence state as well ([taps - 1, channels] behind S in a slot's row), renewed by conv_state_kernel
 // after the preparation has read them.  Everything here is float32 in both modes of the engine.
@@ -27,16 +27,17 @@
 struct DeltaArgs {
     const float* x;                 // [T, ld] the packed float32 projection
     int T, prep_tokens, ld, q_off, k_off, v_off, b_off;
-    const float* a;                 // [T, nh * d] decay projection (before the bias)
+    const float* a;                 // decay projection (before the bias): [T, nh * d], or head_decay [T, nh]; rows a_ld apart
+    int a_ld, head_decay;
     int nh, nkv, d, dv, taps;
     const float *conv_q, *conv_k, *conv_v;      // [channels, taps]
-    const float *a_log, *dt_bias;               // [nh], [nh * d]
+    const float *a_log, *dt_bias;               // [nh], [nh * d] or [nh]
     float q_scale;
     float* state;                   // [slots, state_elems]: S [nh, dv, d], then the convolution's rows [taps - 1, C]
     long long state_elems;
     const int *slots, *cu_q, *token_pos, *token_seq, *seq_lens;
     float* qkv;                     // out [T, C] prepared q, k, v (C = 2 nkv d + nh dv)
-    float* g;                       // out [T, nh * d]
+    float* g;                       // out [T, nh * d] or [T, nh]
     float* beta;                    // out [T, nh]
     float* out;                     // [T, nh * dv]
 };
@@ -105,7 +106,7 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(DeltaArgs p) {
     __syncthreads();
     const int seq = p.token_seq[t], pos = p.token_pos[t];
     const int i_step = t - p.cu_q[seq];            // the token's place among the step's tokens of its sequence
-    const int d = p.d, nq = p.nkv * d, nv = p.nh * p.dv, ng = p.nh * d, C = 2 * nq + nv, K = p.taps;
+    const int d = p.d, nq = p.nkv * d, nv = p.nh * p.dv, ng = p.head_decay ? p.nh : p.nh * d, C = 2 * nq + nv, K = p.taps;
     const float* conv_state = p.state + (size_t)p.slots[seq] * p.state_elems + (size_t)p.nh * d * p.dv;
     float* dst = p.qkv + (size_t)t * C;
     const int hpb = delta_heads_per_block(d), qk_units = (2 * p.nkv + hpb - 1) / hpb;
@@ -168,9 +169,9 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(DeltaArgs p) {
         for (int r = 0; r < 4; r++) {
             const int c = (unit - qk_units - v_units) * 1024 + r * 256 + threadIdx.x;
             if (c < ng) {
-                const float z = p.a[(size_t)t * ng + c] + p.dt_bias[c];
+                const float z = p.a[(size_t)t * p.a_ld + c] + p.dt_bias[c];
                 const float sp = z > 20.f ? z : log1pf(expf(z));
-                p.g[(size_t)t * ng + c] = expf(-expf(p.a_log[c / d]) * sp);
+                p.g[(size_t)t * ng + c] = expf(-expf(p.a_log[p.head_decay ? c : c / d]) * sp);
             }
         }
     } else {
@@ -212,7 +213,9 @@ __device__ __forceinline__ void dl_cp4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src));
 }
 
-template <int L, int ROWS>
+// HEAD: one decay per head and token (a number per token in shared memory).  It is then taken out of the first dot product,
+// S^T k of the decayed state = g (S^T k), and the state is decayed while that product is being added over the lanes.
+template <int L, int ROWS, bool HEAD>
 __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
     pdl_grid_sync();
     extern __shared__ __align__(16) float sm[];
@@ -231,9 +234,10 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
         const int i = 4 * (l + L * (r >> 2)) + (r & 3);
         S[r] = (live && i < d) ? S_col[i] : 0.f;
     }
-    // Two buffers of a tile of tokens in shared memory: q, k, g [tile, DPAD] each, v [tile, COLS], beta [tile].  The next
+    // Two buffers of a tile of tokens in shared memory: q, k, g [tile, DPAD] each (HEAD: g [tile]), v [tile, COLS], beta [tile].  The next
     // tile is on its way (cp.async) while this one is computed.  The padding rows beyond d are written once.
-    constexpr int BUF = DL_TILE * (3 * DPAD + COLS + 1);
+    constexpr int GW = HEAD ? 1 : DPAD;
+    constexpr int BUF = DL_TILE * (2 * DPAD + GW + COLS + 1);
     const int j0 = blockIdx.x * COLS;
     const float* __restrict__ qkv = p.qkv;
     const float* __restrict__ gg = p.g;
@@ -244,16 +248,18 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
             const int at = (r / (DPAD - d)) * DPAD + d + r % (DPAD - d);
             sm[bb * BUF + at] = 0.f;
             sm[bb * BUF + DL_TILE * DPAD + at] = 0.f;
-            sm[bb * BUF + 2 * DL_TILE * DPAD + at] = 1.f;
+            if (!HEAD) sm[bb * BUF + 2 * DL_TILE * DPAD + at] = 1.f;
         }
     const bool wide = (d & 3) == 0 && (C & 3) == 0;          // rows of q, k and the decay start on 16-byte boundaries
     auto stage = [&](int buf, int t0) {
         float* sq = sm + buf * BUF;
         float* sk = sq + DL_TILE * DPAD;
         float* sg = sk + DL_TILE * DPAD;
-        float* sv = sg + DL_TILE * DPAD;
+        float* sv = sg + DL_TILE * GW;
         float* sb = sv + DL_TILE * COLS;
         const int nt = min(DL_TILE, n - t0);
+        if (HEAD)
+            for (int e = threadIdx.x; e < nt; e += DL_THREADS) dl_cp4(sg + e, gg + (size_t)(first + t0 + e) * p.nh + h);
         if (wide) {
             const int per_row = d >> 2;
             for (int e = threadIdx.x; e < nt * per_row; e += DL_THREADS) {
@@ -261,7 +267,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
                 const size_t t = (size_t)(first + t0 + tt);
                 dl_cp16(sq + tt * DPAD + i, qkv + t * C + (size_t)hk * d + i);
                 dl_cp16(sk + tt * DPAD + i, qkv + t * C + nq + (size_t)hk * d + i);
-                dl_cp16(sg + tt * DPAD + i, gg + t * p.nh * d + (size_t)h * d + i);
+                if (!HEAD) dl_cp16(sg + tt * DPAD + i, gg + t * p.nh * d + (size_t)h * d + i);
             }
         } else {
             for (int e = threadIdx.x; e < nt * d; e += DL_THREADS) {
@@ -269,7 +275,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
                 const size_t t = (size_t)(first + t0 + tt);
                 dl_cp4(sq + tt * DPAD + i, qkv + t * C + (size_t)hk * d + i);
                 dl_cp4(sk + tt * DPAD + i, qkv + t * C + nq + (size_t)hk * d + i);
-                dl_cp4(sg + tt * DPAD + i, gg + t * p.nh * d + (size_t)h * d + i);
+                if (!HEAD) dl_cp4(sg + tt * DPAD + i, gg + t * p.nh * d + (size_t)h * d + i);
             }
         }
         for (int e = threadIdx.x; e < nt * COLS; e += DL_THREADS) {
@@ -289,7 +295,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
         const float* sq = sm + (it & 1) * BUF;
         const float* sk = sq + DL_TILE * DPAD;
         const float* sg = sk + DL_TILE * DPAD;
-        const float* sv = sg + DL_TILE * DPAD;
+        const float* sv = sg + DL_TILE * GW;
         const float* sb = sv + DL_TILE * COLS;
         for (int tt = 0; tt < nt; tt++) {
             const float4* q4 = reinterpret_cast<const float4*>(sq + tt * DPAD);
@@ -302,13 +308,16 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
                 kk[r] = k4[l + L * r];
                 qq[r] = q4[l + L * r];           // read now, used after the first reduction
             }
+            const float gh = HEAD ? sg[tt] : 1.f;
 #pragma unroll
             for (int r = 0; r < ROWS / 4; r++) {
-                const float4 g = g4[l + L * r];
-                S[4 * r] *= g.x;
-                S[4 * r + 1] *= g.y;
-                S[4 * r + 2] *= g.z;
-                S[4 * r + 3] *= g.w;
+                if (!HEAD) {
+                    const float4 g = g4[l + L * r];
+                    S[4 * r] *= g.x;
+                    S[4 * r + 1] *= g.y;
+                    S[4 * r + 2] *= g.z;
+                    S[4 * r + 3] *= g.w;
+                }
                 a0 = fmaf(kk[r].x, S[4 * r], a0);
                 a1 = fmaf(kk[r].y, S[4 * r + 1], a1);
                 a2 = fmaf(kk[r].z, S[4 * r + 2], a2);
@@ -317,6 +326,11 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
             float acc = (a0 + a1) + (a2 + a3);
 #pragma unroll
             for (int o = L / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+            if (HEAD) {
+#pragma unroll
+                for (int r = 0; r < ROWS; r++) S[r] *= gh;
+                acc *= gh;
+            }
             const float u = sb[tt] * (sv[tt * COLS + jc] - acc);
             a0 = a1 = a2 = a3 = 0.f;
 #pragma unroll
@@ -349,10 +363,10 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
 
 extern "C" int illm_delta_rule_supported(int d, int dv, int taps) { return d >= 1 && d <= 16 * DL_ROWS && dv >= 1 && taps >= 1 && taps <= 64; }
 
-template <int L, int ROWS>
-static void launch_scan(const DeltaArgs& p, int B, int n_sms, cudaStream_t s) {
+template <int L, int ROWS, bool HEAD>
+static void launch_scan_as(const DeltaArgs& p, int B, int n_sms, cudaStream_t s) {
     constexpr int COLS = DL_THREADS / L;
-    size_t smem = (size_t)(2 * DL_TILE * (3 * ROWS * L + COLS + 1)) * sizeof(float);
+    size_t smem = (size_t)(2 * DL_TILE * (2 * ROWS * L + (HEAD ? 1 : ROWS * L) + COLS + 1)) * sizeof(float);
     // The scan is bound by what an SM's shared memory delivers per clock, so its blocks must spread over the SMs.  Launched
     // behind kernels that still hold most SMs, a small grid would be packed onto the few SMs that are free first (measured: 32
     // blocks, 2.5 ms instead of 0.95 ms).  Asking for more shared memory than the tiles need caps the blocks per SM at what an
@@ -365,10 +379,16 @@ static void launch_scan(const DeltaArgs& p, int B, int n_sms, cudaStream_t s) {
     }
     static bool raised = false;
     if (!raised) {
-        cudaFuncSetAttribute(delta_scan_kernel<L, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(delta_scan_kernel<L, ROWS, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         raised = true;
     }
-    illm_launch(delta_scan_kernel<L, ROWS>, dim3((p.dv + COLS - 1) / COLS, p.nh, B), dim3(DL_THREADS), smem, s, p);
+    illm_launch(delta_scan_kernel<L, ROWS, HEAD>, dim3((p.dv + COLS - 1) / COLS, p.nh, B), dim3(DL_THREADS), smem, s, p);
+}
+
+template <int L, int ROWS>
+static void launch_scan(const DeltaArgs& p, int B, int n_sms, cudaStream_t s) {
+    if (p.head_decay) launch_scan_as<L, ROWS, true>(p, B, n_sms, s);
+    else launch_scan_as<L, ROWS, false>(p, B, n_sms, s);
 }
 
 // A column's rows over L lanes of 32 rows each, or, while the grid of ONE sequence then still fits the SMs once, over 2 L
@@ -393,25 +413,26 @@ static void launch_scan_for(const DeltaArgs& p, int B, cudaStream_t s) {
 
 // x: [T, ld] float32 with q at q_off (nkv * d columns), k at k_off, v at v_off (nh * dv), beta's logits at b_off (nh).
 // state: float32 [slots, state_elems], state_elems >= nh * d * dv + (taps - 1) * (2 nkv d + nh dv).
-// Scratch qkv [T, 2 nkv d + nh dv], g [T, nh d], beta [T, nh]; out [T, nh dv].
-extern "C" int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_off, int v_off, int b_off, const float* a, int nh, int nkv, int d,
+// a: the decay projection, rows a_ld apart: nh * d columns, or with head_decay nh.
+// Scratch qkv [T, 2 nkv d + nh dv], g [T, nh d] (head_decay: [T, nh]), beta [T, nh]; out [T, nh dv].
+extern "C" int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_off, int v_off, int b_off, const float* a, int a_ld, int head_decay, int nh, int nkv, int d,
                                int dv, int taps, const float* conv_q, const float* conv_k, const float* conv_v, const float* a_log,
                                const float* dt_bias, float q_scale, float* state, long long state_elems, const int* slots, const int* cu_q,
                                const int* token_pos, const int* token_seq, const int* seq_lens, float* qkv, float* g, float* beta, float* out,
                                int B, void* stream) {
     if (T <= 0 || B <= 0) return 0;
-    if (!illm_delta_rule_supported(d, dv, taps) || nkv <= 0 || nh % nkv) return ILLM_ERR_BAD_ARG;
+    if (!illm_delta_rule_supported(d, dv, taps) || nkv <= 0 || nh % nkv || a_ld < (head_decay ? nh : nh * d)) return ILLM_ERR_BAD_ARG;
     const long long C = 2LL * nkv * d + (long long)nh * dv;
     if (state_elems < (long long)nh * d * dv + (taps - 1) * C) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     DeltaArgs p;
     p.x = x; p.T = T; p.ld = ld; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.b_off = b_off;
-    p.a = a; p.nh = nh; p.nkv = nkv; p.d = d; p.dv = dv; p.taps = taps;
+    p.a = a; p.a_ld = a_ld; p.head_decay = head_decay; p.nh = nh; p.nkv = nkv; p.d = d; p.dv = dv; p.taps = taps;
     p.conv_q = conv_q; p.conv_k = conv_k; p.conv_v = conv_v; p.a_log = a_log; p.dt_bias = dt_bias; p.q_scale = q_scale;
     p.state = state; p.state_elems = state_elems; p.slots = slots; p.cu_q = cu_q; p.token_pos = token_pos; p.token_seq = token_seq;
     p.seq_lens = seq_lens; p.qkv = qkv; p.g = g; p.beta = beta; p.out = out;
     const int hpb = d > 256 ? 1 : 256 / ((d + 31) / 32 * 32);
-    const long long units = (2LL * nkv + hpb - 1) / hpb + ((long long)nh * dv + 1023) / 1024 + ((long long)nh * d + 1023) / 1024 + 1;
+    const long long units = (2LL * nkv + hpb - 1) / hpb + ((long long)nh * dv + 1023) / 1024 + ((long long)nh * (head_decay ? 1 : d) + 1023) / 1024 + 1;
     if (units > 65535) return ILLM_ERR_BAD_ARG;
     p.prep_tokens = T >= 512 ? DL_PREP_TOKENS : 1;
     const dim3 pgrid((T + p.prep_tokens - 1) / p.prep_tokens, (unsigned)units);

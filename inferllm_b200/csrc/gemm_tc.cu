@@ -31,6 +31,15 @@ template <int ACT> __device__ __forceinline__ float tc_gate_act(float g) {
     if (ACT == 3) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
     return g / (1.0f + __expf(-g));
 }
+// the gated output: act(gate) * up, or (ACT 4) the clamped form g = min(gate, limit), u = clamp(up, -limit, limit),
+// g sigmoid(1.702 g) (u + 1)
+template <int ACT> __device__ __forceinline__ float tc_gated(float gate, float up, float limit) {
+    if (ACT == 4) {
+        const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+        return g / (1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+    }
+    return tc_gate_act<ACT>(gate) * up;
+}
 
 // D[ra, rb] = sum_k A[ra, k] B[rb, k];  SWAP = false: C[ra * ldc + rb];  SWAP = true: C[rb * ldc + ra].
 #define TC_MAX_STAGES 12
@@ -39,7 +48,7 @@ template <int BN, bool SWAP, typename TOut, int GATED = 0>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                TOut* __restrict__ C, long long split_stride, int ldc, int RA, int RB, int k_iters_total,
-               int k_iters_per_split, int STAGES, int* __restrict__ err) {
+               int k_iters_per_split, int STAGES, float act_limit, int* __restrict__ err) {
     constexpr unsigned A_BYTES = TC_BM * TC_BK * 2, B_BYTES = BN * TC_BK * 2;
     constexpr unsigned TMEM_COLS = BN < 32 ? 32 : BN;
     constexpr unsigned IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((unsigned)(BN >> 3) << 17) | ((unsigned)(TC_BM >> 4) << 24);
@@ -145,13 +154,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 tmem_ld16(tmem + ((unsigned)(quad * 32) << 16) + (unsigned)c0, v);
                 if (SWAP && GATED) {
                     // weight rows 2i, 2i + 1 are gate and up of output i: neighbouring lanes hold them,
-                    // the even lane writes act(gate) * up (ldc = outputs per token; GATED 1 silu, 2 relu, 3 tanh-form gelu)
+                    // the even lane writes act(gate) * up (ldc = outputs per token; GATED 1 silu, 2 relu, 3 tanh-form gelu, 4 clamped)
 #pragma unroll
                     for (int j = 0; j < 16; j++) {
                         const float up = __shfl_xor_sync(0xffffffffu, v[j], 1);
                         const int rb = rb0 + c0 + j;
                         if (!(lane & 1) && rb < RB && ra + 1 < RA)
-                            store_out<TOut>(Cz + (size_t)rb * ldc + (ra >> 1), tc_gate_act<GATED>(v[j]) * up);
+                            store_out<TOut>(Cz + (size_t)rb * ldc + (ra >> 1), tc_gated<GATED>(v[j], up, act_limit));
                     }
                 } else if (SWAP) {
 #pragma unroll
@@ -242,7 +251,7 @@ static int pick_stages(int stage_bytes, long long n_blocks, int k_iters_per_bloc
 
 template <int BN, bool SWAP, typename TOut, int GATED = 0>
 static int launch_tc(const CUtensorMap& ma, const CUtensorMap& mb, TOut* C, long long split_stride, int ldc,
-                     int RA, int RB, int k_iters, int splits, int* err, cudaStream_t s) {
+                     int RA, int RB, int k_iters, int splits, int* err, cudaStream_t s, float act_limit = 0.f) {
     const int stage_bytes = TC_BM * TC_BK * 2 + BN * TC_BK * 2;
     const int per_split = (k_iters + splits - 1) / splits;
     dim3 grid((RA + TC_BM - 1) / TC_BM, (RB + BN - 1) / BN, splits);
@@ -251,7 +260,7 @@ static int launch_tc(const CUtensorMap& ma, const CUtensorMap& mb, TOut* C, long
     auto kern = gemm_tc_kernel<BN, SWAP, TOut, GATED>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    illm_launch(kern, dim3(grid), dim3(TC_THREADS), smem, s, ma, mb, C, split_stride, ldc, RA, RB, k_iters, per_split, stages, err);
+    illm_launch(kern, dim3(grid), dim3(TC_THREADS), smem, s, ma, mb, C, split_stride, ldc, RA, RB, k_iters, per_split, stages, act_limit, err);
     return illm_launch_status();
 }
 
@@ -315,12 +324,12 @@ extern "C" int illm_gemm_bf16_tc(const void* X, const void* W, void* out, int ou
 }
 
 // Decode-sized product (M <= 64) of a gated feed-forward's packed weight, whose rows are gate and up
-// of an output in turn: out[M, N / 2] = act(gate) * up (act 1 silu, 2 relu, 3 tanh-form gelu) in bfloat16, straight from the accumulator
+// of an output in turn: out[M, N / 2] = act(gate) * up (act 1 silu, 2 relu, 3 tanh-form gelu, 4 clamped with act_limit) in bfloat16, straight from the accumulator
 // (formula src/kern/naive/naive.cpp:80-89), without splitting K.
-extern "C" int illm_gemm_bf16_tc_gated(const void* X, const void* W, void* out, int M, int N, int K, int act, int* err,
-                                       void* stream) {
+extern "C" int illm_gemm_bf16_tc_gated_ex(const void* X, const void* W, void* out, int M, int N, int K, int act, float act_limit, int* err,
+                                          void* stream) {
     if (M <= 0 || N <= 0) return 0;
-    if (M > 64 || (N & 1) || K <= 0 || (K & 7) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15) || act < 1 || act > 3) return ILLM_ERR_BAD_ARG;
+    if (M > 64 || (N & 1) || K <= 0 || (K & 7) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15) || act < 1 || act > 4 || (act == 4 && !(act_limit > 0.f))) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int k_iters = (K + TC_BK - 1) / TC_BK;
     CUtensorMap ma, mb;
@@ -331,14 +340,18 @@ extern "C" int illm_gemm_bf16_tc_gated(const void* X, const void* W, void* out, 
     bf16* o = (bf16*)out;
 #define ILLM_TCG(ACT)                                                                                                \
     do {                                                                                                             \
-        if (bn == 16) return launch_tc<16, true, bf16, ACT>(ma, mb, o, 0, N / 2, N, M, k_iters, 1, err, s);           \
-        if (bn == 32) return launch_tc<32, true, bf16, ACT>(ma, mb, o, 0, N / 2, N, M, k_iters, 1, err, s);           \
-        return launch_tc<64, true, bf16, ACT>(ma, mb, o, 0, N / 2, N, M, k_iters, 1, err, s);                         \
+        if (bn == 16) return launch_tc<16, true, bf16, ACT>(ma, mb, o, 0, N / 2, N, M, k_iters, 1, err, s, act_limit); \
+        if (bn == 32) return launch_tc<32, true, bf16, ACT>(ma, mb, o, 0, N / 2, N, M, k_iters, 1, err, s, act_limit); \
+        return launch_tc<64, true, bf16, ACT>(ma, mb, o, 0, N / 2, N, M, k_iters, 1, err, s, act_limit); \
     } while (0)
     if (act == 2) ILLM_TCG(2);
     if (act == 3) ILLM_TCG(3);
+    if (act == 4) ILLM_TCG(4);
     ILLM_TCG(1);
 #undef ILLM_TCG
+}
+extern "C" int illm_gemm_bf16_tc_gated(const void* X, const void* W, void* out, int M, int N, int K, int act, int* err, void* stream) {
+    return illm_gemm_bf16_tc_gated_ex(X, W, out, M, N, K, act, 0.f, err, stream);
 }
 
 // out[i] = sum over slices (ascending) of ws[z][i]: the stand-alone form of the reduction.

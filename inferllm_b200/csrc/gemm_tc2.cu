@@ -75,11 +75,20 @@ template <int EPI> __device__ __forceinline__ float t2_gate_act(float g) {
     if (EPI == 3) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
     return g / (1.0f + __expf(-g));
 }
+// the gated output: act(gate) * up, or (EPI 4) the clamped form g = min(gate, limit), u = clamp(up, -limit, limit),
+// g sigmoid(1.702 g) (u + 1)
+template <int EPI> __device__ __forceinline__ float t2_gated(float gate, float up, float limit) {
+    if (EPI == 4) {
+        const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+        return g / (1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+    }
+    return t2_gate_act<EPI>(gate) * up;
+}
 
 template <int EPI, typename TOut>
 __global__ void __launch_bounds__(T2_THREADS)
 gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
-                TOut* __restrict__ C, int ldc, int RA, int RB, int k_iters, int* __restrict__ err) {
+                TOut* __restrict__ C, int ldc, int RA, int RB, int k_iters, float act_limit, int* __restrict__ err) {
     constexpr unsigned A_BYTES = TC_BM * TC_BK * 2, B_BYTES = T2_HALF * TC_BK * 2;
     constexpr unsigned TMEM_COLS = 512;
     // M 256 (the pair), N 256, bfloat16 x bfloat16 -> float32, both operands K-major
@@ -194,7 +203,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
                     float v[16], r[8];
                     tmem_ld16(tbase + c0, v);
 #pragma unroll
-                    for (int j = 0; j < 8; j++) r[j] = t2_gate_act<EPI>(v[2 * j]) * v[2 * j + 1];
+                    for (int j = 0; j < 8; j++) r[j] = t2_gated<EPI>(v[2 * j], v[2 * j + 1], act_limit);
                     if (ra < RA) {
                         const int o0 = (rb0 + c0) / 2;
                         TOut* dst = C + (size_t)ra * ldc + o0;
@@ -267,7 +276,7 @@ static int t2_make_map(CUtensorMap* map, const void* ptr, long long rows, long l
 }
 
 template <int EPI, typename TOut>
-static int t2_launch(const void* X, const void* W, TOut* out, int ldc, int M, int N, int K, int* err, cudaStream_t s) {
+static int t2_launch(const void* X, const void* W, TOut* out, int ldc, int M, int N, int K, float act_limit, int* err, cudaStream_t s) {
     CUtensorMap ma, mb;
     int rc;
     if ((rc = t2_make_map(&ma, X, M, K, TC_BM)) != 0) return rc;
@@ -298,22 +307,27 @@ static int t2_launch(const void* X, const void* W, TOut* out, int ldc, int M, in
     cfg.attrs = attr;
     cfg.numAttrs = g_illm_pdl ? 2 : 1;
     g_illm_launches++;
-    cudaLaunchKernelEx(&cfg, kern, ma, mb, out, ldc, M, N, k_iters, err);
+    cudaLaunchKernelEx(&cfg, kern, ma, mb, out, ldc, M, N, k_iters, act_limit, err);
     return illm_launch_status();
 }
 
-// C = X . W^T (epi 0, C [M, N]) or the gated activation of it (epi 1 silu, 2 relu, 3 tanh-form gelu: C [M, N / 2], W's
-// rows gate and up of an output in turn).  X, W 16-byte aligned; K % 8 == 0.
-extern "C" int illm_gemm_bf16_tc2(const void* X, const void* W, void* out, int out_dtype, int epi, int M, int N,
-                                  int K, int* err, void* stream) {
+// C = X . W^T (epi 0, C [M, N]) or the gated activation of it (epi 1 silu, 2 relu, 3 tanh-form gelu, 4 clamped with
+// act_limit: C [M, N / 2], W's rows gate and up of an output in turn).  X, W 16-byte aligned; K % 8 == 0.
+extern "C" int illm_gemm_bf16_tc2_ex(const void* X, const void* W, void* out, int out_dtype, int epi, float act_limit, int M, int N,
+                                     int K, int* err, void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || (K & 7) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return ILLM_ERR_BAD_ARG;
     if (epi >= 1 && (N & 1)) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
-    if (epi == 0 && out_dtype == ILLM_BF16) return t2_launch<0, bf16>(X, W, (bf16*)out, N, M, N, K, err, s);
-    if (epi == 0 && out_dtype == ILLM_F32) return t2_launch<0, float>(X, W, (float*)out, N, M, N, K, err, s);
-    if (epi == 1 && out_dtype == ILLM_BF16) return t2_launch<1, bf16>(X, W, (bf16*)out, N / 2, M, N, K, err, s);
-    if (epi == 2 && out_dtype == ILLM_BF16) return t2_launch<2, bf16>(X, W, (bf16*)out, N / 2, M, N, K, err, s);
-    if (epi == 3 && out_dtype == ILLM_BF16) return t2_launch<3, bf16>(X, W, (bf16*)out, N / 2, M, N, K, err, s);
+    if (epi == 0 && out_dtype == ILLM_BF16) return t2_launch<0, bf16>(X, W, (bf16*)out, N, M, N, K, act_limit, err, s);
+    if (epi == 0 && out_dtype == ILLM_F32) return t2_launch<0, float>(X, W, (float*)out, N, M, N, K, act_limit, err, s);
+    if (epi == 1 && out_dtype == ILLM_BF16) return t2_launch<1, bf16>(X, W, (bf16*)out, N / 2, M, N, K, act_limit, err, s);
+    if (epi == 2 && out_dtype == ILLM_BF16) return t2_launch<2, bf16>(X, W, (bf16*)out, N / 2, M, N, K, act_limit, err, s);
+    if (epi == 3 && out_dtype == ILLM_BF16) return t2_launch<3, bf16>(X, W, (bf16*)out, N / 2, M, N, K, act_limit, err, s);
+    if (epi == 4 && out_dtype == ILLM_BF16 && act_limit > 0.f) return t2_launch<4, bf16>(X, W, (bf16*)out, N / 2, M, N, K, act_limit, err, s);
     return ILLM_ERR_BAD_ARG;
+}
+
+extern "C" int illm_gemm_bf16_tc2(const void* X, const void* W, void* out, int out_dtype, int epi, int M, int N, int K, int* err, void* stream) {
+    return illm_gemm_bf16_tc2_ex(X, W, out, out_dtype, epi, 0.f, M, N, K, err, stream);
 }

@@ -20,7 +20,7 @@ int illm_attention_decode_gqa(const void* q, int q_stride, const void* kc, const
 
 // attention_decode_ring.cu
 int illm_attention_decode_ring(const void* q, int q_stride, const void* kc, const void* vc, long long n_pages, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, float* part_acc, float* part_ml, void* out, int T, int nh, int nkv, int d, int page_size, int window, float scale, int n_splits, int* err, void* stream);
-int illm_attention_decode_ring_ex(const void* q, int q_stride, const void* kc, const void* vc, long long n_pages, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, float* part_acc, float* part_ml, void* out, int T, int nh, int nkv, int d, int page_size, int window, float scale, int n_splits, int* err, int wide_p, const float* sinks, const float* gate, int gate_stride, void* stream);
+int illm_attention_decode_ring_ex(const void* q, int q_stride, const void* kc, const void* vc, long long n_pages, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, float* part_acc, float* part_ml, void* out, int T, int nh, int nkv, int d, int page_size, int window, float scale, int n_splits, int* err, int wide_p, const float* sinks, const float* gate, int gate_stride, int gate_wide, float softcap, void* stream);
 int illm_attention_decode_ring_rope(const void* qkv, const float* partials, int splits, long long split_stride, const float* cos_sin, int rot, int table_positions, int write_kv, void* kc, void* vc, long long n_pages, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, float* part_acc, float* part_ml, void* out, int T, int nh, int nkv, int d, int page_size, int window, float scale, int n_splits, int* err, int* step_err, void* stream);
 
 // attention_generic.cu
@@ -47,14 +47,14 @@ int illm_gated_scan(const float* x, int T, int ld, int q_off, int k_off, int v_o
 int illm_group_norm_gate_ex(const float* o, int T, int width, int group, const float* w, int w_len, float eps, const float* gate, int gate_ld, int gate_act, int gate_first, const float* row_scale, int head, const float* skip_w, const float* skip_x, int skip_ld, void* y, int act_dtype, void* stream);
 int illm_group_norm_gate(const float* o, int T, int width, int group, const float* w, int w_len, float eps, const float* gate, int gate_ld, int gate_act, void* y, int act_dtype, void* stream);
 
-int illm_attention_prefill_tc_ex(const void* q, int q_stride, int T, const void* kc, const void* vc, long long n_pages, const int* block_table, int max_pages, const int* cu_q, const int* seq_lens, void* out, int B, int max_q, int nh, int nkv, int d, int page_size, int window, float scale, int* err, int wide_p, const float* sinks, const float* gate, int gate_stride, void* stream);
+int illm_attention_prefill_tc_ex(const void* q, int q_stride, int T, const void* kc, const void* vc, long long n_pages, const int* block_table, int max_pages, const int* cu_q, const int* seq_lens, void* out, int B, int max_q, int nh, int nkv, int d, int page_size, int window, float scale, int* err, int wide_p, const float* sinks, const float* gate, int gate_stride, int gate_wide, float softcap, void* stream);
 
 // bigram_embedding.cu
 int illm_bigram_embedding(const int* ids, const int* token_pos, const int* token_seq, const int* cu_q, const int* slots, int* last_token, const void* table, const void* bigram, int table_dtype, float* out, int T, int B, int H, int V, int buckets, long long mul_prev, long long mul_cur, int* err, void* stream);
 
 // delta_state.cu
 int illm_delta_rule_supported(int d, int dv, int taps);
-int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_off, int v_off, int b_off, const float* a, int nh, int nkv, int d, int dv, int taps, const float* conv_q, const float* conv_k, const float* conv_v, const float* a_log, const float* dt_bias, float q_scale, float* state, long long state_elems, const int* slots, const int* cu_q, const int* token_pos, const int* token_seq, const int* seq_lens, float* qkv, float* g, float* beta, float* out, int B, void* stream);
+int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_off, int v_off, int b_off, const float* a, int a_ld, int head_decay, int nh, int nkv, int d, int dv, int taps, const float* conv_q, const float* conv_k, const float* conv_v, const float* a_log, const float* dt_bias, float q_scale, float* state, long long state_elems, const int* slots, const int* cu_q, const int* token_pos, const int* token_seq, const int* seq_lens, float* qkv, float* g, float* beta, float* out, int B, void* stream);
 
 // gated_state.cu
 int illm_mlstm_gates(const float* x, int T, int ld, int q_off, int k_off, int i_off, int f_off, const float* i_bias, const float* f_bias, float cap, float q_scale, int nh, int d, float* state, long long state_stride, long long n_off, long long m_off, const int* slots, const int* cu_q, float* ga, float* gb, float* scale, int B, void* stream);
@@ -67,7 +67,7 @@ int illm_layernorm_sandwich(float* x, const float* y, const float* wb, const flo
 int illm_short_conv(const float* x, int T, int ldx, int x_off, int C, int taps, const float* w, const float* bias, int act, int residual, float* state, long long state_stride, long long state_off, const int* slots, const int* cu_q, const int* token_seq, int B, void* out, int out_dtype, int ldo, int o_off, int update_state, void* stream);
 
 // latent_attention.cu
-int illm_latent_prep(const float* x, int ld, int Q, int R, const float* wq, const float* wkv, float eps, const int* token_pos, const int* token_seq, const int* block_table, int max_pages, int page_size, void* cq_out, void* kc, int act_dtype, int T, int* err, void* stream);
+int illm_latent_prep(const float* x, int ld, int Q, int R, const float* wq, const float* wkv, float eps, const int* token_pos, const int* token_seq, const int* block_table, int max_pages, int page_size, void* cq_out, void* kc, int act_dtype, int T, int* err, int dr, const float* cos_sin, int rot, int pairs, int n_pos, void* stream);
 int illm_latent_attention_any(const void* q, const void* kc, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, void* out, int act_dtype, int T, int H, int R, int page_size, int window, float scale, void* stream);
 int illm_head_gemm(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int y_dtype, int T, int heads, int N, int K, int nn, void* stream);
 
@@ -160,6 +160,13 @@ int illm_latent_rope_prep(const float* x, int ld, int q_off, int H, int d, int d
 // stream_ops.cu
 int illm_add_bias(void* y, int dtype, const float* b, int T, int H, void* stream);
 int illm_scaled_add_rmsnorm(float* resid, const float* delta, const float* ls, const float* w, void* y, int act_dtype, int T, int H, float eps, void* stream);
+int illm_attention_generic_ex(const void* q, int q_stride, const void* kc, const void* vc, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, void* out, int act_dtype, int T, int nh, int nkv, int d, int page_size, int span, float scale, int dv, const float* sinks, const float* gate, int gate_stride, int gate_wide, float softcap, void* stream);
+int illm_qk_prep_mix(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq, const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot, int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages, int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every, const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, void* stream);
+int illm_gemm_bf16_tc_gated_ex(const void* X, const void* W, void* out, int M, int N, int K, int act, float act_limit, int* err, void* stream);
+int illm_gemm_bf16_tc2_ex(const void* X, const void* W, void* out, int out_dtype, int epi, float act_limit, int M, int N, int K, int* err, void* stream);
+int illm_gated_act_ex(const void* gu, void* out, int act_dtype, int T, int I, int act, float limit, void* stream);
+int illm_soft_cap(float* x, long long n, float cap, void* stream);
+int illm_norm_sandwich(float* x, const float* y, const float* wb, const float* w, void* out, int out_dtype, const int* rows, int n_rows, int H, float eps, int write_x, int center, float post_scale, void* stream);
 
 #ifdef __cplusplus
 }

@@ -3,7 +3,9 @@
 // latent_prep_kernel: from a token's packed float32 projection [query latent (Q), key/value latent (R)]:
 //     c_q = rmsnorm(x[0:Q]) * w_q   -> a [T, Q] matrix of the activation dtype (what the query up-projection reads)
 //     c   = rmsnorm(x[Q:Q+R]) * w_kv -> the token's row of the cache's key pages (one head of R channels)
-// Only c is cached: keys and values of every head are linear maps of it, k_h = U_k,h c and v_h = U_v,h c, so
+// With a shared rotated key part (dr > 0), x has dr more columns behind the latent's, which are rotated by the token's
+// position and stored behind c (a cache row of R + dr channels); see latent_rope_prep_kernel for the queries' side.
+// Only this row is cached: keys and values of every head are linear maps of it, k_h = U_k,h c and v_h = U_v,h c, so
 //     score_h = q_h . (U_k,h c) = (U_k,h^T q_h) . c        and        o_h = U_v,h (sum_j p_j c_j)
 // and attention runs as one shared key/value head of R channels (the cached c is key and value at once) with
 // queries U_k,h^T q_h, followed by U_v,h on its output.  Those two per-head maps are head_gemm_kernel:
@@ -13,11 +15,32 @@
 // do not depend on what else is in the step.
 #include "common.cuh"
 
+// channel e of the vector v whose first `rot` channels are turned by the angles of cs (rot / 2 pairs of (cos, sin)):
+// interleaved pairs or rotate-half
+__device__ __forceinline__ float latent_turned(const float* v, int e, int rot, int pairs, const float* cs) {
+    if (e >= rot) return v[e];
+    int j, partner;
+    bool first;
+    if (pairs) {
+        j = e >> 1;
+        first = !(e & 1);
+        partner = e ^ 1;
+    } else {
+        const int half = rot >> 1;
+        first = e < half;
+        j = first ? e : e - half;
+        partner = first ? e + half : e - half;
+    }
+    const float c = cs[2 * j], s = cs[2 * j + 1];
+    return first ? v[e] * c - v[partner] * s : v[e] * c + v[partner] * s;
+}
+
 template <typename TA>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(const float* __restrict__ x, int ld, int Q, int R, const float* __restrict__ wq, const float* __restrict__ wkv, float eps,
                    const int* __restrict__ token_pos, const int* __restrict__ token_seq, const int* __restrict__ block_table, int max_pages,
-                   int page_size, TA* __restrict__ cq_out, TA* __restrict__ kc, int* __restrict__ err) {
+                   int page_size, TA* __restrict__ cq_out, TA* __restrict__ kc, int* __restrict__ err, int dr, const float* __restrict__ cos_sin,
+                   int rot, int pairs, int n_pos) {
     pdl_grid_sync();
     __shared__ float scratch[32];
     const int t = blockIdx.x;
@@ -36,22 +59,31 @@ latent_prep_kernel(const float* __restrict__ x, int ld, int Q, int R, const floa
         if (threadIdx.x == 0) atomicExch(err, 2);
         return;
     }
-    TA* dst = kc + ((size_t)page * page_size + pos % page_size) * R;
+    TA* dst = kc + ((size_t)page * page_size + pos % page_size) * (R + dr);
     for (int c = threadIdx.x; c < R; c += blockDim.x) dst[c] = from_f32<TA>((row[Q + c] * ik) * wkv[c]);
+    if (dr == 0) return;
+    int p = pos;
+    if (rot && (p < 0 || p >= n_pos)) {
+        if (threadIdx.x == 0) atomicExch(err, 3);
+        p = 0;
+    }
+    const float* cs = rot ? cos_sin + (size_t)p * rot : nullptr;
+    for (int e = threadIdx.x; e < dr; e += blockDim.x) dst[R + e] = from_f32<TA>(latent_turned(row + Q + R, e, rot, pairs, cs));
 }
 
 extern "C" int illm_latent_prep(const float* x, int ld, int Q, int R, const float* wq, const float* wkv, float eps, const int* token_pos,
                                 const int* token_seq, const int* block_table, int max_pages, int page_size, void* cq_out, void* kc,
-                                int act_dtype, int T, int* err, void* stream) {
+                                int act_dtype, int T, int* err, int dr, const float* cos_sin, int rot, int pairs, int n_pos,
+                                void* stream) {
     if (T <= 0) return 0;
-    if (Q <= 0 || R <= 0 || !x || !cq_out || !wq || !wkv) return ILLM_ERR_BAD_ARG;
+    if (Q <= 0 || R <= 0 || !x || !cq_out || !wq || !wkv || dr < 0 || rot < 0 || rot > dr || (rot & 1) || (rot && !cos_sin)) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     if (act_dtype == ILLM_BF16)
         illm_launch(latent_prep_kernel<bf16>, dim3(T), dim3(256), 0, s, x, ld, Q, R, wq, wkv, eps, token_pos, token_seq, block_table, max_pages,
-                    page_size, (bf16*)cq_out, (bf16*)kc, err);
+                    page_size, (bf16*)cq_out, (bf16*)kc, err, dr, cos_sin, rot, pairs, n_pos);
     else if (act_dtype == ILLM_F32)
         illm_launch(latent_prep_kernel<float>, dim3(T), dim3(256), 0, s, x, ld, Q, R, wq, wkv, eps, token_pos, token_seq, block_table,
-                    max_pages, page_size, (float*)cq_out, (float*)kc, err);
+                    max_pages, page_size, (float*)cq_out, (float*)kc, err, dr, cos_sin, rot, pairs, n_pos);
     else
         return ILLM_ERR_BAD_ARG;
     return illm_launch_status();
@@ -83,23 +115,7 @@ latent_rope_prep_kernel(const float* __restrict__ x, int ld, int q_off, int H, i
         p = 0;
     }
     const float* cs = rot ? cos_sin + (size_t)p * rot : nullptr;      // rot / 2 pairs of (cos, sin)
-    auto turned = [&](const float* v, int e) {       // channel e of the dr-vector v after the rotation
-        if (e >= rot) return v[e];
-        int j, partner;
-        bool first;
-        if (pairs) {
-            j = e >> 1;
-            first = !(e & 1);
-            partner = e ^ 1;
-        } else {
-            const int half = rot >> 1;
-            first = e < half;
-            j = first ? e : e - half;
-            partner = first ? e + half : e - half;
-        }
-        const float c = cs[2 * j], s = cs[2 * j + 1];
-        return first ? v[e] * c - v[partner] * s : v[e] * c + v[partner] * s;
-    };
+    auto turned = [&](const float* v, int e) { return latent_turned(v, e, rot, pairs, cs); };       // channel e of the dr-vector v
     for (int i = threadIdx.x; i < H * d; i += blockDim.x) {
         const int h = i / d, c = i - h * d;
         q_nope[(size_t)t * H * d + i] = from_f32<TQ>(row[q_off + h * (d + dr) + c]);

@@ -10,6 +10,9 @@
 //   q goes to q_out [T, nh d] in the activation dtype; k and v go into the token's place in the pages
 //       (k: [pages, nkv, page_size, d], v: [pages, nkv, page_size, dv]) if there are pages to write.
 //
+// Values may be mixed with another layer's values of the same tokens, v <- (1 - lambda) v + lambda v_first (v_first
+// float32 rows, lambda one number on the device), and a layer's own, unmixed values may be kept for later layers (v_keep).
+//
 // A layer that attends to another layer's keys and values passes k_off < 0: only q is made.  A layer whose keys are
 // also its values passes v_off < 0: k alone is stored.
 // Everything is float32 until the stores.  One block per token; the sums have a fixed order.
@@ -29,6 +32,10 @@ struct QkPrepArgs {
     int* err;
     float qt_coef;      // query temperature: q *= 1 + qt_coef * ln((p + 1) / qt_every + 1), the division whole-numbered
     int qt_every;       // 0: none
+    const float* v_first;       // [T, v_first_ld] or nullptr
+    int v_first_ld;
+    const float* v_lambda;
+    float* v_keep;              // [T, nkv dv] or nullptr
 };
 
 __device__ __forceinline__ float rotated(const float* buf, int e, int rot, int pairs, const float* cs) {
@@ -110,10 +117,13 @@ __global__ void __launch_bounds__(256) qk_prep_kernel(QkPrepArgs a) {
     }
     if (a.v_off < 0) return;        // the keys are also the values: nothing else to store
     const int nv = a.nkv * a.dv;
+    const float lambda = a.v_first ? *a.v_lambda : 0.f;
     for (int c = threadIdx.x; c < nv; c += blockDim.x) {
         const int hk = c / a.dv, e = c - hk * a.dv;
         float v = to_f32(x[a.v_off + c]);
         if (a.bv) v += a.bv[c];
+        if (a.v_keep) a.v_keep[(size_t)t * nv + c] = v;
+        if (a.v_first) v = (1.0f - lambda) * v + lambda * a.v_first[(size_t)t * a.v_first_ld + c];
         ((TA*)a.vc)[(((size_t)page * a.nkv + hk) * a.page_size + slot) * a.dv + e] = from_f32<TA>(v);
     }
 }
@@ -124,6 +134,12 @@ extern "C" int illm_qk_prep_ex(const void* x, int x_dtype, int ld, int q_off, in
                                int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
                                int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
                                void* stream);
+// the same with mixed values (v_first nullptr: none) and the layer's own values kept (v_keep nullptr: not)
+extern "C" int illm_qk_prep_mix(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq,
+                                const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot,
+                                int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
+                                int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
+                                const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, void* stream);
 extern "C" int illm_qk_prep(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq,
                             const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot,
                             int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
@@ -136,12 +152,21 @@ extern "C" int illm_qk_prep_ex(const void* x, int x_dtype, int ld, int q_off, in
                                int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
                                int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
                                void* stream) {
+    return illm_qk_prep_mix(x, x_dtype, ld, q_off, k_off, v_off, nh, nkv, d, dv, bq, bk, bv, wq, wk, eps, cos_sin, rot, pairs, n_pos, token_pos, token_seq,
+                            block_table, max_pages, page_size, q_out, kc, vc, act_dtype, T, err, qt_coef, qt_every, nullptr, 0, nullptr, nullptr, stream);
+}
+extern "C" int illm_qk_prep_mix(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq,
+                                const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot,
+                                int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
+                                int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
+                                const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, void* stream) {
     if (T <= 0) return 0;
-    if (qt_every < 0) return ILLM_ERR_BAD_ARG;
+    if (qt_every < 0 || (v_first && (!v_lambda || v_first_ld < nkv * dv)) || ((v_first || v_keep) && (k_off < 0 || v_off < 0 || !vc))) return ILLM_ERR_BAD_ARG;
     if (nh <= 0 || d <= 0 || rot < 0 || rot > d || (rot & 1) || (rot && !cos_sin) || !x || !q_out) return ILLM_ERR_BAD_ARG;
     if (k_off >= 0 && (nkv <= 0 || dv <= 0)) return ILLM_ERR_BAD_ARG;      // v_off < 0 with k_off >= 0: keys alone are stored
     QkPrepArgs a{x, ld, q_off, k_off, v_off, nh, nkv, d, dv, bq, bk, bv, wq, wk, eps, cos_sin, rot, pairs, n_pos,
-                 token_pos, token_seq, block_table, max_pages, page_size, q_out, kc, vc, err, qt_coef, qt_every};
+                 token_pos, token_seq, block_table, max_pages, page_size, q_out, kc, vc, err, qt_coef, qt_every,
+                 v_first, v_first_ld, v_lambda, v_keep};
     const size_t smem = (size_t)(nh * d + (k_off >= 0 ? nkv * d : 0)) * sizeof(float);
     if (smem > 200 * 1024) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;

@@ -1,11 +1,13 @@
 // Small element-wise kernels between matrix products.
 //
 // gated_act:    out[t, i] = act(gu[t, 2i]) * gu[t, 2i + 1]  for the activations that the fused silu kernels do not
-//               cover (act 1: silu, 2: relu, 3: tanh-form gelu); the packed projection holds gate and up of an
+//               cover (act 1: silu, 2: relu, 3: tanh-form gelu, 4: clamped, g = min(gate, limit), u = clamp(up, -limit,
+//               limit), g sigmoid(1.702 g) (u + 1)); the packed projection holds gate and up of an
 //               output next to each other, as in swiglu.cu.
 // take_columns: y[t, :] = x[t, off : off + n] of a float32 matrix with row stride ld, as a contiguous matrix of
 //               the activation dtype (what a second, low-rank product reads).
 // join_rows:    y[t, :] = [a[t, :], b[t, :]] of two float32 matrices of equal width, in the activation dtype.
+// soft_cap:     x = cap * tanh(x / cap), in place, of a float32 array (a head's logits).
 #include "common.cuh"
 
 __device__ __forceinline__ float gate_act_of(float v, int act) {
@@ -16,26 +18,34 @@ __device__ __forceinline__ float gate_act_of(float v, int act) {
 }
 
 template <typename TA>
-__global__ void gated_act_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int I, long long n, int act) {
+__global__ void gated_act_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int I, long long n, int act, float limit) {
     pdl_grid_sync();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
     const long long t = i / I;
     const int c = (int)(i - t * I);
     const float g = to_f32(gu[t * 2 * I + 2 * c]), u = to_f32(gu[t * 2 * I + 2 * c + 1]);
+    if (act == 4) {
+        const float a = fminf(g, limit), b = fminf(fmaxf(u, -limit), limit);
+        out[i] = from_f32<TA>(a / (1.0f + expf(-1.702f * a)) * (b + 1.0f));
+        return;
+    }
     out[i] = from_f32<TA>(gate_act_of(g, act) * u);
 }
 
-extern "C" int illm_gated_act(const void* gu, void* out, int act_dtype, int T, int I, int act, void* stream) {
+extern "C" int illm_gated_act_ex(const void* gu, void* out, int act_dtype, int T, int I, int act, float limit, void* stream) {
     if (T <= 0 || I <= 0) return 0;
-    if (act < 1 || act > 3) return ILLM_ERR_BAD_ARG;
+    if (act < 1 || act > 4 || (act == 4 && !(limit > 0.f))) return ILLM_ERR_BAD_ARG;
     const long long n = (long long)T * I;
     const unsigned blocks = (unsigned)((n + 255) / 256);
     cudaStream_t s = (cudaStream_t)stream;
-    if (act_dtype == ILLM_BF16) illm_launch(gated_act_kernel<bf16>, dim3(blocks), dim3(256), 0, s, (const bf16*)gu, (bf16*)out, I, n, act);
-    else if (act_dtype == ILLM_F32) illm_launch(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, s, (const float*)gu, (float*)out, I, n, act);
+    if (act_dtype == ILLM_BF16) illm_launch(gated_act_kernel<bf16>, dim3(blocks), dim3(256), 0, s, (const bf16*)gu, (bf16*)out, I, n, act, limit);
+    else if (act_dtype == ILLM_F32) illm_launch(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, s, (const float*)gu, (float*)out, I, n, act, limit);
     else return ILLM_ERR_BAD_ARG;
     return illm_launch_status();
+}
+extern "C" int illm_gated_act(const void* gu, void* out, int act_dtype, int T, int I, int act, void* stream) {
+    return illm_gated_act_ex(gu, out, act_dtype, T, I, act, 0.f, stream);
 }
 
 template <typename TA>
@@ -227,5 +237,20 @@ extern "C" int illm_add_bias(void* y, int dtype, const float* b, int T, int H, v
     if (dtype == ILLM_BF16) illm_launch(add_bias_kernel<bf16>, dim3(blocks), dim3(256), 0, s, (bf16*)y, b, H, n);
     else if (dtype == ILLM_F32) illm_launch(add_bias_kernel<float>, dim3(blocks), dim3(256), 0, s, (float*)y, b, H, n);
     else return ILLM_ERR_BAD_ARG;
+    return illm_launch_status();
+}
+
+__global__ void soft_cap_kernel(float* __restrict__ x, long long n, float cap) {
+    pdl_grid_sync();
+    const float inv = 1.0f / cap;
+    const long long step = (long long)gridDim.x * blockDim.x;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += step) x[i] = cap * tanhf(x[i] * inv);
+}
+
+extern "C" int illm_soft_cap(float* x, long long n, float cap, void* stream) {
+    if (n <= 0) return 0;
+    if (!x || !(cap > 0.f)) return ILLM_ERR_BAD_ARG;
+    const long long blocks = (n + 255) / 256;
+    illm_launch(soft_cap_kernel, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, (cudaStream_t)stream, x, n, cap);
     return illm_launch_status();
 }

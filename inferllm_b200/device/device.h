@@ -67,6 +67,7 @@ public:
     void* alloc(size_t bytes);                 // from the current lane; 256-byte aligned; valid until that lane is rewound
     template <typename T> T* alloc_n(size_t n) { return (T*)alloc(n * sizeof(T)); }
     void arena_rewind();                       // a new step begins: all lanes rewound, lane 0 current
+    int lane() const { return lane_; }
     void set_lane(int lane, bool rewind);      // allocate from this lane from now on (rewound first if asked)
     void arena_release();                      // give all blocks back to the driver (only while no captured graph uses them)
     size_t arena_bytes() const;                // what the arena holds from the driver

@@ -141,8 +141,8 @@ Mat embedding_scaled(Device& dev, const StepView& ctx, const Mat& table, float s
     return out;
 }
 
-Mat layernorm_sandwich(Device& dev, const Mat& resid, const Mat* delta, const Mat* post_w, const Mat* w, float eps, DType out_dtype, const int* rows,
-                       long long n_rows) {
+Mat norm_sandwich(Device& dev, const Mat& resid, const Mat* delta, const Mat* post_w, const Mat* w, float eps, DType out_dtype, const int* rows,
+                  long long n_rows, bool center, float post_scale) {
     need(resid, "the residual stream", true, DType::F32);
     const long long H = resid.cols, n = rows ? n_rows : resid.rows;
     if (delta) {
@@ -154,10 +154,10 @@ Mat layernorm_sandwich(Device& dev, const Mat& resid, const Mat* delta, const Ma
     if (H > kMaxNormWidth) throw KernelError("layernorm: rows of " + std::to_string(H) + " elements are beyond the kernel");
     Mat y;
     if (w) y = new_mat(dev, n, H, out_dtype);
-    check_kernel(illm_layernorm_sandwich((float*)resid.p, delta ? (const float*)delta->p : nullptr, delta ? (const float*)post_w->p : nullptr,
+    check_kernel(illm_norm_sandwich((float*)resid.p, delta ? (const float*)delta->p : nullptr, delta ? (const float*)post_w->p : nullptr,
                                          w ? (const float*)w->p : nullptr, w ? y.p : nullptr, w ? code_of(out_dtype, "layernorm") : 0, rows, (int)n,
-                                         (int)H, eps, rows == nullptr ? 1 : 0, dev.stream()),
-                 "layernorm_sandwich");
+                                         (int)H, eps, rows == nullptr ? 1 : 0, center ? 1 : 0, post_scale, dev.stream()),
+                 "norm_sandwich");
     return y;
 }
 
@@ -310,11 +310,11 @@ MatOrPartials gemm_bf16_tc(Device& dev, const Mat& x, const Mat& w, DType out_dt
     return r;
 }
 
-Mat gemm_bf16_tc2(Device& dev, const Mat& x, const Mat& w, DType out_dtype, bool gated, int act) {
+Mat gemm_bf16_tc2(Device& dev, const Mat& x, const Mat& w, DType out_dtype, bool gated, int act, float act_limit) {
     check_product(x, w, "gemm_bf16_tc2", gated);
     const long long M = x.rows, K = x.cols, N = w.rows;
     Mat out = new_mat(dev, M, gated ? N / 2 : N, out_dtype);
-    check_kernel(illm_gemm_bf16_tc2(x.p, w.p, out.p, code_of(out_dtype, "gemm_bf16_tc2"), gated ? act : 0, (int)M, (int)N, (int)K,
+    check_kernel(illm_gemm_bf16_tc2_ex(x.p, w.p, out.p, code_of(out_dtype, "gemm_bf16_tc2"), gated ? act : 0, act_limit, (int)M, (int)N, (int)K,
                                     dev.tc_error_word(), dev.stream()),
                  "gemm_bf16_tc2");
     return out;
@@ -349,8 +349,9 @@ MatOrPartials linear(Device& dev, GemmBackend backend, const Mat& x, const Mat& 
     return r;
 }
 
-Mat linear_gated(Device& dev, GemmBackend backend, const Mat& x, const Mat& w, int act) {
-    if (act < kActSilu || act > kActGeluTanh) throw KernelError("linear_gated: unknown activation");
+Mat linear_gated(Device& dev, GemmBackend backend, const Mat& x, const Mat& w, int act, float act_limit) {
+    if (act < kActSilu || act > kActSwishClamped) throw KernelError("linear_gated: unknown activation");
+    if (act == kActSwishClamped && !(act_limit > 0.f)) throw KernelError("linear_gated: the clamped activation needs a positive limit");
     const long long M = x.rows, K = x.cols, N = w.rows;
     if (x.dtype == DType::BF16 && w.dtype == DType::BF16 && M > 0 && K % 8 == 0 && N % 2 == 0 && !((uintptr_t)x.p & 15) &&
         !((uintptr_t)w.p & 15)) {
@@ -358,18 +359,18 @@ Mat linear_gated(Device& dev, GemmBackend backend, const Mat& x, const Mat& w, i
         if (tc && M <= 64 && gemm_tc_splits(M, N, K, dev.n_sms()) == 1) {
             check_product(x, w, "gemm_bf16_tc_gated", true);
             Mat out = new_mat_exact(dev, M, N / 2, DType::BF16);
-            check_kernel(illm_gemm_bf16_tc_gated(x.p, w.p, out.p, (int)M, (int)N, (int)K, act, dev.tc_error_word(), dev.stream()),
+            check_kernel(illm_gemm_bf16_tc_gated_ex(x.p, w.p, out.p, (int)M, (int)N, (int)K, act, act_limit, dev.tc_error_word(), dev.stream()),
                          "gemm_bf16_tc_gated");
             return out;
         }
         if (N >= 256 && ((backend == GemmBackend::TC && M > 128) || (backend == GemmBackend::Auto && M >= kGatedPromptsOnTcMinTokens)))
-            return gemm_bf16_tc2(dev, x, w, DType::BF16, true, act);
+            return gemm_bf16_tc2(dev, x, w, DType::BF16, true, act, act_limit);
     }
     if (act == kActSilu) return swiglu(dev, linear(dev, backend, x, w, x.dtype, true));
     Mat gu = linear(dev, backend, x, w, x.dtype, false).m;
     if (gu.cols % 2) throw KernelError("gated activation: the packed projection must have an even number of columns");
     Mat out = new_mat(dev, gu.rows, gu.cols / 2, gu.dtype);
-    check_kernel(illm_gated_act(gu.p, out.p, code_of(gu.dtype, "gated_act"), (int)gu.rows, (int)(gu.cols / 2), act, dev.stream()), "gated_act");
+    check_kernel(illm_gated_act_ex(gu.p, out.p, code_of(gu.dtype, "gated_act"), (int)gu.rows, (int)(gu.cols / 2), act, act_limit, dev.stream()), "gated_act");
     return out;
 }
 
@@ -432,10 +433,11 @@ Mat attention_generic(Device& dev, const Mat& qkv, const KVView& kv, const StepV
     need(qkv, "qkv");
     check_cache(kv, qkv.dtype, g, "attention_generic");
     Mat out = new_mat(dev, qkv.rows, (long long)g.n_heads * dv, qkv.dtype);
-    check_kernel(illm_attention_generic(qkv.p, (int)qkv.cols, kv.k, kv.v, kv.block_table, kv.width, ctx.token_pos, ctx.token_seq, out.p,
-                                        code_of(qkv.dtype, "attention_generic"), (int)qkv.rows, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size,
-                                        kv.window, scale, dv, extras ? extras->sinks : nullptr, extras ? extras->gate : nullptr,
-                                        extras ? extras->gate_stride : 0, dev.stream()),
+    check_kernel(illm_attention_generic_ex(qkv.p, (int)qkv.cols, kv.k, kv.v, kv.block_table, kv.width, ctx.token_pos, ctx.token_seq, out.p,
+                                           code_of(qkv.dtype, "attention_generic"), (int)qkv.rows, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size,
+                                           kv.span(), scale, dv, extras ? extras->sinks : nullptr, extras ? extras->gate : nullptr,
+                                           extras ? extras->gate_stride : 0, extras && extras->wide_gate ? 1 : 0, extras ? extras->softcap : 0.f,
+                                           dev.stream()),
                  "attention_generic");
     return out;
 }
@@ -471,10 +473,12 @@ Mat qk_prep(Device& dev, const Mat& x, const QkPrep& p, Geometry g, const StepVi
     if (p.rot_dim && !p.cos_sin) throw KernelError("qk_prep: a rotation needs its cos/sin table");
     Mat q = new_mat(dev, x.rows, (long long)g.n_heads * g.head_dim, act_dtype);
     if (p.q_temp_every < 0) throw KernelError("qk_prep: the query temperature's period must not be negative");
-    check_kernel(illm_qk_prep_ex(x.p, code_of(x.dtype, "qk_prep"), (int)x.cols, p.q_off, has_kv ? p.k_off : -1, p.v_off, g.n_heads, g.n_kv_heads, g.head_dim, dv,
+    if (p.v_first && (!p.v_lambda || p.v_first_ld < g.n_kv_heads * dv)) throw KernelError("qk_prep: mixed values need their factor and rows of the values' width");
+    check_kernel(illm_qk_prep_mix(x.p, code_of(x.dtype, "qk_prep"), (int)x.cols, p.q_off, has_kv ? p.k_off : -1, p.v_off, g.n_heads, g.n_kv_heads, g.head_dim, dv,
                                  p.q_bias, p.k_bias, p.v_bias, p.q_norm, p.k_norm, p.eps, p.cos_sin, p.rot_dim, p.pairs ? 1 : 0, (int)p.n_pos,
                                  ctx.token_pos, ctx.token_seq, kv.block_table, kv.width, kv.page_size, q.p, store ? kv.k : nullptr,
-                                 store ? kv.v : nullptr, code_of(act_dtype, "qk_prep"), (int)x.rows, ctx.err, p.q_temp_coef, p.q_temp_every, dev.stream()),
+                                 store ? kv.v : nullptr, code_of(act_dtype, "qk_prep"), (int)x.rows, ctx.err, p.q_temp_coef, p.q_temp_every, p.v_first, p.v_first_ld, p.v_lambda,
+                                  p.v_keep, dev.stream()),
                  "qk_prep");
     return q;
 }
@@ -656,10 +660,10 @@ Mat attention_decode_ring(Device& dev, const MatOrPartials& in, const KVView& kv
         if (extras) {
             check_kernel(illm_attention_decode_ring_ex(row_ptr(in.m, t0), (int)width, kv.k, kv.v, kv.num_pages, kv.block_table, kv.width,
                                                        ctx.token_pos + t0, ctx.token_seq + t0, part_acc, part_ml, row_ptr(out, t0), (int)(t1 - t0),
-                                                       g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size, kv.window, scale, n, dev.tc_error_word(),
+                                                       g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size, kv.span(), scale, n, dev.tc_error_word(),
                                                        extras->wide_weights ? 1 : 0, extras->sinks,
                                                        extras->gate ? extras->gate + (size_t)t0 * extras->gate_stride : nullptr, extras->gate_stride,
-                                                       dev.stream()),
+                                                       extras->wide_gate ? 1 : 0, extras->softcap, dev.stream()),
                          "attention_decode_ring");
             continue;
         }
@@ -700,9 +704,10 @@ Mat attention_prefill_tc(Device& dev, const Mat& qkv, const KVView& kv, const St
     check_cache(kv, DType::BF16, g, "attention_prefill_tc");
     Mat out = new_mat(dev, qkv.rows, (long long)g.n_heads * g.head_dim, DType::BF16);
     check_kernel(illm_attention_prefill_tc_ex(qkv.p, (int)qkv.cols, (int)qkv.rows, kv.k, kv.v, kv.num_pages, kv.block_table, kv.width, ctx.cu_q,
-                                              ctx.seq_lens, out.p, ctx.B, ctx.max_q, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size, kv.window,
+                                              ctx.seq_lens, out.p, ctx.B, ctx.max_q, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size, kv.span(),
                                               scale, dev.tc_error_word(), ex && ex->wide_weights ? 1 : 0, ex ? ex->sinks : nullptr,
-                                              ex ? ex->gate : nullptr, ex ? ex->gate_stride : 0, dev.stream()),
+                                              ex ? ex->gate : nullptr, ex ? ex->gate_stride : 0, ex && ex->wide_gate ? 1 : 0, ex ? ex->softcap : 0.f,
+                                              dev.stream()),
                  "attention_prefill_tc");
     return out;
 }
@@ -730,9 +735,11 @@ Mat attention_ex(Device& dev, const Mat& q, const KVView& kv, const StepView& ct
         if (ctx.is_decode && attention_decode_ring_supported(q.dtype, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size)) {
             MatOrPartials in;
             in.m = q;
-            return attention_decode_ring(dev, in, kv, ctx, g, scale, ctx.max_seq_len, 0, nullptr, &ex);
+            // the blocks are dealt the keys of the longest range a token can see
+            const long long longest = kv.chunk > 0 ? std::min<long long>(kv.chunk, ctx.max_seq_len) : ctx.max_seq_len;
+            return attention_decode_ring(dev, in, kv, ctx, g, scale, longest, 0, nullptr, &ex);
         }
-        if (ctx.is_decode && attention_decode_supported(q.dtype, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size))
+        if (ctx.is_decode && !ex.wide_gate && ex.softcap == 0.f && kv.chunk == 0 && attention_decode_supported(q.dtype, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size))
             return attention_decode_ex(dev, q, kv, ctx, g, scale, ctx.max_seq_len, ex);
         if (!ctx.is_decode && attention_prefill_tc_supported(q.dtype, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size))
             return attention_prefill_tc(dev, q, kv, ctx, g, scale, &ex);
@@ -888,16 +895,19 @@ long long delta_rule_state_elements(int nh, int nkv, int d, int dv, int taps) {
 }
 bool delta_rule_supported(int d, int dv, int taps) { return illm_delta_rule_supported(d, dv, taps) != 0; }
 
-Mat delta_rule(Device& dev, const Mat& x, const Mat& a, const DeltaRule& p, const StepView& ctx, const StateView& st) {
+Mat delta_rule(Device& dev, const Mat& x, const Mat* a, const DeltaRule& p, const StepView& ctx, const StateView& st) {
     need(x, "the packed projection", true, DType::F32);
-    need(a, "the decay projection", true, DType::F32);
     const long long T = x.rows, C = 2LL * p.n_kv_heads * p.head_dim + (long long)p.n_heads * p.v_head_dim;
-    if (a.rows != T || a.cols != (long long)p.n_heads * p.head_dim) throw KernelError("delta_rule: the decay projection must be [T, heads * head_dim]");
+    const long long decays = p.head_decay ? p.n_heads : (long long)p.n_heads * p.head_dim;
+    if (p.head_decay ? (a != nullptr || p.a_off < 0 || p.a_off + p.n_heads > x.cols) : (!a || a->dtype != DType::F32 || a->rows != T || a->cols != decays))
+        throw KernelError("delta_rule: the decay projection must be float32 [T, heads * head_dim], or `heads` columns of the packed projection");
     if (!st.state || st.dtype != DType::F32 || st.elements != delta_rule_state_elements(p.n_heads, p.n_kv_heads, p.head_dim, p.v_head_dim, p.taps))
         throw KernelError("delta_rule: the state entry does not have this layer's size");
-    Mat qkv = new_mat_exact(dev, T, C, DType::F32), g = new_mat_exact(dev, T, a.cols, DType::F32), beta = new_mat_exact(dev, T, p.n_heads, DType::F32);
+    Mat qkv = new_mat_exact(dev, T, C, DType::F32), g = new_mat_exact(dev, T, decays, DType::F32), beta = new_mat_exact(dev, T, p.n_heads, DType::F32);
     Mat out = new_mat_exact(dev, T, (long long)p.n_heads * p.v_head_dim, DType::F32);
-    check_kernel(illm_delta_rule((const float*)x.p, (int)T, (int)x.cols, p.q_off, p.k_off, p.v_off, p.b_off, (const float*)a.p, p.n_heads,
+    check_kernel(illm_delta_rule((const float*)x.p, (int)T, (int)x.cols, p.q_off, p.k_off, p.v_off, p.b_off,
+                                 p.head_decay ? (const float*)x.p + p.a_off : (const float*)a->p, p.head_decay ? (int)x.cols : (int)decays,
+                                 p.head_decay ? 1 : 0, p.n_heads,
                                  p.n_kv_heads, p.head_dim, p.v_head_dim, p.taps, p.conv_q, p.conv_k, p.conv_v, p.a_log, p.dt_bias, p.q_scale,
                                  (float*)st.state, st.elements, st.slots, ctx.cu_q, ctx.token_pos, ctx.token_seq, ctx.seq_lens, (float*)qkv.p,
                                  (float*)g.p, (float*)beta.p, (float*)out.p, ctx.B, dev.stream()),
@@ -906,17 +916,20 @@ Mat delta_rule(Device& dev, const Mat& x, const Mat& a, const DeltaRule& p, cons
 }
 
 Mat latent_prep(Device& dev, const Mat& x, int q_rank, int kv_rank, const float* w_q, const float* w_kv, float eps, const StepView& ctx,
-                const KVView& kv, DType act_dtype) {
+                const KVView& kv, DType act_dtype, const LatentRope* rot) {
     need(x, "the packed latent projection", true, DType::F32);
-    if (x.cols < q_rank + kv_rank) throw KernelError("latent_prep: the projection is narrower than the two latents");
+    const int dr = rot ? rot->rot_head_dim : 0;
+    if (x.cols < q_rank + kv_rank + dr) throw KernelError("latent_prep: the projection is narrower than the two latents");
+    if (rot && rot->rot_dim && !rot->cos_sin) throw KernelError("latent_prep: a rotation needs its cos/sin table");
     if (kv.writes) {
-        if (!kv.k || kv.dtype != act_dtype || kv.n_kv_heads != 1 || kv.head_dim != kv_rank)
+        if (!kv.k || kv.dtype != act_dtype || kv.n_kv_heads != 1 || kv.head_dim != kv_rank + dr)
             throw KernelError("latent_prep: the cache entry must hold one head of kv_rank channels in the activation dtype");
     }
     Mat cq = new_mat(dev, x.rows, q_rank, act_dtype);
     check_kernel(illm_latent_prep((const float*)x.p, (int)x.cols, q_rank, kv_rank, w_q, w_kv, eps, ctx.token_pos, ctx.token_seq, kv.block_table,
                                   kv.width, kv.page_size, cq.p, kv.writes ? kv.k : nullptr, code_of(act_dtype, "latent_prep"), (int)x.rows,
-                                  ctx.err, dev.stream()),
+                                  ctx.err, dr, rot ? rot->cos_sin : nullptr, rot ? rot->rot_dim : 0, rot && rot->pairs ? 1 : 0,
+                                  rot ? (int)rot->n_pos : 0, dev.stream()),
                  "latent_prep");
     return cq;
 }
@@ -980,11 +993,12 @@ Mat head_linear_pieces(Device& dev, const Mat& x, const Mat& w, int heads, bool 
 Mat latent_rope_prep(Device& dev, const Mat& x, const LatentRope& p, const StepView& ctx, const KVView& kv, DType act_dtype, Mat* qa) {
     need(x, "the packed latent projection", true, DType::F32);
     const long long row = (long long)p.kv_rank + p.rot_head_dim;
-    if (p.n_heads <= 0 || p.head_dim <= 0 || p.rot_head_dim < 0 || p.kv_rank <= 0 || p.q_off < 0 || p.c_off < 0 ||
-        p.q_off + (long long)p.n_heads * (p.head_dim + p.rot_head_dim) > x.cols || p.c_off + row > x.cols)
+    const bool stores = kv.writes && p.c_off >= 0;
+    if (p.n_heads <= 0 || p.head_dim <= 0 || p.rot_head_dim < 0 || p.kv_rank <= 0 || p.q_off < 0 ||
+        p.q_off + (long long)p.n_heads * (p.head_dim + p.rot_head_dim) > x.cols || (p.c_off >= 0 && p.c_off + row > x.cols))
         throw KernelError("latent_rope_prep: the projection is narrower than the queries and the latent");
     if (p.rot_dim && !p.cos_sin) throw KernelError("latent_rope_prep: a rotation needs its cos/sin table");
-    if (kv.writes && (!kv.k || kv.dtype != act_dtype || kv.n_kv_heads != 1 || kv.head_dim != row))
+    if (stores && (!kv.k || kv.dtype != act_dtype || kv.n_kv_heads != 1 || kv.head_dim != row))
         throw KernelError("latent_rope_prep: the cache entry must hold one head of kv_rank + rotated channels in the activation dtype");
     if (!qa) throw KernelError("latent_rope_prep: nowhere to put the absorbed queries");
     *qa = new_mat(dev, x.rows, p.n_heads * row, act_dtype);
@@ -992,7 +1006,7 @@ Mat latent_rope_prep(Device& dev, const Mat& x, const LatentRope& p, const StepV
     Mat qn = new_mat(dev, x.rows, (long long)p.n_heads * p.head_dim, q_f32 ? DType::F32 : act_dtype);
     check_kernel(illm_latent_rope_prep((const float*)x.p, (int)x.cols, p.q_off, p.n_heads, p.head_dim, p.rot_head_dim, p.c_off, p.kv_rank, p.w_kv, p.eps,
                                        p.cos_sin, p.rot_dim, p.pairs ? 1 : 0, (int)p.n_pos, ctx.token_pos, ctx.token_seq, kv.block_table, kv.width,
-                                       kv.page_size, qn.p, q_f32 ? 1 : 0, qa->p, kv.writes ? kv.k : nullptr, code_of(act_dtype, "latent_rope_prep"),
+                                       kv.page_size, qn.p, q_f32 ? 1 : 0, qa->p, stores ? kv.k : nullptr, code_of(act_dtype, "latent_rope_prep"),
                                        (int)x.rows, ctx.err, dev.stream()),
                  "latent_rope_prep");
     return qn;
@@ -1099,6 +1113,11 @@ void convert(Device& dev, const void* src, DType src_dtype, void* dst, DType dst
     if (rc == 10001)
         throw KernelError(std::string("a tensor stored as ") + dtype_word(src_dtype) + " cannot be brought to " + dtype_word(dst_dtype));
     check_kernel(rc, "convert");
+}
+
+void soft_cap(Device& dev, const Mat& x, float cap) {
+    need(x, "x", true, DType::F32);
+    check_kernel(illm_soft_cap((float*)x.p, x.rows * x.cols, cap, dev.stream()), "soft_cap");
 }
 
 Mat cast(Device& dev, const Mat& x, DType dtype) {

@@ -122,11 +122,12 @@ Mat embedding(Device& dev, const int* ids, long long T, const Mat& table, int* e
 // table[id] * scale plus, with inv_freq (float32 [ceil(H / 2)] on the device), the sinusoid position vector
 // (sin(p f_i), cos(p f_i)) in entries (2i, 2i + 1)
 Mat embedding_scaled(Device& dev, const StepView& ctx, const Mat& table, float scale, const float* inv_freq);
-// Layer norm (weight, no bias) around the float32 stream: resid += ln(delta) * post_w (delta, post_w nullptr: nothing
-// is added), then ln(resid) * w in `out_dtype` (w nullptr: the addition alone, an empty matrix comes back).  rows
+// Layer norm (weight, no bias) or, with center = false, RMS norm around the float32 stream: resid += post_scale *
+// n(delta) * post_w (delta, post_w nullptr: nothing is added; post_scale other than 1 for the RMS norm only), then
+// n(resid) * w in `out_dtype` (w nullptr: the addition alone, an empty matrix comes back).  rows
 // (int32, device) gathers: only those rows are made and resid is left as it is.
-Mat layernorm_sandwich(Device& dev, const Mat& resid, const Mat* delta_f32, const Mat* post_w_f32, const Mat* w_f32, float eps, DType out_dtype,
-                       const int* rows, long long n_rows);
+Mat norm_sandwich(Device& dev, const Mat& resid, const Mat* delta_f32, const Mat* post_w_f32, const Mat* w_f32, float eps, DType out_dtype,
+                  const int* rows, long long n_rows, bool center = true, float post_scale = 1.f);
 // y = act(conv(x) + bias) (+ x): a causal convolution over time per channel of columns [x_off, x_off + C) of the
 // float32 rows x, `taps` taps w [C, taps] (float32, the last the token's own), the rows before the step from the
 // sequence's state ([taps - 1, C] at state_off of the slot's elements), which is renewed if `update`.  Written to
@@ -149,13 +150,14 @@ Mat materialize(Device& dev, const Partials& p, DType dtype);
 Mat swiglu(Device& dev, const MatOrPartials& gu);
 Mat gemm_f32(Device& dev, const Mat& x, const Mat& w);
 MatOrPartials gemm_bf16_tc(Device& dev, const Mat& x, const Mat& w, DType out_dtype, int splits /* 0: by policy */, bool defer_reduce);
-Mat gemm_bf16_tc2(Device& dev, const Mat& x, const Mat& w, DType out_dtype, bool gated, int act = 1 /* kActSilu */);
+Mat gemm_bf16_tc2(Device& dev, const Mat& x, const Mat& w, DType out_dtype, bool gated, int act = 1 /* kActSilu */, float act_limit = 0.f);
 // x [M, K] . w [N, K]^T.  defer_reduce allows the result to come back as unreduced slices (only a
 // caller that hands it to add_rmsnorm, the rotation or the fused decode attention asks).
 MatOrPartials linear(Device& dev, GemmBackend backend, const Mat& x, const Mat& w, DType out_dtype, bool defer_reduce);
 // act(gate) * up of x . w^T, where w's rows 2i, 2i + 1 are the gate and the up row of output i (act: a GateAct, silu
 // by default); the product kernels of the package apply it in their epilogues.
-Mat linear_gated(Device& dev, GemmBackend backend, const Mat& x, const Mat& w, int act = 1 /* kActSilu */);
+// act_limit: the limit of kActSwishClamped.
+Mat linear_gated(Device& dev, GemmBackend backend, const Mat& x, const Mat& w, int act = 1 /* kActSilu */, float act_limit = 0.f);
 
 struct Geometry { int n_heads, n_kv_heads, head_dim; };
 // Rotate Q (and K) of the packed projection and store K, V in the cache pages.  cos_sin: float32
@@ -164,13 +166,16 @@ struct Geometry { int n_heads, n_kv_heads, head_dim; };
 // as unreduced slices, a new one (the slices are added up on the way).
 Mat rope_kv_write(Device& dev, const MatOrPartials& qkv, const float* cos_sin, int rot_dim, long long n_pos, const StepView& ctx,
                   const KVView& kv, Geometry g);
-// Options of the generic attention kernel beyond the plain softmax attention: a per-head sink in the
-// softmax denominator (float32 [n_heads]), and a per-head output gate, sigmoid(gate[t * gate_stride + h])
-// (float32).  The value head size is the cache entry's (KVView::v_head_dim).
+// Options of the attention kernels beyond the plain softmax attention: a per-head sink in the softmax denominator
+// (float32 [n_heads]; zeros add one to it), an output gate, sigmoid(gate[t * gate_stride + h]) for whole heads or, with
+// wide_gate, sigmoid(gate[t * gate_stride + h * dv + c]) element by element (float32), and a soft cap on the scaled
+// scores, softcap * tanh(score / softcap) (0: none).  The value head size is the cache entry's (KVView::v_head_dim).
 struct AttentionExtras {
     const float* sinks = nullptr;
     const float* gate = nullptr;
     int gate_stride = 0;
+    bool wide_gate = false;
+    float softcap = 0.f;
     // the tensor-core prompt kernel keeps sixteen bits of the softmax weights' mantissa (two bfloat16
     // terms) instead of eight; the other kernels have float32 weights anyway
     bool wide_weights = false;
@@ -188,8 +193,8 @@ Mat attention_prefill_tc(Device& dev, const Mat& qkv, const KVView& kv, const St
 // The split-key decode kernel on CUDA cores (float32 scores and weights) with sinks and gates in its merge.
 Mat attention_decode_ex(Device& dev, const Mat& qkv, const KVView& kv, const StepView& ctx, Geometry g, float scale, long long max_len,
                         const AttentionExtras& extras);
-// Attention with extras: the tensor-core prompt kernel and the split-key decode kernel where the
-// sizes allow (bfloat16, keys and values of one size, 64 or 128), the general kernel otherwise.
+// Attention with extras: the tensor-core prompt kernel and the ring or split-key decode kernel where the sizes allow
+// (bfloat16, keys and values of one size, 64 or 128), the general kernel otherwise.  Windows and chunks (KVView::span).
 Mat attention_ex(Device& dev, const Mat& q, const KVView& kv, const StepView& ctx, Geometry g, float scale, const AttentionExtras& extras);
 // Attention whose heads' scores are mixed before the softmax (mix float32 [n_heads, n_heads] or nullptr), with a
 // logarithmic distance penalty r1_h ln(1 + r2_h (i - j)) (r1, r2 float32 [n_heads] or nullptr), over a keys-only
@@ -241,6 +246,12 @@ struct QkPrep {
     // (whole-numbered division), behind the bias; q_temp_every 0: none
     float q_temp_coef = 0.f;
     int q_temp_every = 0;
+    // values mixed with another layer's values of the same tokens: v <- (1 - *v_lambda) v + *v_lambda v_first, behind the
+    // bias (v_first float32, rows v_first_ld apart; v_lambda one float32; both on the device); v_keep (float32 [T, nkv dv]):
+    // the layer's own values, unmixed, are stored there for later layers
+    const float *v_first = nullptr, *v_lambda = nullptr;
+    int v_first_ld = 0;
+    float* v_keep = nullptr;
 };
 Mat qk_prep(Device& dev, const Mat& x, const QkPrep& p, Geometry g, const StepView& ctx, const KVView& kv, DType act_dtype);
 
@@ -310,7 +321,7 @@ Mat group_norm_gate(Device& dev, const Mat& o_f32, int group, const float* w, fl
 // ---- pieces of further mixers, feed-forwards and embeddings
 
 // Activations of the gated feed-forward: act(gate) * up.
-// kActSwishClamped (routed experts only): g = min(gate, limit), u = clamp(up, -limit, limit); g sigmoid(1.702 g) (u + 1)
+// kActSwishClamped: g = min(gate, limit), u = clamp(up, -limit, limit); g sigmoid(1.702 g) (u + 1)
 enum GateAct { kActSilu = 1, kActRelu = 2, kActGeluTanh = 3, kActSwishClamped = 4 };
 int gate_act_from_name(const std::string& name);        // ConfigError-free: -1 for an unknown name
 // resid += d1 (+ d2), all float32 [T, H], and the RMS norm of the new rows times w (float32 [H]) in `out_dtype`: one kernel
@@ -331,25 +342,30 @@ Mat join_rows(Device& dev, const Mat& a_f32, const Mat& b_f32, DType dtype);
 struct BigramHash { long long buckets = 0, mul_prev = 0, mul_cur = 0; };
 Mat bigram_embedding(Device& dev, const StepView& ctx, const Mat& table, const Mat& bigram, const BigramHash& hash, const StateView& last_token);
 
-// The gated delta rule with a decay per head and key channel (csrc/delta_state.cu).  x_f32: the packed float32
-// projection with q, k, v and beta's logits at the given columns; a_f32 [T, heads * head_dim]: the decay
-// projection.  The state entry holds S and the convolution's rows (delta_rule_state_elements).  Returns float32
+// The gated delta rule with a decay per head and key channel, or (head_decay) per head (csrc/delta_state.cu).  x_f32: the
+// packed float32 projection with q, k, v and beta's logits at the given columns; the decay projection is a_f32 [T, heads *
+// head_dim] or, with head_decay, the `heads` columns of x_f32 at a_off (a_f32 nullptr).  The state entry holds S and the convolution's rows (delta_rule_state_elements).  Returns float32
 // [T, heads * v_head_dim].
 struct DeltaRule {
     int q_off = 0, k_off = 0, v_off = 0, b_off = 0;
     int n_heads = 0, n_kv_heads = 0, head_dim = 0, v_head_dim = 0, taps = 1;
+    bool head_decay = false;
+    int a_off = 0;                                                           // head_decay: the decay projection's columns
     const float *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr;     // float32 [channels, taps]
-    const float *a_log = nullptr, *dt_bias = nullptr;                        // float32 [heads], [heads * head_dim]
+    const float *a_log = nullptr, *dt_bias = nullptr;                        // float32 [heads], [heads * head_dim] or [heads]
     float q_scale = 1.f;
 };
 long long delta_rule_state_elements(int n_heads, int n_kv_heads, int head_dim, int v_head_dim, int taps);
 bool delta_rule_supported(int head_dim, int v_head_dim, int taps);
-Mat delta_rule(Device& dev, const Mat& x_f32, const Mat& a_f32, const DeltaRule& p, const StepView& ctx, const StateView& st);
+Mat delta_rule(Device& dev, const Mat& x_f32, const Mat* a_f32, const DeltaRule& p, const StepView& ctx, const StateView& st);
 
 // Attention through latents (csrc/latent_attention.cu): the two norms and the cache write; returns the normed
 // query latent [T, q_rank] in `act_dtype`.  kv: a keys-only entry of one head of kv_rank channels.
+// With `rot`, the projection has rot->rot_head_dim more columns behind the latent's: one key part shared by all heads, rotated
+// by the position and cached behind the latent (a cache row of kv_rank + rot_head_dim channels).
+struct LatentRope;
 Mat latent_prep(Device& dev, const Mat& x_f32, int q_rank, int kv_rank, const float* w_q, const float* w_kv, float eps, const StepView& ctx,
-                const KVView& kv, DType act_dtype);
+                const KVView& kv, DType act_dtype, const LatentRope* rot = nullptr);
 // Attention of `heads` query heads over one shared key/value head of ANY width (a keys-only cache entry), float32 math:
 // for widths the framework's attention kernels do not take.  q [T, heads * width] in the cache's dtype.
 // gate (float32 [T, gate_stride] or nullptr): head h of token t is multiplied by sigmoid(gate[t * gate_stride + h])
@@ -369,7 +385,8 @@ Mat head_linear_pieces(Device& dev, const Mat& x, const Mat& w, int heads, bool 
 // (latent_rope_prep_kernel, csrc/latent_attention.cu).  x_f32: the packed projection with the queries (heads x (d + dr)) at
 // q_off and [latent (kv_rank), raw shared key part (dr)] at c_off.  Writes the cache row [normed latent, rotated key part],
 // returns q_nope [T, heads * d] (float32 for single tokens, else the activation dtype) and fills the last dr channels per
-// head of qa [T, heads * (kv_rank + dr)] (activation dtype) with the rotated query parts.
+// head of qa [T, heads * (kv_rank + dr)] (activation dtype) with the rotated query parts.  c_off < 0: the queries alone (the latent and the key part
+// were cached by latent_prep).
 struct LatentRope {
     int q_off = 0, c_off = 0, n_heads = 0, head_dim = 0, rot_head_dim = 0, kv_rank = 0;
     const float* w_kv = nullptr;
@@ -410,6 +427,8 @@ void fill_random(Device& dev, void* out, DType dtype, long long n, unsigned long
 void convert(Device& dev, const void* src, DType src_dtype, void* dst, DType dst_dtype, long long n);
 // x in another dtype, as a new activation (x itself if it has that dtype already)
 Mat cast(Device& dev, const Mat& x, DType dtype);
+// x = cap * tanh(x / cap), in place (x float32)
+void soft_cap(Device& dev, const Mat& x_f32, float cap);
 
 long long launch_count();               // kernels of this package launched so far (graph replays counted by the engine)
 void count_replayed_launches(long long n);

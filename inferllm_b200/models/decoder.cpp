@@ -84,6 +84,7 @@ std::map<int, CacheRequest> DecoderModel::cache_requests() const {
 
 Mat DecoderModel::forward(const StepContext& ctx, const SequenceCache& cache, const std::vector<const int*>& tables_dev) {
     Device& dev = *rt->dev;
+    ctx.kept.clear();
     ResidualStream stream;
     if (cache.kind_of(kEmbeddingCacheEntry) == SequenceCache::State) {
         CacheView ev;

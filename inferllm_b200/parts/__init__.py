@@ -320,7 +320,7 @@ class _Proxy:
         if not c:
             return None
         if c["kind"] == "kv":
-            return PagedKV(c["n_kv_heads"], c["head_dim"], c["window"])
+            return PagedKV(c["n_kv_heads"], c["head_dim"], c["window"], bool(c.get("keys_only")), c.get("chunk"))
         return FixedState(tuple(c["shape"]), c["dtype"])
 
     def load(self, tensors: Dict[str, object]) -> None:

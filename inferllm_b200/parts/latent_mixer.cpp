@@ -10,14 +10,14 @@
 // key and value at once: a keys-only cache entry) and `heads` query heads, and the per-head maps U_k,h^T and U_v,h run
 // before and after them (ops::head_linear).  A step's keys and values are never expanded per head.
 //
-// Options: `q_rank` 0 (the queries come straight from the mixer's input, q = W_q h, no query latent);
+// Options, in any combination: `q_rank` 0 (the queries come straight from the mixer's input, q = W_q h, no query latent);
 // `rot_head_dim` dr > 0 with a `position` part (a table rotation): every query head has dr more channels behind its d, the
 // key/value down-projection dr more rows behind the latent's (not normed), both are rotated by the position, and
 //     score = (q_h[0:d] . k_h + rot(q_h[d:d+dr]) . rot(kr)) * scale
 // with the ONE rotated key part kr shared by all heads.  The cache row is then [c, rot(kr)] (kv_rank + dr channels), the
 // absorbed query [U_k,h^T q_h[0:d], rot(q_h[d:])], and the attention kernels' values are the whole row, of which U_v,h
-// reads the first kv_rank channels;  `out_gate` = "head_sigmoid" (a projection of the mixer's input to one number per
-// head, whose sigmoid multiplies the head's output).  These three run on a path of their own (forward_direct).
+// reads the first kv_rank channels (with q_rank > 0 the query up-projection has heads x (d + dr) rows, head by head);  `out_gate` = "head_sigmoid" (a projection of the mixer's input to one number per
+// head, whose sigmoid multiplies the head's output).  The second and third, and q_rank 0, run on a path of their own (forward_rotated).
 #include <cmath>
 
 #include "parts/parts.h"
@@ -50,7 +50,6 @@ struct LatentAttention : Mixer {
         if (og != "none" && og != "head_sigmoid") throw ConfigError("latent_attention: out_gate '" + og + "' is not supported (none, head_sigmoid)");
         has_gate = og == "head_sigmoid";
         if (rot_head_dim < 0) throw ConfigError("latent_attention: rot_head_dim must not be negative");
-        if (q_rank > 0 && (rot_head_dim > 0 || has_gate)) throw ConfigError("latent_attention: rotated channels and the head gate need q_rank 0 (queries straight from the input)");
         if (rot_head_dim > 0) {
             position = build_position(s.get_part("position"), rt);
             if (rt) position->prepare();
@@ -65,6 +64,7 @@ struct LatentAttention : Mixer {
             throw ConfigError("latent_attention: a latent of " + std::to_string(kv_rank + rot_head_dim) + " channels is beyond the kernels (up to 1024)");
     }
     bool direct() const { return q_rank == 0; }
+    bool plain() const { return q_rank > 0 && rot_head_dim == 0 && !has_gate; }
     long long row() const { return (long long)kv_rank + rot_head_dim; }       // channels of a cache row
     bool graph_safe() const override { return true; }
     bool pad_safe() const override { return false; }
@@ -80,12 +80,16 @@ struct LatentAttention : Mixer {
             d.push_back({nm("o"), TensorDecl{{hidden, v}}});
             return d;
         }
-        return {{nm("q_down"), TensorDecl{{(long long)q_rank, hidden}}}, {nm("q_norm"), TensorDecl{{(long long)q_rank}, "norm"}},
-                {nm("q_up"), TensorDecl{{q, (long long)q_rank}}}, {nm("kv_down"), TensorDecl{{(long long)kv_rank, hidden}}},
-                {nm("kv_norm"), TensorDecl{{(long long)kv_rank}, "norm"}}, {nm("k_up"), TensorDecl{{q, (long long)kv_rank}}},
-                {nm("v_up"), TensorDecl{{v, (long long)kv_rank}}}, {nm("o"), TensorDecl{{hidden, v}}}};
+        TensorDecls d = {{nm("q_down"), TensorDecl{{(long long)q_rank, hidden}}}, {nm("q_norm"), TensorDecl{{(long long)q_rank}, "norm"}},
+                         {nm("q_up"), TensorDecl{{dq_rows(), (long long)q_rank}}}, {nm("kv_down"), TensorDecl{{row(), hidden}}},
+                         {nm("kv_norm"), TensorDecl{{(long long)kv_rank}, "norm"}}, {nm("k_up"), TensorDecl{{q, (long long)kv_rank}}},
+                         {nm("v_up"), TensorDecl{{v, (long long)kv_rank}}}};
+        if (has_gate) d.push_back({nm("gate"), TensorDecl{{(long long)n_heads, hidden}}});
+        d.push_back({nm("o"), TensorDecl{{hidden, v}}});
+        return d;
     }
-    // rows of the packed matrix of the direct path: the queries, then latent and raw key part, then the gate
+    // rows of the packed matrix: the queries (direct) or their latent, then latent and raw key part, then the gate
+    long long q_part() const { return direct() ? dq_rows() : q_rank; }
     long long dq_rows() const { return (long long)n_heads * (head_dim + rot_head_dim); }
     void load(TensorSource& src) override {
         const size_t es = dtype_size(rt->dtype);
@@ -102,11 +106,12 @@ struct LatentAttention : Mixer {
             n_kv = fetch_owned(rt, src, names.at("kv_norm"), DType::F32, "a latent norm's weight");
             return;
         }
-        const long long all = (long long)q_rank + kv_rank;
+        const long long all = q_part() + row() + (has_gate ? n_heads : 0);
         w_buf = DeviceBuffer(rt->dev, (size_t)all * hidden * es, "the packed latent projections");
         w_down = Mat{w_buf.get(), all, hidden, rt->dtype, all};
         src.fetch_into(names.at("q_down"), w_down.p, rt->dtype);
         src.fetch_into(names.at("kv_down"), (char*)w_down.p + (size_t)q_rank * hidden * es, rt->dtype);
+        if (has_gate) src.fetch_into(names.at("gate"), (char*)w_down.p + (size_t)(q_part() + row()) * hidden * es, rt->dtype);
         w_uq = fetch_owned(rt, src, names.at("q_up"), rt->dtype, "the query up-projection");
         w_uk = fetch_owned(rt, src, names.at("k_up"), rt->dtype, "the key up-projection");
         w_uv = fetch_owned(rt, src, names.at("v_up"), rt->dtype, "the value up-projection");
@@ -121,7 +126,7 @@ struct LatentAttention : Mixer {
         KVView kv = cache.kv;
         kv.writes = writes;
         if (kv.n_kv_heads != 1 || kv.head_dim != row()) throw EngineError("latent_attention: the cache entry does not hold this layer's latent");
-        if (direct()) return forward_direct(h, ctx, kv, may_defer);
+        if (!plain()) return forward_rotated(h, ctx, kv, may_defer);
         Mat x = ops::linear(dev, rt->gemm, h, w_down, DType::F32, false).m;
         Mat cq = ops::latent_prep(dev, x, q_rank, kv_rank, (const float*)n_q.m.p, (const float*)n_kv.m.p, norm_eps, ctx, kv, rt->dtype);
         // a prompt's queries are rounded to the activation dtype for the library's batched product; single tokens stay float32
@@ -137,13 +142,13 @@ struct LatentAttention : Mixer {
         return ops::linear(dev, rt->gemm, ov, w_o.m, out_f32 ? DType::F32 : rt->dtype, may_defer);
     }
 
-    // queries straight from the input, optionally rotated channels beside the latent and a gate per head
-    MatOrPartials forward_direct(const Mat& h, const StepContext& ctx, const KVView& kv, bool may_defer) {
+    // queries straight from the input or through their latent, optionally rotated channels beside the latent and a gate per head
+    MatOrPartials forward_rotated(const Mat& h, const StepContext& ctx, const KVView& kv, bool may_defer) {
         Device& dev = *rt->dev;
         Mat x = ops::linear(dev, rt->gemm, h, w_down, DType::F32, false).m;
         ops::LatentRope p;
         p.q_off = 0;
-        p.c_off = (int)dq_rows();
+        p.c_off = direct() ? (int)dq_rows() : -1;
         p.n_heads = n_heads;
         p.head_dim = head_dim;
         p.rot_head_dim = rot_head_dim;
@@ -162,8 +167,14 @@ struct LatentAttention : Mixer {
             p.pairs = pairs;
             p.n_pos = n_pos;
         }
+        Mat qx = x;
+        if (!direct()) {
+            // both latents' norms, the rotated key part and the cache row first; then the queries, in float32 until they are split
+            Mat cq = ops::latent_prep(dev, x, q_rank, kv_rank, (const float*)n_q.m.p, (const float*)n_kv.m.p, norm_eps, ctx, kv, rt->dtype, &p);
+            qx = ops::linear(dev, rt->gemm, cq, w_uq.m, DType::F32, false).m;
+        }
         Mat qa;
-        Mat qn = ops::latent_rope_prep(dev, x, p, ctx, kv, rt->dtype, &qa);
+        Mat qn = ops::latent_rope_prep(dev, qx, p, ctx, kv, rt->dtype, &qa);
         ops::HeadPieces into;
         into.into = &qa;
         into.y_head_stride = row();
@@ -172,7 +183,7 @@ struct LatentAttention : Mixer {
         ops::AttentionExtras ex;
         ex.wide_weights = true;       // the softmax weights are not to be rounded to eight bits
         if (has_gate) {
-            ex.gate = (const float*)x.p + (dq_rows() + row());
+            ex.gate = (const float*)x.p + (q_part() + row());
             ex.gate_stride = (int)x.cols;
         }
         // a row whose width the framework's attention kernels do not take (not a multiple of 8, beyond 256) has a plain kernel

@@ -176,19 +176,21 @@ namespace {
 // reference fixes eps in code (1e-6 in the layers, src/graph/llama_like.cpp:77-78; 1e-5 in the head,
 // src/core/graph.h:160-163); here it is a parameter of the part.
 //
-// Three parameters beyond the reference's norm: `weight_offset` (a weight stored as w - offset, e.g.
+// Four parameters beyond the reference's norm: `post_scale` (the norm can also stand behind a sublayer, on its output's way
+// into the stream, x + post_scale * norm(f(..)), see add_normed_pending: the sandwich block; where such a norm and the next
+// sublayer's input norm follow one another both run in one kernel), `weight_offset` (a weight stored as w - offset, e.g.
 // around zero for offset 1; the offset is added once, in float32, when the weight is loaded),
 // `residual_scale` (the factor on the stream in the norm-after-the-sum arrangement, see
 // forward_into_stream) and `tensor` (the weight's name below the part's prefix, "weight" if not given).
 struct RMSNorm : Norm {
     long long size;
-    float eps, weight_offset, residual_scale;
+    float eps, weight_offset, residual_scale, post_scale;
     std::string tensor;
     bool optional, absent = false;
     OwnedMat weight;
     RMSNorm(const PartSpec& s, Runtime* rt)
             : Norm(s, rt), size(s.get_int("size")), eps((float)s.get_double("eps")), weight_offset((float)s.get_double("weight_offset", 0.0)),
-              residual_scale((float)s.get_double("residual_scale", 1.0)), tensor(s.get_string("tensor", "weight")),
+              residual_scale((float)s.get_double("residual_scale", 1.0)), post_scale((float)s.get_double("post_scale", 1.0)), tensor(s.get_string("tensor", "weight")),
               optional(s.get_bool("optional", false)) {
         if (size <= 0 || !(eps > 0)) throw ConfigError("rmsnorm: size and eps must be positive");
     }
@@ -225,7 +227,25 @@ struct RMSNorm : Norm {
         stream.has_pending = false;
         return ops::scale_add_rmsnorm(*rt->dev, stream.x, d, weight.m, residual_scale, eps, rt->dtype);
     }
+    void add_normed_pending(ResidualStream& stream) override {
+        Mat y = stream.pending.is_partials() ? ops::materialize(*rt->dev, stream.pending.part, DType::F32) : ops::cast(*rt->dev, stream.pending.m, DType::F32);
+        ops::norm_sandwich(*rt->dev, stream.x, &y, &weight.m, nullptr, eps, DType::F32, nullptr, 0, false, post_scale);
+        stream.has_pending = false;
+    }
     Mat forward(ResidualStream& stream, const int* rows, long long n_rows) override {
+        // an addition that passes an RMS norm of its own on its way into the stream: both norms in one kernel
+        if (RMSNorm* post = stream.has_pending && !stream.has_pending2 ? dynamic_cast<RMSNorm*>(stream.pending_post) : nullptr) {
+            if (!stream.pending.is_partials() && stream.pending.m.dtype == DType::F32 && post->eps == eps && post->weight.m.dtype == DType::F32 &&
+                weight.m.dtype == DType::F32) {
+                Mat y = ops::norm_sandwich(*rt->dev, stream.x, &stream.pending.m, &post->weight.m, &weight.m, eps, rt->dtype, rows, n_rows, false,
+                                           post->post_scale);
+                if (rows == nullptr) {
+                    stream.has_pending = false;
+                    stream.pending_post = nullptr;
+                }
+                return y;
+            }
+        }
         // an addition that passes a layer scale on its way into the stream: x + factors * pending and the norm in one kernel
         if (stream.has_pending && stream.pending_post) {
             const Mat* ls = stream.pending_post->channel_scale();
@@ -387,6 +407,14 @@ struct NoPosition : PositionEncoding {
 // number for the layer, made once at load; then o / sqrt(mean(o^2) + norm_eps) over the head's values, times 1 - diff;
 // ops::attention_diff), `q_temperature` {coef, every} (the queries of position p are multiplied by
 // 1 + coef ln(floor((p + 1) / every) + 1), behind the bias) and `o_bias` (a bias on the output projection).
+//
+// A fourth: `chunk` c (instead of a window: a query sees the earlier positions of its own chunk of c, counted from the
+// sequence's start), `softcap` (the scaled scores s become softcap * tanh(s / softcap)), `unit_sink` (one is added to the
+// softmax denominator: a sink whose score is 0), `out_gate` = "sigmoid" also without values = keys, and `value_mix`: "first"
+// (the layer keeps its values for later layers of the step) or "mix" (v <- (1 - lambda) v + lambda v_first with the kept
+// values of the same tokens and lambda one number, tensor "v_mix"; the mixed values are what is cached).  Both declare
+// the tensor.
+constexpr const char* kFirstValues = "attention.first_values";      // StepContext::kept: see value_mix
 struct Attention : Mixer {
     long long hidden;
     int n_heads, n_kv_heads, head_dim, v_head_dim, window;
@@ -397,11 +425,14 @@ struct Attention : Mixer {
     bool o_bias = false;
     float diff = 0.f, lambda = 0.f, q_temp_coef = 0.f;
     int q_temp_every = 0;
+    int chunk = 0;
+    float softcap = 0.f;
+    bool unit_sink = false, keeps_values = false, mixes_values = false;
     std::map<std::string, std::string> names;
     std::unique_ptr<PositionEncoding> position;
     DeviceBuffer qkv_buf, o_buf;
     Mat w_qkv, w_o;
-    OwnedMat b_q, b_k, b_v, b_o, n_q, n_k, sinks, dist_r1, dist_r2, mix;
+    OwnedMat b_q, b_k, b_v, b_o, n_q, n_k, sinks, dist_r1, dist_r2, mix, v_mix;
     Attention(const PartSpec& s, Runtime* rt)
             : Mixer(s, rt), hidden(s.get_int("hidden_size")), n_heads((int)s.get_int("n_heads")), n_kv_heads((int)s.get_int("n_kv_heads")),
               head_dim((int)s.get_int("head_dim")), v_head_dim((int)s.get_int("v_head_dim", s.get_int("head_dim"))),
@@ -421,8 +452,8 @@ struct Attention : Mixer {
         const std::string vs = s.get_string("values", "own"), db = s.get_string("distance_bias", "none");
         if (vs != "own" && vs != "keys") throw ConfigError("attention: values '" + vs + "' is not supported (own, keys)");
         if (db != "none" && db != "log1p") throw ConfigError("attention: distance_bias '" + db + "' is not supported (none, log1p)");
-        if ((log_distance || head_mix || wide_gate) && !values_are_keys)
-            throw ConfigError("attention: distance_bias, head_mix and the element-wise gate run on the kernel for values = keys only");
+        if ((log_distance || head_mix) && !values_are_keys)
+            throw ConfigError("attention: distance_bias and head_mix run on the kernel for values = keys only");
         if (values_are_keys && (v_head_dim != head_dim || !own_kv || qkv_bias || proj_norm || has_sink || has_gate))
             throw ConfigError("attention: values = keys needs key and value heads of one size and takes no biases, projection norms, sinks or head gates");
         maps = (int)s.get_int("score_maps", 1);
@@ -441,13 +472,26 @@ struct Attention : Mixer {
             q_temp_coef = (float)qt.at("coef").as_double();
             q_temp_every = (int)qt.at("every").as_int();
         }
+        chunk = (int)s.get_int("chunk", 0);
+        softcap = (float)s.get_double("softcap", 0.0);
+        unit_sink = s.get_bool("unit_sink", false);
+        const std::string vm = s.get_string("value_mix", "none");
+        if (vm != "none" && vm != "first" && vm != "mix") throw ConfigError("attention: value_mix '" + vm + "' is not supported (none, first, mix)");
+        keeps_values = vm == "first";
+        mixes_values = vm == "mix";
+        if (chunk < 0 || (chunk > 0 && window > 0)) throw ConfigError("attention: a layer has a window or a chunk, not both, and neither is negative");
+        if (softcap < 0.f) throw ConfigError("attention: softcap must be positive");
+        if (unit_sink && has_sink) throw ConfigError("attention: unit_sink and learned sinks exclude one another");
+        if ((chunk > 0 || softcap > 0.f || unit_sink || vm != "none" || wide_gate) && (maps == 2 || (values_are_keys && (chunk > 0 || softcap > 0.f || unit_sink || vm != "none"))))
+            throw ConfigError("attention: chunk, softcap, unit_sink and value_mix go neither with two score maps nor with values = keys");
+        if (vm != "none" && !own_kv) throw ConfigError("attention: value_mix needs keys and values of the layer's own");
         if (rt && values_are_keys && !ops::attention_mixed_supported(rt->dtype, n_heads, n_kv_heads, head_dim))
             throw ConfigError("attention: " + std::to_string(n_heads) + " heads of " + std::to_string(head_dim) +
                               " channels are beyond the kernel for mixed scores (heads x head size up to 8192)");
         names = {{"q", "q_proj.weight"}, {"k", "k_proj.weight"}, {"v", "v_proj.weight"}, {"o", "o_proj.weight"},
                  {"q_bias", "q_proj.bias"}, {"k_bias", "k_proj.bias"}, {"v_bias", "v_proj.bias"}, {"q_norm", "q_norm.weight"},
                  {"k_norm", "k_norm.weight"}, {"sink", "sinks"}, {"gate", "gate_proj.weight"}, {"r1", "r1"}, {"r2", "r2"}, {"mix", "mix"},
-                 {"o_bias", "o_proj.bias"}, {"lq1", "lambda_q1"}, {"lk1", "lambda_k1"}, {"lq2", "lambda_q2"}, {"lk2", "lambda_k2"}};
+                 {"o_bias", "o_proj.bias"}, {"lq1", "lambda_q1"}, {"lk1", "lambda_k1"}, {"lq2", "lambda_q2"}, {"lk2", "lambda_k2"}, {"v_mix", "v_mix"}};
         if (s.has("names"))
             for (auto& m : s.params.at("names").members()) names[m.first] = m.second.as_string();
         // the attention kernels read heads 16 bytes at a time: said when the model is built, not at its first step
@@ -463,7 +507,8 @@ struct Attention : Mixer {
     }
     // true if the layer needs the general path (see above)
     bool general() const {
-        return v_head_dim != head_dim || qkv_bias || proj_norm || has_sink || has_gate || !own_kv || out_f32 || maps == 2 || q_temp_every > 0 || o_bias;
+        return v_head_dim != head_dim || qkv_bias || proj_norm || has_sink || has_gate || !own_kv || out_f32 || maps == 2 || q_temp_every > 0 || o_bias ||
+               chunk > 0 || softcap > 0.f || unit_sink || keeps_values || mixes_values || wide_gate;
     }
     long long gate_rows() const { return has_gate ? n_heads : wide_gate ? (long long)n_heads * v_head_dim : 0; }
     bool graph_safe() const override { return true; }     // a decode step's launches depend only on the batch size
@@ -474,7 +519,7 @@ struct Attention : Mixer {
         const float* t;
         int rot;
         long long n;
-        return window == 0 && !values_are_keys && position->rotation_table(&t, &rot, &n);
+        return window == 0 && chunk == 0 && !values_are_keys && position->rotation_table(&t, &rot, &n);
     }
     TensorDecls tensors() const override {
         const long long q = (long long)n_heads * maps * head_dim, k = (long long)n_kv_heads * maps * head_dim, v = (long long)n_kv_heads * v_head_dim;
@@ -502,6 +547,7 @@ struct Attention : Mixer {
         if (head_mix) d.push_back({nm("mix"), TensorDecl{{(long long)n_heads, (long long)n_heads}}});
         if (maps == 2)
             for (const char* role : {"lq1", "lk1", "lq2", "lk2"}) d.push_back({nm(role), TensorDecl{{(long long)head_dim}}});
+        if (keeps_values || mixes_values) d.push_back({nm("v_mix"), TensorDecl{{}}});
         d.push_back({nm("o"), TensorDecl{{hidden, o}}});
         if (o_bias) d.push_back({nm("o_bias"), TensorDecl{{hidden}}});
         return d;
@@ -539,6 +585,13 @@ struct Attention : Mixer {
             if (own_kv) n_k = fetch_owned(rt, src, names.at("k_norm"), DType::F32, "a projection norm's weight");
         }
         if (has_sink) sinks = fetch_owned(rt, src, names.at("sink"), DType::F32, "the attention sinks");
+        if (unit_sink) {       // one more term exp(0) in every head's denominator
+            sinks.buf = DeviceBuffer(rt->dev, (size_t)n_heads * sizeof(float), "the attention sinks");
+            sinks.m = Mat{sinks.buf.get(), 1, n_heads, DType::F32, 1};
+            rt->dev->synchronize();
+            check_cuda(cudaMemset(sinks.m.p, 0, (size_t)n_heads * sizeof(float)), "clearing the attention sinks");
+        }
+        if (mixes_values) v_mix = fetch_owned(rt, src, names.at("v_mix"), DType::F32, "a value-mixing factor");
         if (log_distance) {
             dist_r1 = fetch_owned(rt, src, names.at("r1"), DType::F32, "an attention layer's distance factors");
             dist_r2 = fetch_owned(rt, src, names.at("r2"), DType::F32, "an attention layer's distance factors");
@@ -565,7 +618,7 @@ struct Attention : Mixer {
     }
     CacheRequest cache_request() const override {
         if (values_are_keys) return CacheRequest::paged_keys_only(n_kv_heads, head_dim, window);
-        return own_kv ? CacheRequest::paged(n_kv_heads, maps * head_dim, window, v_head_dim) : CacheRequest();
+        return own_kv ? CacheRequest::paged(n_kv_heads, maps * head_dim, window, v_head_dim).in_chunks(chunk) : CacheRequest();
     }
 
     // values = keys: one float32 product for q, k and the gate; q out and k into the pages (with the table rotation,
@@ -632,6 +685,15 @@ struct Attention : Mixer {
         p.n_pos = n_pos;
         p.q_temp_coef = q_temp_coef;
         p.q_temp_every = q_temp_every;
+        if (keeps_values) p.v_keep = (float*)ctx.keep(kFirstValues, x.rows, v_rows()).p;
+        if (mixes_values) {
+            auto it = ctx.kept.find(kFirstValues);
+            if (it == ctx.kept.end()) throw EngineError("attention: no earlier layer of the step kept its values");
+            if (it->second.rows != x.rows || it->second.cols != v_rows()) throw EngineError("attention: the kept values are not of this layer's width");
+            p.v_first = (const float*)it->second.p;
+            p.v_first_ld = (int)v_rows();
+            p.v_lambda = (const float*)v_mix.m.p;
+        }
         Mat q = ops::qk_prep(dev, x, p, g, ctx, kv, rt->dtype);
         if (maps == 2) {
             ops::DiffAttention da;
@@ -643,10 +705,12 @@ struct Attention : Mixer {
         }
         ops::AttentionExtras ex;
         ex.sinks = (const float*)sinks.m.p;
-        if (has_gate) {
+        if (has_gate || wide_gate) {
             ex.gate = (const float*)x.p + (q_rows() + k_rows() + v_rows());
             ex.gate_stride = (int)x.cols;
+            ex.wide_gate = wide_gate;
         }
+        ex.softcap = softcap;
         ex.wide_weights = true;       // the softmax weights are not to be rounded to eight bits
         Mat o = ops::attention_ex(dev, q, kv, ctx, g, scale, ex);
         return project_out(o, may_defer);
@@ -693,11 +757,13 @@ struct Attention : Mixer {
 // one product feeds the activation, and where the package's own kernels run that product the
 // activation is their epilogue (ops::linear_gated).
 // `names` renames the three tensors; `output_dtype` = "float32" leaves the down projection unrounded;
-// `activation` is "silu" (default), "relu" or "gelu_tanh" (each the epilogue of the package's own product kernels).
+// `activation` is "silu" (default), "relu", "gelu_tanh" or "swish_clamped" with `activation_limit` L (g = min(gate, L),
+// u = clamp(up, -L, L): g sigmoid(1.702 g) (u + 1)); each is the epilogue of the package's own product kernels.
 struct GatedMLP : FeedForward {
     long long hidden, inter;
     bool out_f32;
     int act;
+    float act_limit;
     std::string n_gate = "gate_proj.weight", n_up = "up_proj.weight", n_down = "down_proj.weight";
     DeviceBuffer gu_buf, down_buf;
     Mat w_gate_up, w_down;
@@ -705,8 +771,9 @@ struct GatedMLP : FeedForward {
             : FeedForward(s, rt), hidden(s.get_int("hidden_size")), inter(s.get_int("intermediate_size")),
               out_f32(s.get_string("output_dtype", "compute") == "float32") {
         act = ops::gate_act_from_name(s.get_string("activation", "silu"));
-        if (act < 0 || act == ops::kActSwishClamped)
-            throw ConfigError("gated_mlp: activation '" + s.get_string("activation", "silu") + "' is not supported (silu, relu, gelu_tanh)");
+        if (act < 0) throw ConfigError("gated_mlp: activation '" + s.get_string("activation", "silu") + "' is not supported (silu, relu, gelu_tanh, swish_clamped)");
+        act_limit = (float)s.get_double("activation_limit", 0.0);
+        if (act == ops::kActSwishClamped && !(act_limit > 0.f)) throw ConfigError("gated_mlp: swish_clamped needs a positive activation_limit");
         if (hidden <= 0 || inter <= 0) throw ConfigError("gated_mlp: sizes must be positive");
         if (s.has("names")) {
             const Json& n = s.params.at("names");
@@ -730,7 +797,7 @@ struct GatedMLP : FeedForward {
     }
     MatOrPartials forward(const Mat& h, const StepContext&, bool may_defer) override {
         Device& dev = *rt->dev;
-        return ops::linear(dev, rt->gemm, ops::linear_gated(dev, rt->gemm, h, w_gate_up, act), w_down, out_f32 ? DType::F32 : rt->dtype,
+        return ops::linear(dev, rt->gemm, ops::linear_gated(dev, rt->gemm, h, w_gate_up, act, act_limit), w_down, out_f32 ? DType::F32 : rt->dtype,
                            may_defer);
     }
 };
@@ -832,16 +899,19 @@ struct BigramEmbedding : EmbeddingPart {
 
 // Output head: logits = y . W_out^T in float32 (src/core/op.cpp:230-247 computes it for the last row
 // only and not at all on prefill, src/core/graph.cpp:132-141; here for the rows the caller wants).  A
-// tied head uses the embedding table (the reference has no tying).
+// tied head uses the embedding table (the reference has no tying).  `softcap` c > 0: logits <- c * tanh(logits / c).
 struct LMHead : HeadPart {
     long long vocab, hidden;
     bool is_tied;
     std::string tensor;
+    float softcap;
     OwnedMat own;
     Mat weight;
     LMHead(const PartSpec& s, Runtime* rt)
             : HeadPart(s, rt), vocab(s.get_int("vocab_size")), hidden(s.get_int("hidden_size")), is_tied(s.get_bool("tied", false)),
-              tensor(s.get_string("tensor", "weight")) {}
+              tensor(s.get_string("tensor", "weight")), softcap((float)s.get_double("softcap", 0.0)) {
+        if (softcap < 0.f) throw ConfigError("lm_head: softcap must be positive");
+    }
     TensorDecls tensors() const override {
         if (is_tied) return {};
         return {{tensor, TensorDecl{{vocab, hidden}}}};
@@ -856,7 +926,11 @@ struct LMHead : HeadPart {
         if (!e.table()) throw ConfigError("lm_head: tied to an embedding that has no table");
         weight = *e.table();
     }
-    Mat forward(const Mat& y, const StepContext&) override { return ops::linear(*rt->dev, rt->gemm, y, weight, DType::F32, false).m; }
+    Mat forward(const Mat& y, const StepContext&) override {
+        Mat logits = ops::linear(*rt->dev, rt->gemm, y, weight, DType::F32, false).m;
+        if (softcap > 0.f) ops::soft_cap(*rt->dev, logits, softcap);
+        return logits;
+    }
 };
 
 // "prenorm" is the reference's layer (src/graph/llama_like.cpp:69-105):

@@ -115,6 +115,21 @@ struct StepContext : StepView {
     Runtime* rt = nullptr;
     std::vector<int> q_lens, host_slots;
     std::vector<long long> past;
+    // What a layer keeps for later layers of the same step, by name: `keep` makes a float32 matrix in memory that outlives
+    // the layers' own activations (lane 0 of the step arena).  Emptied when a step's forward pass begins.
+    mutable std::map<std::string, Mat> kept;
+    Mat keep(const std::string& name, long long rows, long long cols) const {
+        Mat m;
+        m.rows = m.rows_held = rows;
+        m.cols = cols;
+        m.dtype = DType::F32;
+        const int lane = dev->lane();
+        dev->set_lane(0, false);
+        m.p = dev->alloc(m.bytes());
+        dev->set_lane(lane, false);
+        kept[name] = m;
+        return m;
+    }
 };
 
 // What a mixer gets of its cache entry for the step.

@@ -6,7 +6,8 @@
 // It can stand in front of a sublayer (Norm::forward) and behind one (add_normed_pending); where one of each follow
 // one another (a sublayer's output norm, then the next sublayer's input norm) both run in one kernel.
 //
-// "sandwich" / "sandwich_mixer": the block above, with and without a feed-forward.
+// "sandwich" / "sandwich_mixer": the block above, with and without a feed-forward.  Its norms are "layernorm" or
+// "rmsnorm" parts (parts/parts.cpp); the latter's `post_scale` is a constant factor on what joins the stream.
 //
 // "input_conv": a mixer around another mixer: what the inner mixer reads is h + conv(h), a causal convolution over
 // time with one filter of `taps` taps per channel (tensor `tensor` [width, taps], no bias).  The last taps - 1 rows of
@@ -38,7 +39,7 @@ struct LayerNorm : Norm {
         // added and normed again here; anything else that is pending is added first
         LayerNorm* post = stream.has_pending && !stream.has_pending2 ? dynamic_cast<LayerNorm*>(stream.pending_post) : nullptr;
         if (post && !stream.pending.is_partials() && stream.pending.m.dtype == DType::F32 && post->eps == eps) {
-            Mat y = ops::layernorm_sandwich(*rt->dev, stream.x, &stream.pending.m, &post->weight.m, &weight.m, eps, out_dtype(), rows, n_rows);
+            Mat y = ops::norm_sandwich(*rt->dev, stream.x, &stream.pending.m, &post->weight.m, &weight.m, eps, out_dtype(), rows, n_rows);
             if (rows == nullptr) {
                 stream.has_pending = false;
                 stream.pending_post = nullptr;
@@ -46,11 +47,11 @@ struct LayerNorm : Norm {
             return y;
         }
         if (stream.has_pending || stream.has_pending2) stream.flush();
-        return ops::layernorm_sandwich(*rt->dev, stream.x, nullptr, nullptr, &weight.m, eps, out_dtype(), rows, n_rows);
+        return ops::norm_sandwich(*rt->dev, stream.x, nullptr, nullptr, &weight.m, eps, out_dtype(), rows, n_rows);
     }
     void add_normed_pending(ResidualStream& stream) override {
         Mat y = stream.pending.is_partials() ? ops::materialize(*rt->dev, stream.pending.part, DType::F32) : ops::cast(*rt->dev, stream.pending.m, DType::F32);
-        ops::layernorm_sandwich(*rt->dev, stream.x, &y, &weight.m, nullptr, eps, DType::F32, nullptr, 0);
+        ops::norm_sandwich(*rt->dev, stream.x, &y, &weight.m, nullptr, eps, DType::F32, nullptr, 0);
         stream.has_pending = false;
     }
 };
