@@ -241,6 +241,29 @@ def tukulorn_config(z, vocab=32000, max_positions=4096):
                 loop=dict(start=1, stop=3, times=2))
 
 
+FIFOTAR_LAYERS = (("delta", "dense"), ("attention", "dense"), ("delta", "dense"), ("latent_attention", "dense"), ("delta", "dense"),
+                  ("attention", "dense"))
+
+
+def fifotar_config(z, vocab=32000, max_positions=4096):
+    """Six layers of the Fifotar design at the size z: delta-rule layers with the linear layers' head count, half as many
+    query/key heads and 128 x 128 state per head (as Vizosun), attention with the size's head counts in chunks of 1,024
+    positions, latent attention over all positions with a query latent of a quarter of the width and a cache row of 64
+    latent and 64 rotated channels (as Vizosun's and Tukulorn's), dense feed-forwards of the size's width."""
+    mlp = dict(kind="dense", ff=z["ff"], limit=7.0)
+    mixers = dict(delta=dict(heads=z["lin_heads"], kv_heads=max(1, z["lin_heads"] // 2), dim=z["lin_d"], vdim=z["lin_d"], conv=4),
+                  attention=dict(heads=z["heads"], kv_heads=z["kv"], dim=z["d"], vdim=z["d"], scale=z["d"] ** -0.5, softcap=50.0, v_mix=True,
+                                 mask=dict(size=1024)),
+                  latent_attention=dict(heads=z["heads"], dim=z["d"], rot_dim=64, vdim=z["d"], q_rank=z["width"] // 4, kv_rank=64,
+                                        scale=(z["d"] + 64) ** -0.5, rot=dict(base=500000.0, dims=64, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0))))
+    return dict(architecture="Fifotar", layers=[dict(type=t, mixer=dict(mixers[t]), mlp=mlp) for t, _ in FIFOTAR_LAYERS], norm=dict(eps=1e-5),
+                embedding=dict(scale=8.0), residual_mult=0.5, logit_softcap=30.0, vocab=vocab, width=z["width"], max_positions=max_positions)
+
+
+DESIGN_LAYER_NAMES = {"vokelix": list(DESIGN_LAYERS), "vizosun": ["/".join(x) for x in VIZOSUN_LAYERS], "kudonex": list(KUDONEX_LAYERS),
+                      "tukulorn": ["/".join(x) for x in TUKULORN_LAYERS], "fifotar": ["/".join(x) for x in FIFOTAR_LAYERS], "llama": len(DESIGN_LAYERS)}
+
+
 def llama_twin(z, vocab=32000, max_positions=4096):
     return dict(architectures=["LlamaForCausalLM"], hidden_size=z["width"], num_hidden_layers=len(DESIGN_LAYERS),
                 num_attention_heads=z["heads"], num_key_value_heads=z["kv"], head_dim=z["d"], intermediate_size=z["ff"],
@@ -251,7 +274,8 @@ def llama_twin(z, vocab=32000, max_positions=4096):
 def run_design(args):
     """Prompt and decode throughput of a design at a few layer sizes, each beside the closest other
     model of the same width, feed-forward, head counts and number of layers (Vokelix beside LLaMA;
-    Vizosun beside Vokelix and LLaMA; Kudonex and Tukulorn beside all three), through Engine.step; and
+    Vizosun beside Vokelix and LLaMA; Kudonex and Tukulorn beside all three; Fifotar beside Vizosun, Tukulorn
+    and LLaMA), through Engine.step; and
     where each of the two spends its time, kernel by kernel (the driver's activity records of one step).
     One JSON line per (size, model)."""
     import torch
@@ -294,6 +318,8 @@ def run_design(args):
             arms = (("kudonex", kudonex_config(z)), ("vizosun", vizosun_config(z))) + arms
         if args.design == "tukulorn":
             arms = (("tukulorn", tukulorn_config(z)), ("vizosun", vizosun_config(z))) + arms
+        if args.design == "fifotar":
+            arms = (("fifotar", fifotar_config(z)), ("vizosun", vizosun_config(z)), ("tukulorn", tukulorn_config(z)), arms[1])
         for which, cfgd in arms:
             eng = Engine.from_config(config_from_dict(cfgd), EngineOptions(dtype="bfloat16", max_tokens=max(B * (C + 64), NP * (T + 64)) + 64,
                                                                            max_seq_len=4096, max_batch=max(B, NP, 8)), seed=0)
@@ -323,7 +349,7 @@ def run_design(args):
             dec_ms = timed(one, K)
             for s in slots:
                 eng.end_sequence(s)
-            print(json.dumps({"design": which, "size": size, "layers": list(DESIGN_LAYERS) if which == "vokelix" else ["/".join(x) for x in VIZOSUN_LAYERS] if which == "vizosun" else list(KUDONEX_LAYERS) if which == "kudonex" else ["/".join(x) for x in TUKULORN_LAYERS] if which == "tukulorn" else len(DESIGN_LAYERS),
+            print(json.dumps({"design": which, "size": size, "layers": DESIGN_LAYER_NAMES[which],
                               "prefill_tokens": T, "prefill_prompts": NP, "prefill_ms": round(pf_ms, 3), "prefill_tok_s": round(NP * T / pf_ms * 1e3, 1),
                               "decode_batch": B, "decode_context": C, "decode_ms": round(dec_ms, 4),
                               "decode_tok_s": round(B / dec_ms * 1e3, 1), "prefill_kernels_us": pf_kernels,
@@ -556,7 +582,7 @@ def main():
                     "lengths uniform in [MIN, MAX] (seeded) prefilled in one step of unequal lengths, then NEW tokens "
                     "each (or 'toN': until position N), through the Python entry point; 'config' = the workload of --model "
                     "(8b: 16:64:2048:256, 13b: 32:128:1024:to4096)")
-    ap.add_argument("--design", choices=["vokelix", "vizosun", "kudonex", "tukulorn"], help="beside the default workload: prompt and decode throughput of this design "
+    ap.add_argument("--design", choices=["vokelix", "vizosun", "kudonex", "tukulorn", "fifotar"], help="beside the default workload: prompt and decode throughput of this design "
                     "at a few layer sizes, each next to LLaMA layers of equal size, with the time per kernel")
     ap.add_argument("--design-size", default="1k,2k,4k", help="with --design: sizes to run (1k, 2k, 4k: the width)")
     ap.add_argument("--design-tokens", type=int, default=2048, help="with --design: tokens of the prompt")

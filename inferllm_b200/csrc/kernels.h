@@ -147,7 +147,11 @@ int illm_head_gemm_ex(const void* x, int x_dtype, const void* w, int w_dtype, vo
 int illm_moe_route_ex2(const float* logits, const float* bias, int T, int E, int top, int bm, int scoring, int groups, int keep, int renorm, int group_top, float sum_eps, float weight_scale, int* expert, float* weight, int* row_of_pair, int* pair_of_row, int* tile_expert, int* tile_row0, int* tile_rows, void* stream);
 int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated, int act, float act_limit, int bm, int tensor_cores, const int* pair_of_row, const int* tile_expert, const int* tile_row0, const int* tile_rows, void* stream);
 int illm_moe_gemm_tc_ex(const void* xs, const void* w, void* y, int P, int E, int N, int K, int gated, int act, float act_limit, int tiles, const int* tile_expert, const int* tile_row0, const int* tile_rows, int* err, void* stream);
-// attention_diff.cu
+// attention_maps.cu
+long long illm_attention_maps_scratch(int T, int nh, int dv, int maps, int splits);
+int illm_attention_one_mma_supported(int d, int dv);
+int illm_attention_one_mma(const void* q, int q_stride, const void* kc, const void* vc, const int* block_table, int max_pages, const int* cu_q, const int* seq_lens, void* out, int B, int max_q, int nh, int nkv, int d, int dv, int page_size, int span, float scale, float softcap, const float* sinks, const float* gate, int gate_stride, int gate_wide, void* stream);
+int illm_attention_one_decode(const void* q, int q_stride, const void* kc, const void* vc, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, void* out, int T, int nh, int nkv, int d, int dv, int page_size, int span, float scale, float softcap, const float* sinks, const float* gate, int gate_stride, int gate_wide, long long longest, int splits, float* scratch, void* stream);
 int illm_attention_diff(const void* q, int q_stride, const void* kc, const void* vc, const int* block_table, int max_pages, const int* token_pos, const int* token_seq, void* out, int act_dtype, int T, int nh, int nkv, int d, int dv, int page_size, int window, float scale, float lambda, float eps, float out_scale, int splits, float* scratch, void* stream);
 long long illm_attention_diff_scratch(int T, int nh, int dv, int splits);
 int illm_attention_diff_mma_supported(int d, int dv);

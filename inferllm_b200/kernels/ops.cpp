@@ -729,6 +729,38 @@ Mat attention_decode_ex(Device& dev, const Mat& qkv, const KVView& kv, const Ste
     return out;
 }
 
+bool attention_one_supported(int nh, int nkv, int d, int dv, bool decode) {
+    if (nkv <= 0 || nh % nkv) return false;
+    return decode ? illm_attention_diff_decode_supported(nh, nkv, d, dv) != 0 : illm_attention_one_mma_supported(d, dv) != 0;
+}
+
+Mat attention_one(Device& dev, const Mat& q, const KVView& kv, const StepView& ctx, Geometry g, float scale, const AttentionExtras& ex) {
+    need(q, "q", true, DType::BF16);
+    check_cache(kv, DType::BF16, g, "attention_one");
+    const int dv = kv.v_head_dim > 0 ? kv.v_head_dim : g.head_dim;
+    if (!attention_one_supported(g.n_heads, g.n_kv_heads, g.head_dim, dv, ctx.is_decode) || q.cols % 8)
+        throw KernelError("attention_one: heads of " + std::to_string(g.head_dim) + " and " + std::to_string(dv) + " channels are not supported");
+    Mat out = new_mat(dev, q.rows, (long long)g.n_heads * dv, DType::BF16);
+    if (!ctx.is_decode) {
+        check_kernel(illm_attention_one_mma(q.p, (int)q.cols, kv.k, kv.v, kv.block_table, kv.width, ctx.cu_q, ctx.seq_lens, out.p, ctx.B, ctx.max_q, g.n_heads,
+                                            g.n_kv_heads, g.head_dim, dv, kv.page_size, kv.span(), scale, ex.softcap, ex.sinks, ex.gate, ex.gate_stride,
+                                            ex.wide_gate ? 1 : 0, dev.stream()),
+                     "attention_one_mma");
+        return out;
+    }
+    // grids and scratch of a single-token step are sized for the longest range of keys the cache allows, so that the launch is
+    // the same at every step
+    const int group = g.n_heads / g.n_kv_heads, hb = group >= 8 ? 8 : group > 2 ? 4 : group;
+    const long long longest = kv.chunk > 0 ? std::min<long long>(kv.chunk, ctx.max_seq_len) : ctx.max_seq_len;
+    const int splits = attention_diff_splits(q.rows, g.n_kv_heads * (int)ceil_div(group, hb), longest, dev.n_sms());
+    float* scratch = dev.alloc_n<float>((size_t)illm_attention_maps_scratch((int)q.rows, g.n_heads, dv, 1, splits));
+    check_kernel(illm_attention_one_decode(q.p, (int)q.cols, kv.k, kv.v, kv.block_table, kv.width, ctx.token_pos, ctx.token_seq, out.p, (int)q.rows, g.n_heads,
+                                           g.n_kv_heads, g.head_dim, dv, kv.page_size, kv.span(), scale, ex.softcap, ex.sinks, ex.gate, ex.gate_stride,
+                                           ex.wide_gate ? 1 : 0, longest, splits, scratch, dev.stream()),
+                 "attention_one_decode");
+    return out;
+}
+
 Mat attention_ex(Device& dev, const Mat& q, const KVView& kv, const StepView& ctx, Geometry g, float scale, const AttentionExtras& ex) {
     const int dv = kv.v_head_dim > 0 ? kv.v_head_dim : g.head_dim;
     if (q.dtype == DType::BF16 && dv == g.head_dim) {
@@ -744,6 +776,9 @@ Mat attention_ex(Device& dev, const Mat& q, const KVView& kv, const StepView& ct
         if (!ctx.is_decode && attention_prefill_tc_supported(q.dtype, g.n_heads, g.n_kv_heads, g.head_dim, kv.page_size))
             return attention_prefill_tc(dev, q, kv, ctx, g, scale, &ex);
     }
+    if (q.dtype == DType::BF16 && attention_one_supported(g.n_heads, g.n_kv_heads, g.head_dim, dv, ctx.is_decode) && q.cols % 8 == 0 &&
+        (kv.k != kv.v || dv == g.head_dim))
+        return attention_one(dev, q, kv, ctx, g, scale, ex);
     return attention_generic(dev, q, kv, ctx, g, scale, &ex);
 }
 

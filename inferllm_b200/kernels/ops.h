@@ -194,8 +194,14 @@ Mat attention_prefill_tc(Device& dev, const Mat& qkv, const KVView& kv, const St
 Mat attention_decode_ex(Device& dev, const Mat& qkv, const KVView& kv, const StepView& ctx, Geometry g, float scale, long long max_len,
                         const AttentionExtras& extras);
 // Attention with extras: the tensor-core prompt kernel and the ring or split-key decode kernel where the sizes allow
-// (bfloat16, keys and values of one size, 64 or 128), the general kernel otherwise.  Windows and chunks (KVView::span).
+// (bfloat16, keys and values of one size, 64 or 128), attention_one for other sizes in bfloat16, the general kernel
+// otherwise.  Windows and chunks (KVView::span).
 Mat attention_ex(Device& dev, const Mat& q, const KVView& kv, const StepView& ctx, Geometry g, float scale, const AttentionExtras& extras);
+// Softmax attention in bfloat16 for head sizes that are multiples of 8 up to 256, keys and values of any two such sizes
+// (csrc/attention_maps.cu, one score map): prompts on warp-level MMA with 64-token tiles, single tokens on a kernel that
+// reads every key and value row once for the query heads that share it.
+bool attention_one_supported(int nh, int nkv, int d, int dv, bool decode);
+Mat attention_one(Device& dev, const Mat& q, const KVView& kv, const StepView& ctx, Geometry g, float scale, const AttentionExtras& ex);
 // Attention whose heads' scores are mixed before the softmax (mix float32 [n_heads, n_heads] or nullptr), with a
 // logarithmic distance penalty r1_h ln(1 + r2_h (i - j)) (r1, r2 float32 [n_heads] or nullptr), over a keys-only
 // cache entry whose keys are also the values, and an element-wise sigmoid gate (float32 [T, gate_stride] or nullptr).
@@ -205,7 +211,7 @@ struct MixedAttention {
 };
 bool attention_mixed_supported(DType dtype, int nh, int nkv, int d);
 Mat attention_mixed(Device& dev, const Mat& q, const KVView& kv, const StepView& ctx, Geometry g, float scale, const MixedAttention& m);
-// Differential attention (csrc/attention_diff.cu): every head has two score maps over the same values.  q [T, heads * 2 d]
+// Differential attention (csrc/attention_maps.cu): every head has two score maps over the same values.  q [T, heads * 2 d]
 // (a head's row is [q_1, q_2]), the cache entry's key rows [k_1, k_2] (kv.head_dim == 2 d) and value rows of
 // kv.v_head_dim; o = a_1 - lambda a_2, divided by its root mean square over the head's values (eps inside the root), times
 // out_scale.  g.head_dim is d, the size of ONE map.  Returns [T, heads * v_head_dim] in q's dtype.

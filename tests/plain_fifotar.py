@@ -225,3 +225,128 @@ def greedy_generate(cfg, W, prompt, n_new):
     for _ in range(n_new):
         ids.append(int(np.argmax(forward(cfg, W, ids)[-1])))
     return ids[len(prompt):]
+
+
+# ---------------------------------------------------------------- test infrastructure: configurations and weights
+
+
+def delta_mixer(heads=6, kv_heads=2, dim=12, vdim=20, conv=4):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}
+
+
+def chunk_mixer(heads=4, kv_heads=2, dim=24, vdim=16, size=20, scale=0.3, softcap=9.0, v_mix=True):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "softcap": softcap, "v_mix": v_mix}
+    if size:
+        m["mask"] = {"size": size}
+    return m
+
+
+def latent_mixer(heads=3, dim=16, rot_dim=8, vdim=24, q_rank=28, kv_rank=40, scale=0.25, base=100.0, scaling=(3.0, 64, 4.0, 1.0)):
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": scale,
+         "rot": {"base": base, "dims": rot_dim}}
+    if scaling:
+        m["rot"]["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return m
+
+
+def dense(ff=40, limit=1.5):
+    return {"kind": "dense", "ff": ff, "limit": limit}
+
+
+def make_config(layers, width=48, vocab=97, eps=1e-5, scale=3.0, mult=0.6, logit_softcap=20.0, max_positions=2048):
+    """layers: a list of (type, mixer, mlp or None)."""
+    return {"architecture": "Fifotar", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale}, "residual_mult": mult,
+            "logit_softcap": logit_softcap, "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in layers], "max_positions": max_positions}
+
+
+def tensor_shapes(cfg):
+    """name -> (shape, kind); kind says how random_weights draws the tensor."""
+    width = cfg["width"]
+    out = {"embed": ((cfg["vocab"], width), "embed"), "final.norm": ((width,), "norm")}
+    for i, L in enumerate(cfg["layers"]):
+        p, m = "l%d." % i, L["mixer"]
+        x = p + "mix."
+        out[p + "norm1"] = out[p + "norm1b"] = ((width,), "norm")
+        H, dv = m["heads"], m["vdim"]
+        if L["type"] == "delta":
+            G, d, K = m["kv_heads"], m["dim"], m["conv"]
+            for t, rows in (("q", G * d), ("k", G * d), ("v", H * dv)):
+                out[x + t] = ((rows, width), "mat")
+                out[x + t + ".conv"] = ((rows, K), "conv")
+            out.update({x + "b": ((H, width), "mat"), x + "A_log": ((H,), "a_log"), x + "norm": ((dv,), "norm"), x + "a": ((H, width), "mat"),
+                        x + "dt_bias": ((H,), "dt"), x + "g": ((H * dv, width), "mat"), x + "o": ((width, H * dv), "mat")})
+        elif L["type"] == "attention":
+            G, d = m["kv_heads"], m["dim"]
+            out.update({x + "q": ((H * d, width), "mat"), x + "k": ((G * d, width), "mat"), x + "v": ((G * dv, width), "mat"),
+                        x + "g": ((H * dv, width), "mat"), x + "o": ((width, H * dv), "mat")})
+            if m.get("v_mix"):
+                out[x + "vmix"] = ((), "lambda")
+        else:
+            d, dr, qr, rank = m["dim"], m["rot_dim"], m["q_rank"], m["kv_rank"]
+            out.update({x + "dq": ((qr, width), "mat"), x + "dq.norm": ((qr,), "norm"), x + "uq": ((H * (d + dr), qr), "mat"),
+                        x + "dkv": ((rank + dr, width), "mat"), x + "dkv.norm": ((rank,), "norm"), x + "uk": ((H * d, rank), "mat"),
+                        x + "uv": ((H * dv, rank), "mat"), x + "g": ((H, width), "mat"), x + "o": ((width, H * dv), "mat")})
+        if L.get("mlp"):
+            f, ff = p + "mlp.", L["mlp"]["ff"]
+            out[p + "norm2"] = out[p + "norm2b"] = ((width,), "norm")
+            out.update({f + "gate": ((ff, width), "gate"), f + "up": ((ff, width), "gate"), f + "down": ((width, ff), "mat")})
+    return out
+
+
+def bf16_round(a):
+    """float32 array rounded to the nearest bfloat16 value (ties to even), still float32."""
+    u = np.ascontiguousarray(a, np.float32).view(np.uint32).astype(np.uint64)
+    u = ((u + 0x7FFF + ((u >> 16) & 1)) >> 16) << 16
+    return u.astype(np.uint32).view(np.float32).reshape(np.shape(a))
+
+
+def random_weights(cfg, seed, gain=1.0):
+    """Random weights, rounded to bfloat16 values.  Drawn so that faults show: norm weights far from 1, convolution taps of
+    like size, decays spread over (0, 1), gate and up maps that reach the feed-forward's limit, a mixing factor far from 0."""
+    rng, w = np.random.default_rng(seed), {}
+    for name, (shape, kind) in tensor_shapes(cfg).items():
+        n_in = shape[-1] if shape else 1
+        z = rng.standard_normal(shape)
+        if kind == "mat":
+            a = z * gain / math.sqrt(n_in)
+        elif kind == "gate":
+            a = z * 1.5 * gain / math.sqrt(n_in)
+        elif kind == "embed":
+            a = z
+        elif kind == "norm":
+            a = 1.0 + 0.3 * z
+        elif kind == "conv":
+            a = 0.8 * z / math.sqrt(n_in) + 0.3
+        elif kind == "a_log":
+            a = 0.5 * z - 1.0
+        elif kind == "dt":
+            a = z - 1.0
+        elif kind == "lambda":
+            a = 0.5 + 0.15 * z
+        else:
+            raise ValueError(kind)
+        w[name] = bf16_round(np.asarray(a, np.float32))
+    return w
+
+
+def write_model(folder, cfg, w):
+    """config.json and model.safetensors (bfloat16) of (cfg, w) in `folder`."""
+    import json
+    import os
+    import struct
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    header, blobs, off = {}, [], 0
+    for name, a in w.items():
+        blob = (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype("<u2").tobytes()
+        header[name] = {"dtype": "BF16", "shape": list(np.shape(a)), "data_offsets": [off, off + len(blob)]}
+        blobs.append(blob)
+        off += len(blob)
+    hj = json.dumps(header).encode()
+    hj += b" " * (-len(hj) % 8)
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(hj)))
+        f.write(hj)
+        for b in blobs:
+            f.write(b)

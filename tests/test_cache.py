@@ -70,6 +70,19 @@ def test_window_releases_pages_that_left_the_window():
     assert sorted(led1.pages[0]) == [2]
 
 
+def test_chunks_release_pages_of_finished_chunks():
+    led = PageLedger(num_pages=16, page_size=4, num_slots=1, chunk=10)
+    led.reserve(0, 19)
+    led.release_outside_window(0, 19)      # the next query (19) still sees 10 .. 19: pages 2, 3, 4
+    assert sorted(led.pages[0]) == [2, 3, 4]
+    led.reserve(0, 20)
+    led.release_outside_window(0, 20)      # the next query starts a chunk: nothing before position 20 is seen again
+    assert led.pages[0] == {}
+    led.reserve(0, 21)
+    assert sorted(led.pages[0]) == [5]
+    led.check()
+
+
 def _cache(num_slots=3, num_pages=6, page=4, max_len=16, extra=None):
     reqs = {0: PagedKV(2, 8), 1: PagedKV(2, 8)}
     reqs.update(extra or {})
@@ -152,7 +165,7 @@ def test_freed_slots_and_pages_are_used_again():
 
 def test_random_walk_keeps_invariants():
     rng = random.Random(3)
-    c = _cache(num_slots=5, num_pages=12, page=4, max_len=24, extra={2: PagedKV(1, 8, window=6)})
+    c = _cache(num_slots=5, num_pages=12, page=4, max_len=24, extra={2: PagedKV(1, 8, window=6), 3: PagedKV(1, 8, chunk=7)})
     live = {}
     for _ in range(600):
         r = rng.random()
@@ -183,13 +196,15 @@ def test_random_walk_keeps_invariants():
                 for gi, g in enumerate(c.stats()["paged"]):
                     w = g["request"]["window"]
                     lo = max(0, live[s] - w + 1) if w else 0
+                    if g["request"].get("chunk"):
+                        lo = live[s] // g["request"]["chunk"] * g["request"]["chunk"]
                     held = c.pages_of(gi, s)
                     for pos in range(lo, live[s]):
                         assert pos // 4 in held
         c.check()
     c.reset()
     c.check()
-    assert c.slots_free == 5 and c.pages_free() == [12, 12]
+    assert c.slots_free == 5 and c.pages_free() == [12, 12, 12]
 
 
 def test_a_step_that_failed_gives_its_pages_back():
