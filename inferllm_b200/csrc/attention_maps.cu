@@ -621,8 +621,9 @@ attention_maps_mma_kernel(const bf16* __restrict__ q, int q_stride, const bf16* 
     pdl_grid_sync();
     constexpr int NT_V = DV / 8;          // n-tiles of the output
     const int KW = MAPS * d;              // channels of a query or key row (all maps)
-    const int KP = (KW + 15) & ~15;       // and as staged
+    const int KP = MAPS == 2 ? KW : (KW + 15) & ~15;      // and as staged
     const bool shared_kv = MAPS == 1 && kc == vc;              // the key tile is the value tile
+    const int dvw = MAPS == 2 ? DV : dv;                       // channels of a value row
     const int LDK = KP + 8, LDV = shared_kv ? LDK : DV + 8;    // padded rows (elements)
     const int CHK = KP / 8, CHV = shared_kv ? 0 : DV / 8;      // 16-byte chunks per row
     const int span = ma.span;
@@ -651,7 +652,7 @@ attention_maps_mma_kernel(const bf16* __restrict__ q, int q_stride, const bf16* 
 
     for (int i = tid; i < DM_BM * CHK; i += DM_THREADS) {
         const int r = i / CHK, c = i - r * CHK;
-        const bool ok = r < rows_here && c * 8 < KW;
+        const bool ok = r < rows_here && (MAPS == 2 || c * 8 < KW);
         const bf16* src = ok ? q + (size_t)(q0 + row0 + r) * q_stride + (size_t)h * KW + c * 8 : q;
         dm_cp16(dm_smem(Qs + r * LDK + c * 8), src, ok ? 16 : 0);
     }
@@ -671,11 +672,11 @@ attention_maps_mma_kernel(const bf16* __restrict__ q, int q_stride, const bf16* 
                 if (ok) rowi = ((size_t)page * nkv + hk) * page_size + (key % page_size);
             }
             if (c < CHK) {
-                const bool in = ok && c * 8 < KW;
+                const bool in = ok && (MAPS == 2 || c * 8 < KW);
                 dm_cp16(dm_smem(kd + r * LDK + c * 8), in ? kc + rowi * KW + c * 8 : kc, in ? 16 : 0);
             } else {
-                const bool in = ok && (c - CHK) * 8 < dv;
-                dm_cp16(dm_smem(vd + r * LDV + (c - CHK) * 8), in ? vc + rowi * dv + (c - CHK) * 8 : vc, in ? 16 : 0);
+                const bool in = ok && (MAPS == 2 || (c - CHK) * 8 < dvw);
+                dm_cp16(dm_smem(vd + r * LDV + (c - CHK) * 8), in ? vc + rowi * dvw + (c - CHK) * 8 : vc, in ? 16 : 0);
             }
         }
     };
@@ -740,7 +741,8 @@ attention_maps_mma_kernel(const bf16* __restrict__ q, int q_stride, const bf16* 
                         if (MAPS == 1 && ma.softcap > 0.f) v = 1.4426950408889634f * soft_cap_fast(s[nt][e], ma.softcap, ma.cap_x);
                         if (need_mask) {
                             const int key = key0 + nt * 8 + t4 * 2 + (e & 1);
-                            if (key > pos_r[e >> 1] || key < lo_r[e >> 1]) v = -INFINITY;
+                            const int pr = pos_r[e >> 1];
+                            if (key > pr || (MAPS == 2 ? (span > 0 && key < pr - span + 1) : key < lo_r[e >> 1])) v = -INFINITY;
                         }
                         s[nt][e] = v;
                         m_new[e >> 1] = fmaxf(m_new[e >> 1], v);

@@ -169,6 +169,11 @@ __device__ __forceinline__ unsigned long long f2_fma(unsigned long long a, unsig
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
     return r;
 }
+__device__ __forceinline__ unsigned long long f2_mul(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
 __device__ __forceinline__ unsigned long long f2_add(unsigned long long a, unsigned long long b) {
     unsigned long long r;
     asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
@@ -180,14 +185,37 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
     return r;
 }
 
+// A soft cap on the scores.  The special-function unit would need two operations per score for it, beside the exponential
+// of the softmax, and the softmax warps would be bound by it; so while all of a warp's scores of a block lie within
+// `limit` (0.6 cap / scale), where tanh x is x times a polynomial in x^2 (minimax, relative error 7e-8), the capped score
+// cap log2(e) tanh(q.k scale / cap) is q.k times a polynomial in (q.k)^2 with the coefficients a[] (two scores per instruction).
+// Blocks with a score beyond that take the exponential form (soft_cap_fast with cap2 = cap log2(e), cap_x).
+struct FtCap {
+    float a[5], limit, cap2, cap_x;
+};
+static FtCap ft_make_cap(float softcap, float scale) {
+    const double c[5] = {0.999999927, -0.3333231, 0.133101737, -0.0521014808, 0.015475427};
+    const double k = (double)scale / softcap, cap2 = (double)softcap * 1.4426950408889634;
+    FtCap r;
+    double kp = k;
+    for (int i = 0; i < 5; i++) {
+        r.a[i] = (float)(cap2 * c[i] * kp);
+        kp *= k * k;
+    }
+    r.limit = (float)(0.6 / (k < 0 ? -k : k));
+    r.cap2 = (float)cap2;
+    r.cap_x = (float)(2.0 * k * 1.4426950408889634);
+    return r;
+}
+
 // WIDE_P: the softmax weights enter the product with V as two bfloat16 terms, P = P1 + P2 with
 // P2 = P - P1 rounded again (sixteen bits of mantissa instead of eight): P2 lies in the other half of
 // the S block's columns and P V is issued once more with it.  For mixers whose softmax weights are to
 // stay float32; the plain attention passes false and is compiled as before.  `sinks` (float32 [nh]):
 // one more term exp(sink) of the row's denominator, without a value; `gate` (float32,
 // gate[row * gate_stride + head], or with gate_wide gate[row * gate_stride + head * D + channel]): the output is multiplied by
-// its sigmoid.  Either may be nullptr.  CAP: the scaled scores s become cap * tanh(s / cap) before the mask; the kernel
-// then works on capped scores and its scale is log2(e) (cap, and 2 scale log2(e) / cap as cap_x).
+// its sigmoid.  Either may be nullptr.  CAP: the scaled scores s become cap * tanh(s / cap) before the mask (FtCap); the kernel
+// then works on capped scores in units of log2 and its scale is 1.
 template <int D, bool WIDE_P, bool CAP>
 __global__ void __launch_bounds__(FT_THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -195,7 +223,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             int max_pages, const int* __restrict__ cu_q, const int* __restrict__ seq_lens,
                             bf16* __restrict__ out, int nh, int nkv, int page_size, int span,
                             float scale_log2e, int* __restrict__ err, const float* __restrict__ sinks,
-                            const float* __restrict__ gate, int gate_stride, int gate_wide, float cap, float cap_x) {
+                            const float* __restrict__ gate, int gate_stride, int gate_wide, const FtCap cap) {
     constexpr int FT_MMA_WARP = 4, FT_TMA_WARP = 5;
     constexpr int NA = D / 64;                            // 64-channel atoms of the head
     constexpr unsigned Q_TILE = FT_BM * D * 2;            // the query tile: [NA][128 rows][128 B]
@@ -372,8 +400,26 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tmem_ld32_issue(s_addr + 32, sr + 32);
             tmem_wait_ld<FT_BN>(sr);
             if (CAP) {
+                float top = 0.f;
 #pragma unroll
-                for (int c = 0; c < FT_BN; c++) sr[c] = __float_as_uint(soft_cap_fast(__uint_as_float(sr[c]), cap, cap_x));
+                for (int c = 0; c < FT_BN; c += 2) top = max3(top, fabsf(__uint_as_float(sr[c])), fabsf(__uint_as_float(sr[c + 1])));
+                if (__any_sync(0xffffffffu, !(top <= cap.limit))) {
+#pragma unroll
+                    for (int c = 0; c < FT_BN; c++) sr[c] = __float_as_uint(soft_cap_fast(__uint_as_float(sr[c]), cap.cap2, cap.cap_x));
+                } else {
+                    const unsigned long long a0 = f2_pack(cap.a[0], cap.a[0]), a1 = f2_pack(cap.a[1], cap.a[1]), a2 = f2_pack(cap.a[2], cap.a[2]),
+                                             a3 = f2_pack(cap.a[3], cap.a[3]), a4 = f2_pack(cap.a[4], cap.a[4]);
+#pragma unroll
+                    for (int c = 0; c < FT_BN; c += 2) {
+                        const unsigned long long s = f2_pack(__uint_as_float(sr[c]), __uint_as_float(sr[c + 1]));
+                        const unsigned long long y = f2_mul(s, s);
+                        const unsigned long long p = f2_fma(f2_fma(f2_fma(f2_fma(a4, y, a3), y, a2), y, a1), y, a0);
+                        float lo, hi;
+                        f2_unpack(f2_mul(s, p), lo, hi);
+                        sr[c] = __float_as_uint(lo);
+                        sr[c + 1] = __float_as_uint(hi);
+                    }
+                }
             }
             const bool need_mask = (key0 + FT_BN - 1 > first_pos) || (span != 0);
             if (need_mask) {
@@ -510,8 +556,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                         for (int e = 0; e < 8; e++) f[e] = __uint_as_float(orr[c + e]) * inv;
                         if (gate && gate_wide) {
                             const float* gr = gate + (size_t)(q0 + row0 + r) * gate_stride + (size_t)h * D + c0 + c;
+                            float g8[8];
+                            if (gate_wide == 2) {          // rows of whole 16-byte pieces
+                                load8(gr, g8);
+                            } else {
 #pragma unroll
-                            for (int e = 0; e < 8; e++) f[e] *= 1.0f / (1.0f + expf(-gr[e]));
+                                for (int e = 0; e < 8; e++) g8[e] = gr[e];
+                            }
+#pragma unroll
+                            for (int e = 0; e < 8; e++) f[e] = __fdividef(f[e], 1.0f + __expf(-g8[e]));
                         }
                         store8(dst + c0 + c, f);
                     }
@@ -577,8 +630,8 @@ static int ft_launch(const void* q, int q_stride, int T, const void* kc, const v
     if (e != cudaSuccess) return (int)e;
     dim3 grid(nh, (max_q + FT_BM - 1) / FT_BM, B);
     illm_launch(kern, grid, dim3(FT_THREADS), smem, s, mq, mk, mv, block_table, max_pages, cu_q, seq_lens,
-                (bf16*)out, nh, nkv, page_size, span, (CAP ? 1.0f : scale) * 1.4426950408889634f, err, sinks, gate, gate_stride, gate_wide, softcap,
-                CAP ? 2.0f * scale * 1.4426950408889634f / softcap : 0.f);
+                (bf16*)out, nh, nkv, page_size, span, CAP ? 1.0f : scale * 1.4426950408889634f, err, sinks, gate, gate_stride, gate_wide,
+                CAP ? ft_make_cap(softcap, scale) : FtCap{});
     return illm_launch_status();
 }
 
@@ -597,6 +650,7 @@ extern "C" int illm_attention_prefill_tc_ex(const void* q, int q_stride, int T, 
         return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     if (softcap > 0.f && !wide_p) return ILLM_ERR_BAD_ARG;
+    if (gate && gate_wide) gate_wide = gate_stride % 4 == 0 && !((uintptr_t)gate & 15) ? 2 : 1;
 #define FT_CASE(DD, WW, CC)                                                                                                   \
     if (d == DD && (wide_p != 0) == WW && (softcap > 0.f) == CC)                                                              \
         return ft_launch<DD, WW, CC>(q, q_stride, T, kc, vc, n_pages, block_table, max_pages, cu_q, seq_lens, out, B, max_q, \

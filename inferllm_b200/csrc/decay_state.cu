@@ -522,6 +522,51 @@ __global__ void __launch_bounds__(128) group_norm_gate_kernel(GroupNormGateArgs 
     }
 }
 
+// The same without factors, skips and gates in front, for groups of up to 512 columns in rows of whole 16-byte pieces: a warp
+// per (token, group), four neighbouring columns per lane and load, a lane's part of the sum in the order of its columns.
+// Which of the two kernels runs follows from the sizes and the layout of the rows alone.
+template <typename TA, int NV>
+__global__ void __launch_bounds__(256) group_norm_gate_vec_kernel(GroupNormGateArgs a, TA* __restrict__ y, int T) {
+    pdl_grid_sync();
+    const int groups = a.width / a.group, lane = threadIdx.x & 31;
+    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (item >= (long long)T * groups) return;
+    const int t = (int)(item / groups), g0 = (int)(item - (long long)t * groups) * a.group;
+    const float* row = a.o + (size_t)t * a.width + g0;
+    const float* gate = a.gate ? a.gate + (size_t)t * a.gate_ld + g0 : nullptr;
+    float4 v[NV], gv[NV];
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int c = (lane + 32 * i) * 4;
+        v[i] = c < a.group ? *reinterpret_cast<const float4*>(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        gv[i] = gate && c < a.group ? *reinterpret_cast<const float4*>(gate + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) ss = fmaf(v[i].x, v[i].x, ss), ss = fmaf(v[i].y, v[i].y, ss), ss = fmaf(v[i].z, v[i].z, ss), ss = fmaf(v[i].w, v[i].w, ss);
+    ss = warp_sum(ss);
+    const float inv = 1.0f / sqrtf(ss / (float)a.group + a.eps);
+    TA* out = y + (size_t)t * a.width + g0;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int c = (lane + 32 * i) * 4;
+        if (c >= a.group) continue;
+        float r[4] = {v[i].x * inv, v[i].y * inv, v[i].z * inv, v[i].w * inv};
+        const float g[4] = {gv[i].x, gv[i].y, gv[i].z, gv[i].w};
+#pragma unroll
+        for (int k = 0; k < 4; k++) {
+            if (a.w) r[k] *= a.w[(g0 + c + k) % a.w_len];
+            if (gate) r[k] *= act_of(g[k], a.gate_act);
+        }
+        if (sizeof(TA) == 4) {
+            *reinterpret_cast<float4*>(out + c) = make_float4(r[0], r[1], r[2], r[3]);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+            *reinterpret_cast<uint2*>(out + c) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+        }
+    }
+}
+
 // w_len: the weight's length, the whole width or a divisor of it (a weight of one group's size is shared by the groups);
 // head: columns per entry of row_scale and skip_w (0 when neither is given)
 extern "C" int illm_group_norm_gate_ex(const float* o, int T, int width, int group, const float* w, int w_len, float eps, const float* gate,
@@ -537,6 +582,20 @@ extern "C" int illm_group_norm_gate_ex(const float* o, int T, int width, int gro
     GroupNormGateArgs a{o, width, group, w, w_len, eps, gate, gate_ld, gate_act, gate_first, row_scale, head, skip_w, skip_x, skip_ld};
     dim3 grid(T, width / group);
     cudaStream_t s = (cudaStream_t)stream;
+    if (!row_scale && !skip_w && !(gate && gate_first) && group <= 512 && group % 4 == 0 && !((uintptr_t)o & 15) && !((uintptr_t)y & 15) &&
+        (!gate || (gate_ld % 4 == 0 && !((uintptr_t)gate & 15))) && (act_dtype == ILLM_BF16 || act_dtype == ILLM_F32)) {
+        const dim3 vgrid((unsigned)(((long long)T * (width / group) + 7) / 8));
+#define ILLM_GNG(NV)                                                                                                                    \
+    do {                                                                                                                                \
+        if (act_dtype == ILLM_BF16) illm_launch((group_norm_gate_vec_kernel<bf16, NV>), vgrid, dim3(256), 0, s, a, (bf16*)y, T);          \
+        else illm_launch((group_norm_gate_vec_kernel<float, NV>), vgrid, dim3(256), 0, s, a, (float*)y, T);                               \
+    } while (0)
+        if (group <= 128) ILLM_GNG(1);
+        else if (group <= 256) ILLM_GNG(2);
+        else ILLM_GNG(4);
+#undef ILLM_GNG
+        return illm_launch_status();
+    }
     if (act_dtype == ILLM_BF16) illm_launch(group_norm_gate_kernel<bf16>, grid, dim3(128), 0, s, a, (bf16*)y);
     else if (act_dtype == ILLM_F32) illm_launch(group_norm_gate_kernel<float>, grid, dim3(128), 0, s, a, (float*)y);
     else return ILLM_ERR_BAD_ARG;

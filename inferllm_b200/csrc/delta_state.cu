@@ -17,6 +17,15 @@
 // 512 key channels) and live in registers for the whole step.  The step's tokens are staged through shared memory in tiles.  The two dot
 // products of a token are added over the L lanes by a fixed tree of shuffles, and a token's arithmetic does not
 // depend on where the step's cut falls, so prompts, portions and single tokens give the same bits.
+//
+// delta_chunk_scan_kernel: the same with one decay per head, eight tokens at a time, for steps where that order of the sums is
+// allowed (the bfloat16 mode).  With S the state before the eight, G_j the product of the decays up to token j and D_ji
+// the product of those behind i up to j,
+//     u_j = beta_j (v_j - G_j S^T k_j - sum_(i<j) D_ji (k_i . k_j) u_i)
+//     o_j = G_j S^T q_j + sum_(i<=j) D_ji (k_i . q_j) u_i
+//     S  <- G_7 S + sum_i D_7i k_i u_i
+// so the sixteen products with S are independent of one another (one round of shuffles for all), and only the short
+// triangular sums follow in order.  The coefficients, which the columns share, are made by delta_chunk_prep_kernel.  float32.
 #include "common.cuh"
 
 #define DL_THREADS 128
@@ -361,6 +370,286 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs p) {
     }
 }
 
+// ---- eight tokens at a time
+
+#define DC 8                       // tokens per chunk
+#define DC_REC (4 * DC + 2 * DC * DC)      // floats per (chunk, head): beta, beta G, G, D_7i, then M[j][i] and P[j][i]
+
+// Chunk c of the step's sequence b has its record at slot cu_q[b] / DC + b + c (distinct for all chunks of a step).
+__device__ __forceinline__ int dc_slot(int first, int b, int c) { return first / DC + b + c; }
+
+// grid (chunks of the longest sequence, query/key heads, sequences), 128 threads: the products k_i . k_j and k_i . q_j of a
+// chunk, then the records of the value heads that share the keys.  Tokens beyond the sequence's end count as k = q = 0,
+// g = 1, beta = 0.
+__global__ void __launch_bounds__(128) delta_chunk_prep_kernel(DeltaArgs p, float* __restrict__ rec) {
+    pdl_grid_sync();
+    extern __shared__ float sm[];            // k [DC][d], q [DC][d]
+    __shared__ float kk[DC][DC], kq[DC][DC];
+    const int c = blockIdx.x, hk = blockIdx.y, b = blockIdx.z;
+    const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, t0 = c * DC;
+    if (t0 >= n) return;
+    const int nt = min(DC, n - t0), d = p.d, nq = p.nkv * d, C = 2 * nq + p.nh * p.dv;
+    float *sk = sm, *sq = sm + DC * d;
+    for (int e = threadIdx.x; e < DC * d; e += 128) {
+        const int j = e / d, i = e - j * d;
+        const float* row = p.qkv + (size_t)(first + t0 + j) * C + (size_t)hk * d + i;
+        sq[e] = j < nt ? row[0] : 0.f;
+        sk[e] = j < nt ? row[nq] : 0.f;
+    }
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int e = warp; e < 2 * DC * DC; e += 4) {
+        const int j = (e / DC) % DC, i = e % DC;
+        const bool with_q = e >= DC * DC;
+        if (i > j || (!with_q && i == j)) continue;          // uniform over the warp
+        const float *a = sk + i * d, *bb = (with_q ? sq : sk) + j * d;
+        float s = 0.f;
+        for (int x = lane; x < d; x += 32) s = fmaf(a[x], bb[x], s);
+        s = warp_sum(s);
+        if (lane == 0) (with_q ? kq : kk)[j][i] = s;
+    }
+    __syncthreads();
+    const int share = p.nh / p.nkv;
+    for (int e = threadIdx.x; e < share * DC; e += 128) {
+        const int h = hk * share + e / DC, j = e % DC;
+        float g[DC];
+#pragma unroll
+        for (int i = 0; i < DC; i++) g[i] = i < nt ? p.g[(size_t)(first + t0 + i) * p.nh + h] : 1.f;
+        const float beta = j < nt ? p.beta[(size_t)(first + t0 + j) * p.nh + h] : 0.f;
+        float G = 1.f, E = 1.f;
+#pragma unroll
+        for (int i = 0; i < DC; i++) {
+            if (i <= j) G *= g[i];
+            if (i > j) E *= g[i];
+        }
+        float* r = rec + ((size_t)dc_slot(first, b, c) * p.nh + h) * DC_REC;
+        r[j] = beta;
+        r[DC + j] = beta * G;
+        r[2 * DC + j] = G;
+        r[3 * DC + j] = E;
+        float D = 1.f;
+#pragma unroll
+        for (int i = DC - 1; i >= 0; i--) {          // D_ji, from i = j down
+            const bool in = i <= j;
+            r[4 * DC + j * DC + i] = i < j ? beta * D * (i + 1 <= j ? g[i + 1 < DC ? i + 1 : DC - 1] : 1.f) * kk[j][i] : 0.f;
+            if (i < j) D *= g[i + 1 < DC ? i + 1 : DC - 1];
+            r[4 * DC + DC * DC + j * DC + i] = in ? D * kq[j][i] : 0.f;
+        }
+    }
+}
+
+__device__ __forceinline__ unsigned long long dl_pack(float lo, float hi) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void dl_unpack(unsigned long long v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ unsigned long long dl_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ unsigned long long dl_mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+// The layout of delta_scan_kernel: grid (column groups, heads, sequences), L lanes per column, a thread's ROWS rows the quads
+// 4 (l + L r) .. + 3, held as pairs for the two-at-a-time float32 instructions.
+template <int L, int ROWS>
+__global__ void __launch_bounds__(DL_THREADS) delta_chunk_scan_kernel(DeltaArgs p, const float* __restrict__ rec) {
+    pdl_grid_sync();
+    extern __shared__ __align__(16) float sm[];
+    constexpr int COLS = DL_THREADS / L, DPAD = ROWS * L, CHUNKS = DL_TILE / DC, Q4 = ROWS / 4;
+    const int b = blockIdx.z, h = blockIdx.y, hk = h / (p.nh / p.nkv);
+    const int d = p.d, dv = p.dv;
+    const int l = threadIdx.x % L, jc = threadIdx.x / L;
+    const int col = blockIdx.x * COLS + jc;
+    const bool live = col < dv;
+    const int first = p.cu_q[b], n = p.cu_q[b + 1] - first;
+    const int nq = p.nkv * d, C = 2 * nq + p.nh * dv;
+    float* S_col = p.state + (size_t)p.slots[b] * p.state_elems + ((size_t)h * dv + (live ? col : 0)) * d;
+    unsigned long long S[ROWS / 2];
+#pragma unroll
+    for (int r = 0; r < ROWS / 2; r++) {
+        const int i = 4 * (l + L * (r >> 1)) + 2 * (r & 1);
+        S[r] = dl_pack(live && i < d ? S_col[i] : 0.f, live && i + 1 < d ? S_col[i + 1] : 0.f);
+    }
+    // two buffers of a tile: q, k [tile, DPAD], the chunks' records, v [tile, COLS]
+    constexpr int BUF = DL_TILE * (2 * DPAD + COLS) + CHUNKS * DC_REC;
+    const int j0 = blockIdx.x * COLS;
+    const float* __restrict__ qkv = p.qkv;
+    float* __restrict__ out = p.out;
+    if (d < DPAD)
+        for (int e = threadIdx.x; e < 2 * 2 * DL_TILE * (DPAD - d); e += DL_THREADS) {
+            const int bb = e / (2 * DL_TILE * (DPAD - d)), r = e % (2 * DL_TILE * (DPAD - d));
+            sm[bb * BUF + (r / (DPAD - d)) * DPAD + d + r % (DPAD - d)] = 0.f;
+        }
+    const bool wide = (d & 3) == 0 && (C & 3) == 0;
+    auto stage = [&](int buf, int t0) {
+        float* sq = sm + buf * BUF;
+        float* sk = sq + DL_TILE * DPAD;
+        float* sr = sk + DL_TILE * DPAD;
+        float* sv = sr + CHUNKS * DC_REC;
+        const int nt = min(DL_TILE, n - t0), nc = (nt + DC - 1) / DC, np = nc * DC;        // np: with the last chunk's missing tokens
+        if (wide) {
+            const int per_row = d >> 2;
+            for (int e = threadIdx.x; e < np * per_row; e += DL_THREADS) {
+                const int tt = e / per_row, i = (e - tt * per_row) * 4;
+                if (tt < nt) {
+                    const float* row = qkv + (size_t)(first + t0 + tt) * C + (size_t)hk * d + i;
+                    dl_cp16(sq + tt * DPAD + i, row);
+                    dl_cp16(sk + tt * DPAD + i, row + nq);
+                } else {
+                    *reinterpret_cast<float4*>(sq + tt * DPAD + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+                    *reinterpret_cast<float4*>(sk + tt * DPAD + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+                }
+            }
+        } else {
+            for (int e = threadIdx.x; e < np * d; e += DL_THREADS) {
+                const int tt = e / d, i = e - tt * d;
+                if (tt < nt) {
+                    const float* row = qkv + (size_t)(first + t0 + tt) * C + (size_t)hk * d + i;
+                    dl_cp4(sq + tt * DPAD + i, row);
+                    dl_cp4(sk + tt * DPAD + i, row + nq);
+                } else {
+                    sq[tt * DPAD + i] = 0.f;
+                    sk[tt * DPAD + i] = 0.f;
+                }
+            }
+        }
+        for (int e = threadIdx.x; e < nc * (DC_REC / 4); e += DL_THREADS) {
+            const int cc = e / (DC_REC / 4), x = (e - cc * (DC_REC / 4)) * 4;
+            dl_cp16(sr + cc * DC_REC + x, rec + ((size_t)dc_slot(first, b, t0 / DC + cc) * p.nh + h) * DC_REC + x);
+        }
+        for (int e = threadIdx.x; e < np * COLS; e += DL_THREADS) {
+            const int tt = e / COLS, c = e - tt * COLS;
+            if (tt < nt && j0 + c < dv) dl_cp4(sv + e, qkv + (size_t)(first + t0 + tt) * C + 2 * nq + (size_t)h * dv + j0 + c);
+            else sv[e] = 0.f;
+        }
+    };
+    if (n > 0) stage(0, 0);
+    asm volatile("cp.async.commit_group;\n" ::);
+    for (int t0 = 0, it = 0; t0 < n; t0 += DL_TILE, it++) {
+        const int nt = min(DL_TILE, n - t0);
+        if (t0 + DL_TILE < n) stage((it + 1) & 1, t0 + DL_TILE);
+        asm volatile("cp.async.commit_group;\n" ::);
+        asm volatile("cp.async.wait_group 1;\n" ::);
+        __syncthreads();
+        const float* sq = sm + (it & 1) * BUF;
+        const float* sk = sq + DL_TILE * DPAD;
+        const float* sr = sk + DL_TILE * DPAD;
+        const float* sv = sr + CHUNKS * DC_REC;
+#pragma unroll 1
+        for (int c0 = 0; c0 < nt; c0 += DC) {
+            const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(sk + c0 * DPAD) + l;
+            const ulonglong2* q2 = reinterpret_cast<const ulonglong2*>(sq + c0 * DPAD) + l;
+            const float4* r4 = reinterpret_cast<const float4*>(sr + (c0 / DC) * DC_REC);
+            // S^T k_j and S^T q_j of all eight tokens
+            unsigned long long ak[DC], aq[DC];
+#pragma unroll
+            for (int j = 0; j < DC; j++) ak[j] = aq[j] = 0ull;
+#pragma unroll
+            for (int r = 0; r < Q4; r++) {
+#pragma unroll
+                for (int j = 0; j < DC; j++) {
+                    const ulonglong2 kv = k2[j * (DPAD / 4) + L * r], qv = q2[j * (DPAD / 4) + L * r];
+                    ak[j] = dl_fma2(kv.y, S[2 * r + 1], dl_fma2(kv.x, S[2 * r], ak[j]));
+                    aq[j] = dl_fma2(qv.y, S[2 * r + 1], dl_fma2(qv.x, S[2 * r], aq[j]));
+                }
+            }
+            float A[DC], O[DC];
+#pragma unroll
+            for (int j = 0; j < DC; j++) {
+                float lo, hi;
+                dl_unpack(ak[j], lo, hi);
+                A[j] = lo + hi;
+                dl_unpack(aq[j], lo, hi);
+                O[j] = lo + hi;
+            }
+#pragma unroll
+            for (int o = L / 2; o > 0; o >>= 1)
+#pragma unroll
+                for (int j = 0; j < DC; j++) {
+                    A[j] += __shfl_xor_sync(0xffffffffu, A[j], o);
+                    O[j] += __shfl_xor_sync(0xffffffffu, O[j], o);
+                }
+            // the triangular sums
+            float u[DC];
+            float bv[DC], bg[DC], gg[DC];
+#pragma unroll
+            for (int x = 0; x < DC / 4; x++) {
+                const float4 t1 = r4[x], t2 = r4[DC / 4 + x], t3 = r4[2 * (DC / 4) + x];
+                bv[4 * x] = t1.x, bv[4 * x + 1] = t1.y, bv[4 * x + 2] = t1.z, bv[4 * x + 3] = t1.w;
+                bg[4 * x] = t2.x, bg[4 * x + 1] = t2.y, bg[4 * x + 2] = t2.z, bg[4 * x + 3] = t2.w;
+                gg[4 * x] = t3.x, gg[4 * x + 1] = t3.y, gg[4 * x + 2] = t3.z, gg[4 * x + 3] = t3.w;
+            }
+#pragma unroll
+            for (int j = 0; j < DC; j++) {
+                float m[DC], pr[DC];
+#pragma unroll
+                for (int x = 0; x < DC / 4; x++) {
+                    const float4 t1 = r4[DC + j * (DC / 4) + x], t2 = r4[DC + DC * DC / 4 + j * (DC / 4) + x];
+                    m[4 * x] = t1.x, m[4 * x + 1] = t1.y, m[4 * x + 2] = t1.z, m[4 * x + 3] = t1.w;
+                    pr[4 * x] = t2.x, pr[4 * x + 1] = t2.y, pr[4 * x + 2] = t2.z, pr[4 * x + 3] = t2.w;
+                }
+                float v = fmaf(-bg[j], A[j], bv[j] * sv[(c0 + j) * COLS + jc]);
+#pragma unroll
+                for (int i = 0; i < j; i++) v = fmaf(-m[i], u[i], v);
+                u[j] = v;
+                float o = gg[j] * O[j];
+#pragma unroll
+                for (int i = 0; i <= j; i++) o = fmaf(pr[i], u[i], o);
+                O[j] = o;
+            }
+#pragma unroll
+            for (int j = 0; j < DC; j++)
+                if (live && l == j % L && c0 + j < nt) out[(size_t)(first + t0 + c0 + j) * p.nh * dv + (size_t)h * dv + col] = O[j];
+            // the state behind the chunk; long columns read the keys a second time instead of keeping them in registers
+            if (ROWS > 8) asm volatile("" ::: "memory");
+            const unsigned long long g2 = dl_pack(gg[DC - 1], gg[DC - 1]);
+            unsigned long long w2[DC];
+#pragma unroll
+            for (int x = 0; x < DC / 4; x++) {
+                const float4 t1 = r4[3 * (DC / 4) + x];
+                const float e4[4] = {t1.x, t1.y, t1.z, t1.w};
+#pragma unroll
+                for (int y = 0; y < 4; y++) {
+                    const float w = e4[y] * u[4 * x + y];
+                    w2[4 * x + y] = dl_pack(w, w);
+                }
+            }
+#pragma unroll
+            for (int r = 0; r < Q4; r++) {
+                unsigned long long s0 = dl_mul2(S[2 * r], g2), s1 = dl_mul2(S[2 * r + 1], g2);
+#pragma unroll
+                for (int j = 0; j < DC; j++) {
+                    const ulonglong2 kv = k2[j * (DPAD / 4) + L * r];
+                    s0 = dl_fma2(kv.x, w2[j], s0);
+                    s1 = dl_fma2(kv.y, w2[j], s1);
+                }
+                S[2 * r] = s0;
+                S[2 * r + 1] = s1;
+            }
+        }
+        __syncthreads();          // the tile after the next one goes into this buffer
+    }
+    if (live) {
+#pragma unroll
+        for (int r = 0; r < ROWS / 2; r++) {
+            const int i = 4 * (l + L * (r >> 1)) + 2 * (r & 1);
+            float lo, hi;
+            dl_unpack(S[r], lo, hi);
+            if (i < d) S_col[i] = lo;
+            if (i + 1 < d) S_col[i + 1] = hi;
+        }
+    }
+}
+
+// floats of scratch for the chunks' records of a step
+extern "C" long long illm_delta_chunk_scratch(int T, int B, int nh) { return ((long long)T / DC + B + 1) * nh * DC_REC; }
+
 extern "C" int illm_delta_rule_supported(int d, int dv, int taps) { return d >= 1 && d <= 16 * DL_ROWS && dv >= 1 && taps >= 1 && taps <= 64; }
 
 template <int L, int ROWS, bool HEAD>
@@ -386,7 +675,23 @@ static void launch_scan_as(const DeltaArgs& p, int B, int n_sms, cudaStream_t s)
 }
 
 template <int L, int ROWS>
-static void launch_scan(const DeltaArgs& p, int B, int n_sms, cudaStream_t s) {
+static void launch_scan(const DeltaArgs& p, int B, int n_sms, cudaStream_t s, const float* rec) {
+    if constexpr (ROWS <= 16) if (rec) {        // (eight tokens at a time with 32 rows per thread do not fit the registers)
+        constexpr int COLS = DL_THREADS / L;
+        size_t smem = (size_t)2 * (DL_TILE * (2 * ROWS * L + COLS) + (DL_TILE / DC) * DC_REC) * sizeof(float);
+        const long long blocks = (long long)((p.dv + COLS - 1) / COLS) * p.nh * B, per_sm = (blocks + n_sms - 1) / n_sms;
+        if (per_sm < 5) {          // as for the scan above: an even spread over the SMs
+            const size_t spread = (size_t)(220 * 1024) / (size_t)per_sm - 2048;
+            smem = smem > spread ? smem : (spread < (size_t)200 * 1024 ? spread : (size_t)200 * 1024);
+        }
+        static bool raised = false;
+        if (!raised) {
+            cudaFuncSetAttribute(delta_chunk_scan_kernel<L, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+            raised = true;
+        }
+        illm_launch((delta_chunk_scan_kernel<L, ROWS>), dim3((p.dv + COLS - 1) / COLS, p.nh, B), dim3(DL_THREADS), smem, s, p, rec);
+        return;
+    }
     if (p.head_decay) launch_scan_as<L, ROWS, true>(p, B, n_sms, s);
     else launch_scan_as<L, ROWS, false>(p, B, n_sms, s);
 }
@@ -396,7 +701,7 @@ static void launch_scan(const DeltaArgs& p, int B, int n_sms, cudaStream_t s) {
 // (one prompt of 2,048 tokens, 8 heads of 128 x 128: 0.78 / 0.62 ms with 32 / 16 rows; with two blocks on an SM the
 // shorter rows gain nothing).  The choice does not depend on the batch, or a row's bits would.
 template <int L>
-static void launch_scan_for(const DeltaArgs& p, int B, cudaStream_t s) {
+static void launch_scan_for(const DeltaArgs& p, int B, cudaStream_t s, const float* rec) {
     static int n_sms = 0;
     if (!n_sms) {
         int dev = 0;
@@ -406,22 +711,24 @@ static void launch_scan_for(const DeltaArgs& p, int B, cudaStream_t s) {
     }
     constexpr int L2 = 2 * L <= 32 ? 2 * L : L, L4 = 4 * L <= 32 ? 4 * L : L2;
     auto blocks_of = [&](int lanes) { return (long long)((p.dv + DL_THREADS / lanes - 1) / (DL_THREADS / lanes)) * p.nh; };
-    if (L4 != L2 && blocks_of(L4) <= n_sms) launch_scan<L4, 8>(p, B, n_sms, s);
-    else if (L2 != L && blocks_of(L2) <= n_sms) launch_scan<L2, 16>(p, B, n_sms, s);
-    else launch_scan<L, 32>(p, B, n_sms, s);
+    if (L4 != L2 && blocks_of(L4) <= n_sms) launch_scan<L4, 8>(p, B, n_sms, s, rec);
+    else if (L2 != L && (rec || blocks_of(L2) <= n_sms)) launch_scan<L2, 16>(p, B, n_sms, s, rec);
+    else launch_scan<L, 32>(p, B, n_sms, s, rec);
 }
 
 // x: [T, ld] float32 with q at q_off (nkv * d columns), k at k_off, v at v_off (nh * dv), beta's logits at b_off (nh).
 // state: float32 [slots, state_elems], state_elems >= nh * d * dv + (taps - 1) * (2 nkv d + nh dv).
 // a: the decay projection, rows a_ld apart: nh * d columns, or with head_decay nh.
+// chunks (head_decay only; nullptr: token by token): illm_delta_chunk_scratch floats, the scan then takes eight tokens at a
+// time; max_q the most tokens of one sequence.
 // Scratch qkv [T, 2 nkv d + nh dv], g [T, nh d] (head_decay: [T, nh]), beta [T, nh]; out [T, nh dv].
 extern "C" int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_off, int v_off, int b_off, const float* a, int a_ld, int head_decay, int nh, int nkv, int d,
                                int dv, int taps, const float* conv_q, const float* conv_k, const float* conv_v, const float* a_log,
                                const float* dt_bias, float q_scale, float* state, long long state_elems, const int* slots, const int* cu_q,
                                const int* token_pos, const int* token_seq, const int* seq_lens, float* qkv, float* g, float* beta, float* out,
-                               int B, void* stream) {
+                               int B, int max_q, float* chunks, void* stream) {
     if (T <= 0 || B <= 0) return 0;
-    if (!illm_delta_rule_supported(d, dv, taps) || nkv <= 0 || nh % nkv || a_ld < (head_decay ? nh : nh * d)) return ILLM_ERR_BAD_ARG;
+    if (!illm_delta_rule_supported(d, dv, taps) || nkv <= 0 || nh % nkv || a_ld < (head_decay ? nh : nh * d) || (chunks && (!head_decay || max_q <= 0 || nkv > 65535 || B > 65535))) return ILLM_ERR_BAD_ARG;
     const long long C = 2LL * nkv * d + (long long)nh * dv;
     if (state_elems < (long long)nh * d * dv + (taps - 1) * C) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
@@ -442,10 +749,14 @@ extern "C" int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_o
     else if (taps == 4) illm_launch(delta_prep_kernel<4>, pgrid, dim3(256), 0, s, p);
     else illm_launch(delta_prep_kernel<0>, pgrid, dim3(256), 0, s, p);
     if (taps > 1) illm_launch(conv_state_kernel, dim3((unsigned)((C + 127) / 128), B), dim3(128), 0, s, p);
-    if (d <= 32) launch_scan_for<1>(p, B, s);
-    else if (d <= 64) launch_scan_for<2>(p, B, s);
-    else if (d <= 128) launch_scan_for<4>(p, B, s);
-    else if (d <= 256) launch_scan_for<8>(p, B, s);
-    else launch_scan_for<16>(p, B, s);
+    if (chunks) {
+        const size_t smem = (size_t)2 * DC * d * sizeof(float);
+        illm_launch(delta_chunk_prep_kernel, dim3((max_q + DC - 1) / DC, nkv, B), dim3(128), smem, s, p, chunks);
+    }
+    if (d <= 32) launch_scan_for<1>(p, B, s, chunks);
+    else if (d <= 64) launch_scan_for<2>(p, B, s, chunks);
+    else if (d <= 128) launch_scan_for<4>(p, B, s, chunks);
+    else if (d <= 256) launch_scan_for<8>(p, B, s, chunks);
+    else launch_scan_for<16>(p, B, s, chunks);
     return illm_launch_status();
 }

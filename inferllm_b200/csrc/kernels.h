@@ -54,7 +54,8 @@ int illm_bigram_embedding(const int* ids, const int* token_pos, const int* token
 
 // delta_state.cu
 int illm_delta_rule_supported(int d, int dv, int taps);
-int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_off, int v_off, int b_off, const float* a, int a_ld, int head_decay, int nh, int nkv, int d, int dv, int taps, const float* conv_q, const float* conv_k, const float* conv_v, const float* a_log, const float* dt_bias, float q_scale, float* state, long long state_elems, const int* slots, const int* cu_q, const int* token_pos, const int* token_seq, const int* seq_lens, float* qkv, float* g, float* beta, float* out, int B, void* stream);
+long long illm_delta_chunk_scratch(int T, int B, int nh);
+int illm_delta_rule(const float* x, int T, int ld, int q_off, int k_off, int v_off, int b_off, const float* a, int a_ld, int head_decay, int nh, int nkv, int d, int dv, int taps, const float* conv_q, const float* conv_k, const float* conv_v, const float* a_log, const float* dt_bias, float q_scale, float* state, long long state_elems, const int* slots, const int* cu_q, const int* token_pos, const int* token_seq, const int* seq_lens, float* qkv, float* g, float* beta, float* out, int B, int max_q, float* chunks, void* stream);
 
 // gated_state.cu
 int illm_mlstm_gates(const float* x, int T, int ld, int q_off, int k_off, int i_off, int f_off, const float* i_bias, const float* f_bias, float cap, float q_scale, int nh, int d, float* state, long long state_stride, long long n_off, long long m_off, const int* slots, const int* cu_q, float* ga, float* gb, float* scale, int B, void* stream);

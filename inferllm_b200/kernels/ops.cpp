@@ -940,12 +940,14 @@ Mat delta_rule(Device& dev, const Mat& x, const Mat* a, const DeltaRule& p, cons
         throw KernelError("delta_rule: the state entry does not have this layer's size");
     Mat qkv = new_mat_exact(dev, T, C, DType::F32), g = new_mat_exact(dev, T, decays, DType::F32), beta = new_mat_exact(dev, T, p.n_heads, DType::F32);
     Mat out = new_mat_exact(dev, T, (long long)p.n_heads * p.v_head_dim, DType::F32);
+    const bool chunked = p.head_decay && !p.in_order && ctx.max_q >= kDeltaChunkMinTokens;
+    float* chunks = chunked ? dev.alloc_n<float>((size_t)illm_delta_chunk_scratch((int)T, ctx.B, p.n_heads)) : nullptr;
     check_kernel(illm_delta_rule((const float*)x.p, (int)T, (int)x.cols, p.q_off, p.k_off, p.v_off, p.b_off,
                                  p.head_decay ? (const float*)x.p + p.a_off : (const float*)a->p, p.head_decay ? (int)x.cols : (int)decays,
                                  p.head_decay ? 1 : 0, p.n_heads,
                                  p.n_kv_heads, p.head_dim, p.v_head_dim, p.taps, p.conv_q, p.conv_k, p.conv_v, p.a_log, p.dt_bias, p.q_scale,
                                  (float*)st.state, st.elements, st.slots, ctx.cu_q, ctx.token_pos, ctx.token_seq, ctx.seq_lens, (float*)qkv.p,
-                                 (float*)g.p, (float*)beta.p, (float*)out.p, ctx.B, dev.stream()),
+                                 (float*)g.p, (float*)beta.p, (float*)out.p, ctx.B, ctx.max_q, chunks, dev.stream()),
                  "delta_rule");
     return out;
 }

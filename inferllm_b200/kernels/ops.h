@@ -356,11 +356,15 @@ struct DeltaRule {
     int q_off = 0, k_off = 0, v_off = 0, b_off = 0;
     int n_heads = 0, n_kv_heads = 0, head_dim = 0, v_head_dim = 0, taps = 1;
     bool head_decay = false;
+    // head_decay: false allows steps of several tokens to take eight tokens at a time (the order of the sums then differs from
+    // token by token); true: always token by token, bit for bit
+    bool in_order = true;
     int a_off = 0;                                                           // head_decay: the decay projection's columns
     const float *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr;     // float32 [channels, taps]
     const float *a_log = nullptr, *dt_bias = nullptr;                        // float32 [heads], [heads * head_dim] or [heads]
     float q_scale = 1.f;
 };
+constexpr int kDeltaChunkMinTokens = 16;      // the most tokens of a sequence in a step from which the scan takes eight at a time
 long long delta_rule_state_elements(int n_heads, int n_kv_heads, int head_dim, int v_head_dim, int taps);
 bool delta_rule_supported(int head_dim, int v_head_dim, int taps);
 Mat delta_rule(Device& dev, const Mat& x_f32, const Mat* a_f32, const DeltaRule& p, const StepView& ctx, const StateView& st);

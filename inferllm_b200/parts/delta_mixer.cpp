@@ -104,9 +104,10 @@ struct DeltaMixer : Mixer {
         return d;
     }
     long long off_v() const { return 2 * qk_rows(); }
-    long long off_b() const { return off_v() + v_rows(); }
-    long long off_a() const { return off_b() + n_heads; }
-    long long off_g() const { return off_a() + a_cols(); }
+    // rows of the packed matrix: q, k, v, the gate, then the decay and the write strengths, and zero rows up to a multiple of 8
+    long long off_g() const { return off_v() + v_rows(); }
+    long long off_a() const { return off_g() + gate_cols(); }
+    long long off_b() const { return off_a() + a_cols(); }
     void load(TensorSource& src) override {
         auto rank_of = [&](const char* down, const char* up) {
             const long long r = src.shape(names.at(down)).at(0);
@@ -116,10 +117,11 @@ struct DeltaMixer : Mixer {
         };
         if (!head_decay) a_rank = rank_of("a_down", "a_up");
         if (!full_gate) g_rank = rank_of("g_down", "g_up");
-        const long long all = off_g() + gate_cols();
+        const long long used = off_b() + n_heads, all = (used + 7) / 8 * 8;
         const size_t es = dtype_size(rt->dtype);
         w_buf = DeviceBuffer(rt->dev, (size_t)all * hidden * es, "the packed projections of a delta-rule layer");
         w_in = Mat{w_buf.get(), all, hidden, rt->dtype, all};
+        check_cuda(cudaMemsetAsync(w_in.p, 0, w_buf.bytes(), rt->dev->stream()), "clearing the packed projections");
         char* p = (char*)w_in.p;
         auto at = [&](long long row) { return p + (size_t)row * hidden * es; };
         src.fetch_into(names.at("q"), at(0), rt->dtype);
@@ -159,6 +161,7 @@ struct DeltaMixer : Mixer {
         p.v_head_dim = v_head_dim;
         p.taps = taps;
         p.head_decay = head_decay;
+        p.in_order = rt->is_f32();
         p.a_off = (int)off_a();
         p.conv_q = (const float*)conv_q.m.p;
         p.conv_k = (const float*)conv_k.m.p;

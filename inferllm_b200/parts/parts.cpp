@@ -588,8 +588,7 @@ struct Attention : Mixer {
         if (unit_sink) {       // one more term exp(0) in every head's denominator
             sinks.buf = DeviceBuffer(rt->dev, (size_t)n_heads * sizeof(float), "the attention sinks");
             sinks.m = Mat{sinks.buf.get(), 1, n_heads, DType::F32, 1};
-            rt->dev->synchronize();
-            check_cuda(cudaMemset(sinks.m.p, 0, (size_t)n_heads * sizeof(float)), "clearing the attention sinks");
+            check_cuda(cudaMemsetAsync(sinks.m.p, 0, (size_t)n_heads * sizeof(float), rt->dev->stream()), "clearing the attention sinks");
         }
         if (mixes_values) v_mix = fetch_owned(rt, src, names.at("v_mix"), DType::F32, "a value-mixing factor");
         if (log_distance) {
