@@ -285,11 +285,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     // blocks (the causal mask gives tile t of a prompt t + 1 blocks of 128 keys) start first, on all
     // heads, and the short ones fill the SMs as those finish.  (Two tiles per block, the x-th from the
     // end and the x-th from the start, which gives all blocks equal work, was slower at every prompt
-    // length: 52.5 against 50.2 us at 2,048 tokens of 32 heads, 138 against 101 us at 3,072.)
+    // length: 52.5 against 50.2 us at 2,048 tokens of 32 heads, 138 against 101 us at 3,072.)  With chunks the work of a
+    // tile grows with its place inside its chunk, and the tiles of all chunks are taken in the order of that place.
     const int b = blockIdx.z, h = blockIdx.x;
     const int q0 = cu_q[b], qlen = cu_q[b + 1] - q0;
     const int n_tiles = (qlen + FT_BM - 1) / FT_BM;
-    const int tile = n_tiles - 1 - (int)blockIdx.y;           // < 0: this sequence is shorter than the longest
+    int tile = n_tiles - 1 - (int)blockIdx.y;                 // < 0: this sequence is shorter than the longest
+    if (span < 0 && tile >= 0) {
+        const int per = (-span + FT_BM - 1) / FT_BM, chunks = (n_tiles + per - 1) / per;      // tiles per chunk, chunks begun
+        if (chunks > 1) {
+            const int rest = n_tiles - (chunks - 1) * per;    // tiles of the last one
+            const int whole = (per - rest) * (chunks - 1);    // tiles at the places that the last one does not reach
+            const int y = (int)blockIdx.y;
+            if (y < whole) tile = (y % (chunks - 1)) * per + per - 1 - y / (chunks - 1);
+            else tile = ((y - whole) % chunks) * per + rest - 1 - (y - whole) / chunks;
+        }
+    }
     const int row0 = tile * FT_BM;
     const int total = seq_lens[b], past = total - qlen;
     const int hk = h / (nh / nkv);
@@ -384,7 +395,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int r = threadIdx.x & 127;
         const unsigned lane_addr = tmem + ((unsigned)(warp * 32) << 16);
         const int pos = (r < rows) ? first_pos + r : last_pos;
-        const int lo_pos = first_visible(pos, span);
+        const int lo_pos = first_visible(pos, span), lo_last = has_rows ? first_visible(last_pos, span) : 0;
         float m_ref = -INFINITY, l_run = 0.f;
         bool alive = has_rows;
         for (int i = 0; i < n_blocks && alive; i++) {
@@ -421,7 +432,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     }
                 }
             }
-            const bool need_mask = (key0 + FT_BN - 1 > first_pos) || (span != 0);
+            const bool need_mask = key0 + FT_BN - 1 > first_pos || key0 < lo_last;
             if (need_mask) {
 #pragma unroll
                 for (int c = 0; c < FT_BN; c++) {
@@ -543,6 +554,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             }
             if (gate && !gate_wide && r < rows) inv *= 1.0f / (1.0f + expf(-gate[(size_t)(q0 + row0 + r) * gate_stride + h]));
             bf16* dst = out + ((size_t)(q0 + row0 + r) * nh + h) * D;
+            // a gate per channel: a warp brings its 32 rows, whole rows at a time, into the shared memory that the tiles of
+            // Q and K no longer need (every product has been done), from where a thread reads its own row
+            constexpr int G_ROW = D * 4 + 16;
+            const unsigned g_s = base + warp * 32 * G_ROW;
+            static_assert(4 * 32 * G_ROW <= (int)(Q_TILE + FT_KSTAGES * KV_BYTES), "the gate rows must fit the tiles of Q and K");
+            if (WIDE_P && gate && gate_wide == 2) {
+#pragma unroll 8
+                for (int rr = 0; rr < 32; rr++) {
+                    const int row = warp * 32 + rr;
+                    if (row < rows && lane * 4 < D) {
+                        const float4 v = *reinterpret_cast<const float4*>(gate + (size_t)(q0 + row0 + row) * gate_stride + (size_t)h * D + lane * 4);
+                        asm volatile("st.shared.v4.f32 [%0], {%1,%2,%3,%4};" ::"r"(g_s + rr * G_ROW + lane * 16), "f"(v.x), "f"(v.y), "f"(v.z), "f"(v.w) : "memory");
+                    }
+                }
+                __syncwarp();
+            }
 #pragma unroll 1
             for (int c0 = 0; c0 < D; c0 += 32) {
                 unsigned orr[32];
@@ -554,11 +581,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                         float f[8];
 #pragma unroll
                         for (int e = 0; e < 8; e++) f[e] = __uint_as_float(orr[c + e]) * inv;
-                        if (gate && gate_wide) {
+                        if (WIDE_P && gate && gate_wide) {
                             const float* gr = gate + (size_t)(q0 + row0 + r) * gate_stride + (size_t)h * D + c0 + c;
                             float g8[8];
                             if (gate_wide == 2) {          // rows of whole 16-byte pieces
-                                load8(gr, g8);
+                                const unsigned at = g_s + lane * G_ROW + (c0 + c) * 4;
+                                asm volatile("ld.shared.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(g8[0]), "=f"(g8[1]), "=f"(g8[2]), "=f"(g8[3]) : "r"(at));
+                                asm volatile("ld.shared.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(g8[4]), "=f"(g8[5]), "=f"(g8[6]), "=f"(g8[7]) : "r"(at + 16));
                             } else {
 #pragma unroll
                                 for (int e = 0; e < 8; e++) g8[e] = gr[e];
@@ -636,7 +665,8 @@ static int ft_launch(const void* q, int q_stride, int T, const void* kc, const v
 }
 
 // q: the packed projection [T, q_stride] whose first nh*d columns are the query heads;
-// kc, vc: one cache entry [n_pages, nkv, page_size, d].  wide_p, sinks, gate, gate_wide, softcap (0: none; needs wide_p): see
+// kc, vc: one cache entry [n_pages, nkv, page_size, d].  wide_p, sinks, gate, gate_wide, softcap (0: none; the last two need
+// wide_p): see
 // the kernel; span: see first_visible.
 extern "C" int illm_attention_prefill_tc_ex(const void* q, int q_stride, int T, const void* kc, const void* vc,
                                             long long n_pages, const int* block_table, int max_pages,
@@ -649,7 +679,7 @@ extern "C" int illm_attention_prefill_tc_ex(const void* q, int q_stride, int T, 
         ((uintptr_t)q & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15))
         return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
-    if (softcap > 0.f && !wide_p) return ILLM_ERR_BAD_ARG;
+    if ((softcap > 0.f || (gate && gate_wide)) && !wide_p) return ILLM_ERR_BAD_ARG;
     if (gate && gate_wide) gate_wide = gate_stride % 4 == 0 && !((uintptr_t)gate & 15) ? 2 : 1;
 #define FT_CASE(DD, WW, CC)                                                                                                   \
     if (d == DD && (wide_p != 0) == WW && (softcap > 0.f) == CC)                                                              \
