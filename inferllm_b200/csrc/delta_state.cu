@@ -487,36 +487,40 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_scan_kernel(DeltaArgs 
             sm[bb * BUF + (r / (DPAD - d)) * DPAD + d + r % (DPAD - d)] = 0.f;
         }
     const bool wide = (d & 3) == 0 && (C & 3) == 0;
+    // a thread's first piece of a tile's rows and the step to its next one, so that staging divides nothing
+    const int per_row = wide ? d >> 2 : d, piece = wide ? 4 : 1;
+    const int tt_first = threadIdx.x / per_row, i_first = threadIdx.x % per_row, tt_step = DL_THREADS / per_row, i_step = DL_THREADS % per_row;
     auto stage = [&](int buf, int t0) {
         float* sq = sm + buf * BUF;
         float* sk = sq + DL_TILE * DPAD;
         float* sr = sk + DL_TILE * DPAD;
         float* sv = sr + CHUNKS * DC_REC;
         const int nt = min(DL_TILE, n - t0), nc = (nt + DC - 1) / DC, np = nc * DC;        // np: with the last chunk's missing tokens
-        if (wide) {
-            const int per_row = d >> 2;
-            for (int e = threadIdx.x; e < np * per_row; e += DL_THREADS) {
-                const int tt = e / per_row, i = (e - tt * per_row) * 4;
+        const float* base = qkv + (size_t)(first + t0) * C + (size_t)hk * d;
+        for (int tt = tt_first, ip = i_first; tt < np;) {
+            const int i = ip * piece;
+            float *dq = sq + tt * DPAD + i, *dk = sk + tt * DPAD + i;
+            const float* row = base + (size_t)tt * C + i;
+            if (wide) {
                 if (tt < nt) {
-                    const float* row = qkv + (size_t)(first + t0 + tt) * C + (size_t)hk * d + i;
-                    dl_cp16(sq + tt * DPAD + i, row);
-                    dl_cp16(sk + tt * DPAD + i, row + nq);
+                    dl_cp16(dq, row);
+                    dl_cp16(dk, row + nq);
                 } else {
-                    *reinterpret_cast<float4*>(sq + tt * DPAD + i) = make_float4(0.f, 0.f, 0.f, 0.f);
-                    *reinterpret_cast<float4*>(sk + tt * DPAD + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+                    *reinterpret_cast<float4*>(dq) = make_float4(0.f, 0.f, 0.f, 0.f);
+                    *reinterpret_cast<float4*>(dk) = make_float4(0.f, 0.f, 0.f, 0.f);
                 }
+            } else if (tt < nt) {
+                dl_cp4(dq, row);
+                dl_cp4(dk, row + nq);
+            } else {
+                *dq = 0.f;
+                *dk = 0.f;
             }
-        } else {
-            for (int e = threadIdx.x; e < np * d; e += DL_THREADS) {
-                const int tt = e / d, i = e - tt * d;
-                if (tt < nt) {
-                    const float* row = qkv + (size_t)(first + t0 + tt) * C + (size_t)hk * d + i;
-                    dl_cp4(sq + tt * DPAD + i, row);
-                    dl_cp4(sk + tt * DPAD + i, row + nq);
-                } else {
-                    sq[tt * DPAD + i] = 0.f;
-                    sk[tt * DPAD + i] = 0.f;
-                }
+            tt += tt_step;
+            ip += i_step;
+            if (ip >= per_row) {
+                ip -= per_row;
+                tt++;
             }
         }
         for (int e = threadIdx.x; e < nc * (DC_REC / 4); e += DL_THREADS) {
@@ -603,9 +607,15 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_scan_kernel(DeltaArgs 
                 for (int i = 0; i <= j; i++) o = fmaf(pr[i], u[i], o);
                 O[j] = o;
             }
+            // every lane of a column has all of them: lane l stores token j0 + l
+            constexpr int LS = L < DC ? L : DC;
 #pragma unroll
-            for (int j = 0; j < DC; j++)
-                if (live && l == j % L && c0 + j < nt) out[(size_t)(first + t0 + c0 + j) * p.nh * dv + (size_t)h * dv + col] = O[j];
+            for (int j0 = 0; j0 < DC; j0 += LS) {
+                float o = O[j0];
+#pragma unroll
+                for (int k = 1; k < LS; k++) o = l == k ? O[j0 + k] : o;
+                if (live && l < LS && c0 + j0 + l < nt) out[(size_t)(first + t0 + c0 + j0 + l) * p.nh * dv + (size_t)h * dv + col] = o;
+            }
             // the state behind the chunk; long columns read the keys a second time instead of keeping them in registers
             if (ROWS > 8) asm volatile("" ::: "memory");
             const unsigned long long g2 = dl_pack(gg[DC - 1], gg[DC - 1]);
