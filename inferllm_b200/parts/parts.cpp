@@ -409,8 +409,8 @@ struct NoPosition : PositionEncoding {
 // 1 + coef ln(floor((p + 1) / every) + 1), behind the bias) and `o_bias` (a bias on the output projection).
 //
 // A fourth: `chunk` c (instead of a window: a query sees the earlier positions of its own chunk of c, counted from the
-// sequence's start), `softcap` (the scaled scores s become softcap * tanh(s / softcap)), `unit_sink` (one is added to the
-// softmax denominator: a sink whose score is 0), `out_gate` = "sigmoid" also without values = keys, and `value_mix`: "first"
+// sequence's start), `softcap` (the scaled scores s become softcap * tanh(s / softcap)), `unit_sink` (every head's softmax
+// denominator gets one more term exp(0) without a value), `out_gate` = "sigmoid" also without values = keys, and `value_mix`: "first"
 // (the layer keeps its values for later layers of the step) or "mix" (v <- (1 - lambda) v + lambda v_first with the kept
 // values of the same tokens and lambda one number, tensor "v_mix"; the mixed values are what is cached).  Both declare
 // the tensor.
