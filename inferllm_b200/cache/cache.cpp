@@ -24,6 +24,15 @@ CacheRequest CacheRequest::paged_keys_only(int n_kv_heads, int head_dim, int win
     r.keys_only = true;
     return r;
 }
+CacheRequest CacheRequest::reaching(int window2, int chunk2) const {
+    CacheRequest r = *this;
+    if (window == window2 && chunk == chunk2) return r;
+    // a chunk of c never reaches farther back than a window of c
+    const int a = chunk > 0 ? chunk : window, b = chunk2 > 0 ? chunk2 : window2;
+    r.chunk = 0;
+    r.window = a == 0 || b == 0 ? 0 : std::max(a, b);
+    return r;
+}
 CacheRequest CacheRequest::state(std::vector<long long> shape, DType dtype) {
     CacheRequest r;
     r.kind = FixedState;

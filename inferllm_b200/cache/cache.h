@@ -50,6 +50,8 @@ struct CacheRequest {
     static CacheRequest paged(int n_kv_heads, int head_dim, int window = 0, int v_head_dim = 0);
     static CacheRequest paged_keys_only(int n_kv_heads, int head_dim, int window = 0);
     CacheRequest in_chunks(int size) const { CacheRequest r = *this; r.chunk = size; return r; }
+    // the request widened to what a second reader with this window or chunk (0, 0: all positions) needs as well
+    CacheRequest reaching(int window2, int chunk2) const;
     static CacheRequest state(std::vector<long long> shape, DType dtype = DType::F32);
     long long elements() const { long long n = 1; for (long long s : shape) n *= s; return n; }
     bool operator==(const CacheRequest& o) const;

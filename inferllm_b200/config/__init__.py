@@ -241,8 +241,16 @@ class FifotarConfig(LibraryConfig):
     architecture = "Fifotar"
 
 
+class ZeluzenConfig(LibraryConfig):
+    """The Zeluzen decoder (`config/zeluzen.h`): `layers` (a list of {type: "wkv" | "attention", mixer: {...}, mlp: {kind:
+    "dense", ff} | {kind: "moe", expert: {ff}, router: {experts, identity, top}} | None}), `width`, `vocab`, `norm` ({eps}),
+    optionally `max_positions`.  The dictionary names the class under `architecture`."""
+
+    architecture = "Zeluzen"
+
+
 _PY_CLASSES: Dict[str, type] = {"LlamaForCausalLM": LlamaConfig, "Vokelix": VokelixConfig, "Vizosun": VizosunConfig, "Kudonex": KudonexConfig,
-                                "Tukulorn": TukulornConfig, "Fifotar": FifotarConfig}
+                                "Tukulorn": TukulornConfig, "Fifotar": FifotarConfig, "Zeluzen": ZeluzenConfig}
 _CALLBACKS = {}      # name -> (ctypes callback, holder of the last returned text): kept alive while registered
 
 
@@ -285,7 +293,7 @@ def register_architecture(name: str, config_cls: type, aliases=()):
 def unregister_architecture(name: str):
     _b.check(_b.lib().illm_unregister_architecture(name.encode()))
     _CALLBACKS.pop(name, None)
-    if _PY_CLASSES.get(name) not in (LlamaConfig, VokelixConfig, VizosunConfig, KudonexConfig, TukulornConfig, FifotarConfig):
+    if _PY_CLASSES.get(name) not in (LlamaConfig, VokelixConfig, VizosunConfig, KudonexConfig, TukulornConfig, FifotarConfig, ZeluzenConfig):
         _PY_CLASSES.pop(name, None)
 
 

@@ -215,6 +215,7 @@ void register_vizosun_architecture();   // config/vizosun.cpp
 void register_kudonex_architecture();   // config/kudonex.cpp
 void register_tukulorn_architecture();  // config/tukulorn.cpp
 void register_fifotar_architecture();   // config/fifotar.cpp
+void register_zeluzen_architecture();   // config/zeluzen.cpp
 
 static void ensure_builtin() {
     static bool done = false;
@@ -226,6 +227,7 @@ static void ensure_builtin() {
         register_kudonex_architecture();
         register_tukulorn_architecture();
         register_fifotar_architecture();
+        register_zeluzen_architecture();
     }
 }
 

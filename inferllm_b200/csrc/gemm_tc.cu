@@ -22,6 +22,8 @@
 // kernel adds them in ascending order of the split (the result does not depend on timing).
 // Rows beyond M or N and columns beyond K are zero-filled by the TMA unit, so any M, any N and
 // any K that is a multiple of 8 (the 16-byte stride rule of tensor maps) is taken.
+// Several products of the decode form may run in one launch (GROUPED): group g's weight rows are a run of the stacked W and
+// its inputs rows of their own in a stacked X (one matrix per group, x_rows apart); its outputs are a run of columns of C.
 // Every wait on an mbarrier is bounded: after the limit the thread raises the error word and
 // goes on, so a fault in the pipeline ends the kernel instead of hanging the GPU.
 #include "tc_common.cuh"
@@ -44,11 +46,19 @@ template <int ACT> __device__ __forceinline__ float tc_gated(float gate, float u
 // D[ra, rb] = sum_k A[ra, k] B[rb, k];  SWAP = false: C[ra * ldc + rb];  SWAP = true: C[rb * ldc + ra].
 #define TC_MAX_STAGES 12
 
-template <int BN, bool SWAP, typename TOut, int GATED = 0>
+#define TC_MAX_GROUPS 8
+struct TcGroups {
+    int n = 0;                          // groups
+    int tile0[TC_MAX_GROUPS + 1];       // first tile of 128 weight rows of each group, and their number
+    int row0[TC_MAX_GROUPS + 1];        // first weight row (= output column) of each group, and their number
+    int x_rows;                         // rows of X from one group's inputs to the next's
+};
+
+template <int BN, bool SWAP, typename TOut, int GATED = 0, bool GROUPED = false>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                TOut* __restrict__ C, long long split_stride, int ldc, int RA, int RB, int k_iters_total,
-               int k_iters_per_split, int STAGES, float act_limit, int* __restrict__ err) {
+               int k_iters_per_split, int STAGES, float act_limit, const TcGroups groups, int* __restrict__ err) {
     constexpr unsigned A_BYTES = TC_BM * TC_BK * 2, B_BYTES = BN * TC_BK * 2;
     constexpr unsigned TMEM_COLS = BN < 32 ? 32 : BN;
     constexpr unsigned IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((unsigned)(BN >> 3) << 17) | ((unsigned)(TC_BM >> 4) << 24);
@@ -62,7 +72,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     const unsigned done_bar = tc_smem_u32(&bars[2 * TC_MAX_STAGES]);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int ra0 = blockIdx.x * TC_BM, rb0 = blockIdx.y * BN;
+    int ra0 = blockIdx.x * TC_BM, xr0 = 0;
+    const int rb0 = blockIdx.y * BN;
+    if (GROUPED) {
+        int g = 0;
+        while (g + 1 < groups.n && (int)blockIdx.x >= groups.tile0[g + 1]) g++;
+        ra0 = groups.row0[g] + ((int)blockIdx.x - groups.tile0[g]) * TC_BM;
+        RA = groups.row0[g + 1];            // rows of the tile beyond the group's are computed and not stored
+        xr0 = g * groups.x_rows;
+    }
     const int k_begin = blockIdx.z * k_iters_per_split;
     int k_end = k_begin + k_iters_per_split;
     if (k_end > k_iters_total) k_end = k_iters_total;
@@ -105,7 +123,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             asm volatile("griddepcontrol.wait;" ::: "memory");
             for (int i = 0; i < n_pre; i++) {
                 const int kx = (k_begin + i) * TC_BK;
-                if (SWAP) tma_load_2d(b_base + i * B_BYTES, &map_b, kx, rb0, full0 + 8 * i);
+                if (SWAP) tma_load_2d(b_base + i * B_BYTES, &map_b, kx, xr0 + rb0, full0 + 8 * i);
                 else tma_load_2d(a_base + i * A_BYTES, &map_a, kx, ra0, full0 + 8 * i);
             }
             bool alive = true;
@@ -116,7 +134,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 mbar_expect_tx(full0 + 8 * s, A_BYTES + B_BYTES);
                 const int kx = (k_begin + i) * TC_BK;
                 tma_load_2d(a_base + s * A_BYTES, &map_a, kx, ra0, full0 + 8 * s);
-                tma_load_2d(b_base + s * B_BYTES, &map_b, kx, rb0, full0 + 8 * s);
+                tma_load_2d(b_base + s * B_BYTES, &map_b, kx, xr0 + rb0, full0 + 8 * s);
             }
         }
     } else if (warp == 1) {
@@ -260,7 +278,59 @@ static int launch_tc(const CUtensorMap& ma, const CUtensorMap& mb, TOut* C, long
     auto kern = gemm_tc_kernel<BN, SWAP, TOut, GATED>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    illm_launch(kern, dim3(grid), dim3(TC_THREADS), smem, s, ma, mb, C, split_stride, ldc, RA, RB, k_iters, per_split, stages, act_limit, err);
+    illm_launch(kern, dim3(grid), dim3(TC_THREADS), smem, s, ma, mb, C, split_stride, ldc, RA, RB, k_iters, per_split, stages, act_limit, TcGroups(), err);
+    return illm_launch_status();
+}
+
+template <int BN, typename TOut>
+static int launch_tc_grouped(const CUtensorMap& ma, const CUtensorMap& mb, TOut* C, long long split_stride, const TcGroups& g, int N, int M, int k_iters,
+                             int splits, int* err, cudaStream_t s) {
+    const int stage_bytes = TC_BM * TC_BK * 2 + BN * TC_BK * 2;
+    const int per_split = (k_iters + splits - 1) / splits;
+    dim3 grid(g.tile0[g.n], 1, splits);
+    const int stages = pick_stages(stage_bytes, (long long)grid.x * grid.z, per_split);
+    const size_t smem = (size_t)stages * stage_bytes + 1024;
+    auto kern = gemm_tc_kernel<BN, true, TOut, 0, true>;
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    illm_launch(kern, dim3(grid), dim3(TC_THREADS), smem, s, ma, mb, C, split_stride, N, N, M, k_iters, per_split, stages, 0.f, g, err);
+    return illm_launch_status();
+}
+
+// Products of n_groups stacked weights with inputs of their own, for at most 64 rows: X [n_groups * x_rows, K] (the first M rows
+// of every x_rows are group g's inputs), W [sum of n[g], K], out [M, sum of n[g]] float32.  splits and skip_reduce as in
+// illm_gemm_bf16_tc.
+extern "C" int illm_gemm_bf16_tc_grouped(const void* X, int x_rows, const void* W, const int* n, int n_groups, float* out, int M, int K, float* ws,
+                                         int splits, int* err, void* stream, int skip_reduce) {
+    if (M <= 0) return 0;
+    if (M > 64 || x_rows < M || n_groups < 1 || n_groups > TC_MAX_GROUPS || K <= 0 || (K & 7) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15) || splits < 1)
+        return ILLM_ERR_BAD_ARG;
+    TcGroups g;
+    g.n = n_groups;
+    g.x_rows = x_rows;
+    g.tile0[0] = g.row0[0] = 0;
+    for (int i = 0; i < n_groups; i++) {
+        if (n[i] <= 0) return ILLM_ERR_BAD_ARG;
+        g.tile0[i + 1] = g.tile0[i] + (n[i] + TC_BM - 1) / TC_BM;
+        g.row0[i + 1] = g.row0[i] + n[i];
+    }
+    const int N = g.row0[n_groups], k_iters = (K + TC_BK - 1) / TC_BK, bn = M <= 16 ? 16 : (M <= 32 ? 32 : 64);
+    const int per = (k_iters + splits - 1) / splits;
+    splits = (k_iters + per - 1) / per;
+    if (splits > 1 && !ws) return ILLM_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    CUtensorMap ma, mb;
+    int rc;
+    if ((rc = make_map(&ma, W, N, K, TC_BM)) != 0) return rc;
+    if ((rc = make_map(&mb, X, (long long)n_groups * x_rows, K, bn)) != 0) return rc;
+    float* dst = splits > 1 ? ws : out;
+    const long long stride = splits > 1 ? (long long)M * N : 0;
+    if (bn == 16) rc = launch_tc_grouped<16, float>(ma, mb, dst, stride, g, N, M, k_iters, splits, err, s);
+    else if (bn == 32) rc = launch_tc_grouped<32, float>(ma, mb, dst, stride, g, N, M, k_iters, splits, err, s);
+    else rc = launch_tc_grouped<64, float>(ma, mb, dst, stride, g, N, M, k_iters, splits, err, s);
+    if (rc != 0 || splits == 1 || skip_reduce) return rc;
+    const long long total = (long long)M * N;
+    illm_launch(splitk_reduce_kernel<float>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, ws, out, total, splits);
     return illm_launch_status();
 }
 

@@ -145,7 +145,7 @@ int illm_window_put(int* window, int n_last, const int* rows, int col, const int
 // entry points with further parameters (the shorter forms above call them)
 int illm_qk_prep_ex(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq, const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot, int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages, int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every, void* stream);
 int illm_head_gemm_ex(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int y_dtype, int T, int heads, int N, int K, int nn, int x_ld, int x_hs, int y_ld, int y_hs, void* stream);
-int illm_moe_route_ex2(const float* logits, const float* bias, int T, int E, int top, int bm, int scoring, int groups, int keep, int renorm, int group_top, float sum_eps, float weight_scale, int* expert, float* weight, int* row_of_pair, int* pair_of_row, int* tile_expert, int* tile_row0, int* tile_rows, void* stream);
+int illm_moe_route_ex2(const float* logits, const float* bias, int T, int E, int identity, int top, int bm, int scoring, int groups, int keep, int renorm, int group_top, float sum_eps, float weight_scale, int* expert, float* weight, int* row_of_pair, int* pair_of_row, int* tile_expert, int* tile_row0, int* tile_rows, void* stream);
 int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated, int act, float act_limit, int bm, int tensor_cores, const int* pair_of_row, const int* tile_expert, const int* tile_row0, const int* tile_rows, void* stream);
 int illm_moe_gemm_tc_ex(const void* xs, const void* w, void* y, int P, int E, int N, int K, int gated, int act, float act_limit, int tiles, const int* tile_expert, const int* tile_row0, const int* tile_rows, int* err, void* stream);
 // attention_maps.cu
@@ -172,6 +172,20 @@ int illm_gemm_bf16_tc2_ex(const void* X, const void* W, void* out, int out_dtype
 int illm_gated_act_ex(const void* gu, void* out, int act_dtype, int T, int I, int act, float limit, void* stream);
 int illm_soft_cap(float* x, long long n, float cap, void* stream);
 int illm_norm_sandwich(float* x, const float* y, const float* wb, const float* w, void* out, int out_dtype, const int* rows, int n_rows, int H, float eps, int write_x, int center, float post_scale, void* stream);
+
+// outnorm.cu
+int illm_join_rmsnorm(float* x, const float* y, int splits, long long stride, const float* w, void* h, int h_dtype, int n_rows, int H, float eps, void* stream);
+int illm_embedding_normed(const int* ids, const void* table, int table_dtype, const float* w, float* x, void* h, int h_dtype, int T, int H, int V, float eps, int* err, void* stream);
+
+// wkv_state.cu
+int illm_token_mix(const float* x, int T, int H, int n_mix, const float* mu, float* prev, long long prev_stride, const int* slots, const int* cu_q, const int* token_seq, int B, int single, void* out, int act_dtype, long long group_stride, void* stream);
+int illm_wkv_supported(int d, int dv);
+int illm_wkv_scan(const float* y, int T, int ld, int r_off, int k_off, int v_off, int z_off, int rank, int nh, int d, int dv, const void* w2, int w2_dtype, const float* w0, const float* u, float* state, long long state_stride, const int* slots, const int* cu_q, float* w, float* bonus, float* out, int B, int segments, float* seg_state, float* seg_decay, void* stream);
+
+// gemm_tc.cu, qk_prep.cu, moe.cu: further forms
+int illm_gemm_bf16_tc_grouped(const void* X, int x_rows, const void* W, const int* n, int n_groups, float* out, int M, int K, float* ws, int splits, int* err, void* stream, int skip_reduce);
+int illm_qk_prep_heads(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq, const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot, int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages, int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every, const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, int head_norm, void* stream);
+int illm_moe_combine_ex(const float* rows, const int* row_of_pair, const float* weight, const float* plus, const void* x, int x_dtype, float* out, int T, int D, int top, void* stream);
 
 #ifdef __cplusplus
 }

@@ -7,9 +7,13 @@
 //                      (row_of_pair, pair_of_row), and the list of row tiles (tile -> expert, first row, rows)
 //   moe_gemm_kernel    one block per (row tile, 64 columns): rows of one expert against that expert's matrix; GATED:
 //                      the matrix's rows 2i, 2i + 1 are gate and up of output i (packed so at load), x is gathered by
-//                      token and hid = act(gate) * up; else the down product into float32 rows.  One chain of fused multiply-adds over the inner index per
+//                      token and hid = act(gate) * up (PLAIN: the matrix's rows are the outputs themselves, hid = act(x W^T),
+//                      for experts without a gate); else the down product into float32 rows.  One chain of fused multiply-adds over the inner index per
 //                      output, so a row's bits depend neither on its place among the rows nor on the step.
 //   moe_combine_kernel out[t] = sum over the choices, in their order, of weight * row
+//
+// Experts numbered E and higher (the router has more outputs than there are experts with matrices) are identity experts:
+// their output is the token's input; their pairs get no row (row_of_pair -1) and the combine kernel adds weight * x[t].
 //
 // Which row a pair gets within its expert is decided by atomics in shared memory and may differ from run to run;
 // no result depends on it.
@@ -158,7 +162,8 @@ moe_layout_kernel(const int* __restrict__ expert, int P, int E, int bm, int* __r
     int* cursor = si + 2 * E;
     for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = cursor[e] = 0;
     __syncthreads();
-    for (int i = threadIdx.x; i < P; i += blockDim.x) atomicAdd(&count[expert[i]], 1);
+    for (int i = threadIdx.x; i < P; i += blockDim.x)
+        if (expert[i] < E) atomicAdd(&count[expert[i]], 1);
     __syncthreads();
     if (threadIdx.x == 0) {
         int rows = 0, tiles = 0;
@@ -172,10 +177,16 @@ moe_layout_kernel(const int* __restrict__ expert, int P, int E, int bm, int* __r
             rows += count[e];
         }
         for (; tiles < max_tiles; tiles++) tile_rows[tiles] = 0;
+        si[3 * E] = rows;
     }
     __syncthreads();
+    for (int i = si[3 * E] + threadIdx.x; i < P; i += blockDim.x) pair_of_row[i] = -1;       // rows that no pair fills
     for (int i = threadIdx.x; i < P; i += blockDim.x) {
         const int e = expert[i];
+        if (e >= E) {
+            row_of_pair[i] = -1;
+            continue;
+        }
         const int row = offset[e] + atomicAdd(&cursor[e], 1);
         row_of_pair[i] = row;
         pair_of_row[row] = i;
@@ -193,6 +204,20 @@ __device__ __forceinline__ float moe_gated(float v, float u, int act, float limi
     }
     return v * u;
 }
+// act of an expert without a gate: 1 silu, 2 relu, 3 tanh-form gelu, 5 the square of relu
+__device__ __forceinline__ float moe_act(float v, int act) {
+    if (act == 5) {
+        const float r = fmaxf(v, 0.f);
+        return r * r;
+    }
+    return moe_gated(v, 1.f, act, 0.f);
+}
+
+// what a product's rows are: MOE_DOWN float32 rows by row; MOE_GATED act(gate) * up of row pairs; MOE_PLAIN act(row), the last
+// two from x gathered by token and in the dtype of x
+#define MOE_DOWN 0
+#define MOE_GATED 1
+#define MOE_PLAIN 2
 
 #define MOE_BN 64
 #define MOE_BK 16
@@ -200,7 +225,7 @@ __device__ __forceinline__ float moe_gated(float v, float u, int act, float limi
 // grid (ceil(Nw / 64), max_tiles); 256 threads = 16 x 16, a (BM / 16) x 4 patch of outputs each.  w [E, Nw, K].
 // GATED: x [T, K] gathered through pair_of_row / top; the matrix's rows 2i, 2i + 1 are gate and up of output i, and
 // y [P, Nw / 2] = act(gate) * up; else x [P, K] by row and y [P, Nw].
-template <typename TX, typename TW, typename TY, int BM, bool GATED>
+template <typename TX, typename TW, typename TY, int BM, int MODE>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TY* __restrict__ y, int Nw, int K, int top, int act, float act_limit,
                 const int* __restrict__ pair_of_row, const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
@@ -215,7 +240,7 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TY* __restri
     if (rows == 0) return;
     const int e = tile_expert[tile], row0 = tile_row0[tile], n0 = blockIdx.x * MOE_BN;
     const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
-    for (int m = threadIdx.x; m < BM; m += 256) src_row[m] = m < rows ? (GATED ? pair_of_row[row0 + m] / top : row0 + m) : -1;
+    for (int m = threadIdx.x; m < BM; m += 256) src_row[m] = m < rows ? (MODE != MOE_DOWN ? pair_of_row[row0 + m] / top : row0 + m) : -1;
     const TW* we = w + (size_t)e * Nw * K;
     float acc[RM][4];
 #pragma unroll
@@ -252,7 +277,7 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TY* __restri
     for (int i = 0; i < RM; i++) {
         const int m = ty * RM + i;
         if (m >= rows) continue;
-        if (GATED) {
+        if (MODE == MOE_GATED) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx * 4 + j;
@@ -262,7 +287,7 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TY* __restri
 #pragma unroll
             for (int j = 0; j < 4; j++) {
                 const int n = n0 + tx * 4 + j;
-                if (n < Nw) y[(size_t)(row0 + m) * Nw + n] = from_f32<TY>(acc[i][j]);
+                if (n < Nw) y[(size_t)(row0 + m) * Nw + n] = from_f32<TY>(MODE == MOE_PLAIN ? moe_act(acc[i][j], act) : acc[i][j]);
             }
         }
     }
@@ -293,7 +318,7 @@ __device__ __forceinline__ void mm_mma(float* c, const unsigned* a, unsigned b0,
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <typename TY, bool GATED>
+template <typename TY, int MODE>
 __global__ void __launch_bounds__(256)
 moe_gemm_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* __restrict__ y, int N, int K, int top, int act, float act_limit,
                     const int* __restrict__ pair_of_row, const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
@@ -309,7 +334,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* 
     if (rows == 0) return;
     const int e = tile_expert[tile], row0 = tile_row0[tile], n0 = blockIdx.x * MM_BN;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wm = warp >> 2, wn = warp & 3;
-    for (int m = tid; m < MM_BM; m += 256) src_row[m] = m < rows ? (GATED ? pair_of_row[row0 + m] / top : row0 + m) : -1;
+    for (int m = tid; m < MM_BM; m += 256) src_row[m] = m < rows ? (MODE != MOE_DOWN ? pair_of_row[row0 + m] / top : row0 + m) : -1;
     __syncthreads();
     const bf16* wg = w + (size_t)e * N * K;
     const int KT = (K + MM_BK - 1) / MM_BK;
@@ -383,28 +408,34 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* 
 #pragma unroll
         for (int j = 0; j < 4; j++)
 #pragma unroll
-            for (int c = 0; c < 4; c += GATED ? 2 : 1) {
+            for (int c = 0; c < 4; c += MODE == MOE_GATED ? 2 : 1) {
                 const int m = wm * 32 + i * 16 + (lane >> 2) + (c >> 1) * 8;
                 const int n = n0 + wn * 32 + j * 8 + (lane & 3) * 2 + (c & 1);
                 if (m >= rows) continue;
-                if (GATED) {          // columns n, n + 1 are gate and up of output n / 2
+                if (MODE == MOE_GATED) {          // columns n, n + 1 are gate and up of output n / 2
                     if (n + 1 < N) y[(size_t)(row0 + m) * (N / 2) + n / 2] = from_f32<TY>(moe_gated(acc[0][i][j][c], acc[0][i][j][c + 1], act, act_limit));
                 } else if (n < N) {
-                    y[(size_t)(row0 + m) * N + n] = from_f32<TY>(acc[0][i][j][c]);
+                    y[(size_t)(row0 + m) * N + n] = from_f32<TY>(MODE == MOE_PLAIN ? moe_act(acc[0][i][j][c], act) : acc[0][i][j][c]);
                 }
             }
 }
 
-// plus: float32 [T, D] added to the experts' sum (a shared expert's output), or nullptr
+// plus: float32 [T, D] added to the experts' sum (a shared expert's output), or nullptr; x [T, D]: what an identity expert
+// gives back (nullptr: there are none)
+template <typename TX>
 __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ row_of_pair, const float* __restrict__ weight,
-                                   const float* __restrict__ plus, float* __restrict__ out, int D, int top, long long n) {
+                                   const float* __restrict__ plus, const TX* __restrict__ x, float* __restrict__ out, int D, int top, long long n) {
     pdl_grid_sync();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
     const long long t = i / D;
     const int c = (int)(i - t * D);
     float acc = 0.f;
-    for (int k = 0; k < top; k++) acc = fmaf(weight[t * top + k], rows[(size_t)row_of_pair[t * top + k] * D + c], acc);
+    for (int k = 0; k < top; k++) {
+        const int row = row_of_pair[t * top + k];
+        const float v = row >= 0 ? rows[(size_t)row * D + c] : x ? to_f32(x[i]) : 0.f;
+        acc = fmaf(weight[t * top + k], v, acc);
+    }
     out[i] = plus ? acc + plus[i] : acc;
 }
 
@@ -416,6 +447,7 @@ extern "C" int illm_moe_row_tile(int T, int top, int tensor_cores) { return tens
 __global__ void moe_gather_rows_kernel(const bf16* __restrict__ x, bf16* __restrict__ xs, const int* __restrict__ pair_of_row, int K, int top) {
     pdl_grid_sync();
     const int row = blockIdx.x;
+    if (pair_of_row[row] < 0) return;
     const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)(pair_of_row[row] / top) * K);
     uint4* dst = reinterpret_cast<uint4*>(xs + (size_t)row * K);
     for (int c = threadIdx.x; c < K / 8; c += blockDim.x) dst[c] = src[c];
@@ -437,32 +469,34 @@ extern "C" int illm_moe_route(const float* logits, const float* bias, int T, int
     return illm_moe_route_ex(logits, bias, T, E, top, bm, 0, 1, 1, 1, expert, weight, row_of_pair, pair_of_row, tile_expert, tile_row0, tile_rows, stream);
 }
 
-extern "C" int illm_moe_route_ex2(const float* logits, const float* bias, int T, int E, int top, int bm, int scoring, int groups, int keep, int renorm,
+extern "C" int illm_moe_route_ex2(const float* logits, const float* bias, int T, int E, int identity, int top, int bm, int scoring, int groups, int keep, int renorm,
                                   int group_top, float sum_eps, float weight_scale, int* expert, float* weight, int* row_of_pair, int* pair_of_row,
                                   int* tile_expert, int* tile_row0, int* tile_rows, void* stream);
 extern "C" int illm_moe_route_ex(const float* logits, const float* bias, int T, int E, int top, int bm, int scoring, int groups, int keep, int renorm,
                                  int* expert, float* weight, int* row_of_pair, int* pair_of_row, int* tile_expert, int* tile_row0, int* tile_rows,
                                  void* stream) {
-    return illm_moe_route_ex2(logits, bias, T, E, top, bm, scoring, groups, keep, renorm, 1, 0.f, 1.f, expert, weight, row_of_pair, pair_of_row, tile_expert,
+    return illm_moe_route_ex2(logits, bias, T, E, 0, top, bm, scoring, groups, keep, renorm, 1, 0.f, 1.f, expert, weight, row_of_pair, pair_of_row, tile_expert,
                               tile_row0, tile_rows, stream);
 }
 // scoring 0: the `top` largest logits + bias, weights the softmax over the chosen; scoring 1: scores are the softmax
 // over all experts, 2: the sigmoid of every logit; with 1 and 2 the bias enters the choice only, `keep` of `groups` groups
 // (scored by the sum of their group_top largest) may be chosen from, weights divided by their sum + sum_eps if renorm and
-// multiplied by weight_scale (moe_route_scored_kernel)
-extern "C" int illm_moe_route_ex2(const float* logits, const float* bias, int T, int E, int top, int bm, int scoring, int groups, int keep, int renorm,
+// multiplied by weight_scale (moe_route_scored_kernel).  identity: how many experts without matrices the router knows beside
+// the E with matrices (the logits have E + identity columns)
+extern "C" int illm_moe_route_ex2(const float* logits, const float* bias, int T, int E, int identity, int top, int bm, int scoring, int groups, int keep, int renorm,
                                   int group_top, float sum_eps, float weight_scale, int* expert, float* weight, int* row_of_pair, int* pair_of_row,
                                   int* tile_expert, int* tile_row0, int* tile_rows, void* stream) {
     if (T <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || (bm != 16 && bm != 64 && bm != 128) || (size_t)(3 * E + 1) * sizeof(int) > 160 * 1024) return ILLM_ERR_BAD_ARG;
+    const int all = E + identity;
+    if (E <= 0 || identity < 0 || top <= 0 || top > all || (bm != 16 && bm != 64 && bm != 128) || (size_t)(3 * E + 1) * sizeof(int) > 160 * 1024) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     if (scoring == 1 || scoring == 2) {
-        if (groups < 1 || groups > 32 || E % groups || keep < 1 || keep > groups || (long long)keep * (E / groups) < top || group_top < 1 || group_top > 4)
+        if (groups < 1 || groups > 32 || all % groups || keep < 1 || keep > groups || (long long)keep * (all / groups) < top || group_top < 1 || group_top > 4)
             return ILLM_ERR_BAD_ARG;
-        illm_launch(moe_route_scored_kernel, dim3((T + 3) / 4), dim3(128), 0, s, logits, bias, T, E, top, groups, keep, renorm, scoring == 2 ? 1 : 0,
+        illm_launch(moe_route_scored_kernel, dim3((T + 3) / 4), dim3(128), 0, s, logits, bias, T, all, top, groups, keep, renorm, scoring == 2 ? 1 : 0,
                     group_top, sum_eps, weight_scale, expert, weight);
     } else if (scoring == 0) {
-        illm_launch(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, s, logits, bias, T, E, top, expert, weight);
+        illm_launch(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, s, logits, bias, T, all, top, expert, weight);
     } else {
         return ILLM_ERR_BAD_ARG;
     }
@@ -477,8 +511,8 @@ extern "C" int illm_moe_route_ex2(const float* logits, const float* bias, int T,
     return illm_launch_status();
 }
 
-// w [E, N, K].  gated != 0: x [T, K] (x_dtype), the matrix's rows 2i, 2i + 1 gate and up of output i, y [T * top, N / 2] in
-// the dtype of x; else x [T * top, K], y [T * top, N] float32.
+// w [E, N, K].  gated 1: x [T, K] (x_dtype), the matrix's rows 2i, 2i + 1 gate and up of output i, y [T * top, N / 2] in
+// the dtype of x; gated 2: x [T, K], y [T * top, N] = act of the rows in the dtype of x; 0: x [T * top, K], y [T * top, N] float32.
 // tensor_cores != 0 (bfloat16, K % 8 == 0, tiles of 64 rows): the mma kernel.
 extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated,
                                 int act, float act_limit, int bm, int tensor_cores, const int* pair_of_row, const int* tile_expert,
@@ -494,7 +528,7 @@ extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w
                                 int act, float act_limit, int bm, int tensor_cores, const int* pair_of_row, const int* tile_expert,
                                 const int* tile_row0, const int* tile_rows, void* stream) {
     if (T <= 0) return 0;
-    if (N <= 0 || K <= 0 || x_dtype != w_dtype || (bm != 16 && bm != 64) || (gated && (N & 1))) return ILLM_ERR_BAD_ARG;
+    if (N <= 0 || K <= 0 || x_dtype != w_dtype || (bm != 16 && bm != 64) || gated < 0 || gated > 2 || (gated == 1 && (N & 1))) return ILLM_ERR_BAD_ARG;
     const int tiles = illm_moe_max_tiles(T, top, E, bm);
     if (tiles > 65535) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
@@ -504,15 +538,19 @@ extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w
         const size_t smem = (size_t)MM_STAGES * (MM_BM + MM_BN) * MM_LD * sizeof(bf16);
         static bool raised = false;
         if (!raised) {
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<bf16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<float, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<bf16, MOE_GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<bf16, MOE_PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<float, MOE_DOWN>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
             raised = true;
         }
-        if (gated)
-            illm_launch(moe_gemm_mma_kernel<bf16, true>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (bf16*)y, N, K, top, act, act_limit,
+        if (gated == 1)
+            illm_launch(moe_gemm_mma_kernel<bf16, MOE_GATED>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (bf16*)y, N, K, top, act, act_limit,
+                        pair_of_row, tile_expert, tile_row0, tile_rows);
+        else if (gated == 2)
+            illm_launch(moe_gemm_mma_kernel<bf16, MOE_PLAIN>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (bf16*)y, N, K, top, act, act_limit,
                         pair_of_row, tile_expert, tile_row0, tile_rows);
         else
-            illm_launch(moe_gemm_mma_kernel<float, false>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (float*)y, N, K, top, act, act_limit,
+            illm_launch(moe_gemm_mma_kernel<float, MOE_DOWN>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (float*)y, N, K, top, act, act_limit,
                         pair_of_row, tile_expert, tile_row0, tile_rows);
         return illm_launch_status();
     }
@@ -521,11 +559,13 @@ extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w
     illm_launch(moe_gemm_kernel<TX, TX, TY, BM, G>, grid, dim3(256), 0, s, (const TX*)x, (const TX*)w, (TY*)y, N, K, top, act, act_limit, pair_of_row, \
                 tile_expert, tile_row0, tile_rows)
     if (x_dtype == ILLM_BF16) {
-        if (gated) { if (bm == 16) ILLM_MOE(bf16, bf16, 16, true); else ILLM_MOE(bf16, bf16, 64, true); }
-        else { if (bm == 16) ILLM_MOE(bf16, float, 16, false); else ILLM_MOE(bf16, float, 64, false); }
+        if (gated == 1) { if (bm == 16) ILLM_MOE(bf16, bf16, 16, MOE_GATED); else ILLM_MOE(bf16, bf16, 64, MOE_GATED); }
+        else if (gated == 2) { if (bm == 16) ILLM_MOE(bf16, bf16, 16, MOE_PLAIN); else ILLM_MOE(bf16, bf16, 64, MOE_PLAIN); }
+        else { if (bm == 16) ILLM_MOE(bf16, float, 16, MOE_DOWN); else ILLM_MOE(bf16, float, 64, MOE_DOWN); }
     } else if (x_dtype == ILLM_F32) {
-        if (gated) { if (bm == 16) ILLM_MOE(float, float, 16, true); else ILLM_MOE(float, float, 64, true); }
-        else { if (bm == 16) ILLM_MOE(float, float, 16, false); else ILLM_MOE(float, float, 64, false); }
+        if (gated == 1) { if (bm == 16) ILLM_MOE(float, float, 16, MOE_GATED); else ILLM_MOE(float, float, 64, MOE_GATED); }
+        else if (gated == 2) { if (bm == 16) ILLM_MOE(float, float, 16, MOE_PLAIN); else ILLM_MOE(float, float, 64, MOE_PLAIN); }
+        else { if (bm == 16) ILLM_MOE(float, float, 16, MOE_DOWN); else ILLM_MOE(float, float, 64, MOE_DOWN); }
     } else {
         return ILLM_ERR_BAD_ARG;
     }
@@ -533,12 +573,21 @@ extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w
     return illm_launch_status();
 }
 
-extern "C" int illm_moe_combine_plus(const float* rows, const int* row_of_pair, const float* weight, const float* plus, float* out, int T, int D,
-                                     int top, void* stream) {
+// x (x_dtype, [T, D]): the input rows, for pairs without a row (identity experts); nullptr: there are none
+extern "C" int illm_moe_combine_ex(const float* rows, const int* row_of_pair, const float* weight, const float* plus, const void* x, int x_dtype,
+                                   float* out, int T, int D, int top, void* stream) {
     if (T <= 0) return 0;
     const long long n = (long long)T * D;
-    illm_launch(moe_combine_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, rows, row_of_pair, weight, plus, out, D, top, n);
+    const dim3 grid((unsigned)((n + 255) / 256));
+    cudaStream_t s = (cudaStream_t)stream;
+    if (x && x_dtype == ILLM_BF16) illm_launch(moe_combine_kernel<bf16>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const bf16*)x, out, D, top, n);
+    else if (!x || x_dtype == ILLM_F32) illm_launch(moe_combine_kernel<float>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const float*)x, out, D, top, n);
+    else return ILLM_ERR_BAD_ARG;
     return illm_launch_status();
+}
+extern "C" int illm_moe_combine_plus(const float* rows, const int* row_of_pair, const float* weight, const float* plus, float* out, int T, int D,
+                                     int top, void* stream) {
+    return illm_moe_combine_ex(rows, row_of_pair, weight, plus, nullptr, 0, out, T, D, top, stream);
 }
 extern "C" int illm_moe_combine(const float* rows, const int* row_of_pair, const float* weight, float* out, int T, int D, int top,
                                 void* stream) {

@@ -7,7 +7,7 @@
 //      the box reads beyond them (the next expert's rows, zeros beyond P) is computed and not stored;
 //   B  the experts' matrices stacked [E * N, K]; the tile's rows start at expert * N + column offset.
 // GATED: the matrix's rows 2i, 2i + 1 are gate and up of output i; a thread of the epilogue holds neighbouring
-// columns and stores act(gate) * up.  The tile list is written by the kernel before this one, so every thread waits
+// columns and stores act(gate) * up.  PLAIN: the rows are the outputs themselves, stored as act of them.  The tile list is written by the kernel before this one, so every thread waits
 // for it (griddepcontrol.wait) before anything else, and a block whose tile is empty leaves at once.
 #include "tc_common.cuh"
 
@@ -25,7 +25,20 @@ __device__ __forceinline__ float mt_gated(float v, float u, int act, float limit
     return v * u;
 }
 
-template <int BN, typename TOut, bool GATED>
+// act of an expert without a gate: 5 is the square of relu
+__device__ __forceinline__ float mt_act(float v, int act) {
+    if (act == 5) {
+        const float r = fmaxf(v, 0.f);
+        return r * r;
+    }
+    return mt_gated(v, 1.f, act, 0.f);
+}
+
+#define MT_DOWN 0
+#define MT_GATED 1
+#define MT_PLAIN 2
+
+template <int BN, typename TOut, int MODE>
 __global__ void __launch_bounds__(TC_THREADS)
 moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, TOut* __restrict__ C, int ldc,
                    int n_per_expert, int n_k, int STAGES, int act, float act_limit, const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
@@ -112,7 +125,7 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                 float v[16];
                 tmem_ld16(tmem + ((unsigned)(quad * 32) << 16) + (unsigned)c0, v);
                 if (m >= rows) continue;
-                if (GATED) {
+                if (MODE == MT_GATED) {
                     TOut* dst = C + ra * ldc + (nb0 + c0) / 2;
                     float o[8];
 #pragma unroll
@@ -126,6 +139,10 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                     }
                 } else {
                     TOut* dst = C + ra * ldc + nb0 + c0;
+                    if (MODE == MT_PLAIN) {
+#pragma unroll
+                        for (int j = 0; j < 16; j++) v[j] = mt_act(v[j], act);
+                    }
                     if (nb0 + c0 + 16 <= n_per_expert && (ldc & 7) == 0) {
                         store8(dst, v);
                         store8(dst + 8, v + 8);
@@ -168,7 +185,7 @@ static int mt_make_map(CUtensorMap* map, const void* ptr, long long rows, long l
     return r == CUDA_SUCCESS ? 0 : ILLM_ERR_BAD_ARG;
 }
 
-template <int BN, typename TOut, bool GATED>
+template <int BN, typename TOut, int MODE>
 static int mt_launch(const CUtensorMap& ma, const CUtensorMap& mb, TOut* y, int ldc, int N, int k_iters, int tiles, int act, float act_limit, const int* tile_expert,
                      const int* tile_row0, const int* tile_rows, int* err, cudaStream_t s) {
     const int stage_bytes = TC_BM * TC_BK * 2 + BN * TC_BK * 2;
@@ -180,7 +197,7 @@ static int mt_launch(const CUtensorMap& ma, const CUtensorMap& mb, TOut* y, int 
     if (stages > k_iters) stages = k_iters;
     if (stages < 2) stages = 2;
     const size_t smem = (size_t)stages * stage_bytes + 1024;
-    auto kern = moe_gemm_tc_kernel<BN, TOut, GATED>;
+    auto kern = moe_gemm_tc_kernel<BN, TOut, MODE>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     illm_launch(kern, dim3(tiles, (N + BN - 1) / BN), dim3(TC_THREADS), smem, s, ma, mb, y, ldc, N, k_iters, stages, act, act_limit, tile_expert, tile_row0,
@@ -189,7 +206,8 @@ static int mt_launch(const CUtensorMap& ma, const CUtensorMap& mb, TOut* y, int 
 }
 
 // xs [P, K] bfloat16: the rows in the experts' order; w [E * N, K] bfloat16; the tile list with tiles of up to 128 rows
-// (`tiles` entries).  gated != 0: y [P, N / 2] bfloat16 = act(gate) * up of the matrix's row pairs; else y [P, N] float32.
+// (`tiles` entries).  gated 1: y [P, N / 2] bfloat16 = act(gate) * up of the matrix's row pairs; 2: y [P, N] bfloat16 = act of the
+// rows; 0: y [P, N] float32.
 extern "C" int illm_moe_gemm_tc_ex(const void* xs, const void* w, void* y, int P, int E, int N, int K, int gated, int act, float act_limit, int tiles,
                                    const int* tile_expert, const int* tile_row0, const int* tile_rows, int* err, void* stream);
 extern "C" int illm_moe_gemm_tc(const void* xs, const void* w, void* y, int P, int E, int N, int K, int gated, int act, int tiles,
@@ -200,7 +218,7 @@ extern "C" int illm_moe_gemm_tc(const void* xs, const void* w, void* y, int P, i
 extern "C" int illm_moe_gemm_tc_ex(const void* xs, const void* w, void* y, int P, int E, int N, int K, int gated, int act, float act_limit, int tiles,
                                    const int* tile_expert, const int* tile_row0, const int* tile_rows, int* err, void* stream) {
     if (P <= 0) return 0;
-    if (N <= 0 || K <= 0 || (K & 7) || (gated && (N & 1)) || ((uintptr_t)xs & 15) || ((uintptr_t)w & 15) || tiles <= 0) return ILLM_ERR_BAD_ARG;
+    if (N <= 0 || K <= 0 || (K & 7) || gated < 0 || gated > 2 || (gated == 1 && (N & 1)) || ((uintptr_t)xs & 15) || ((uintptr_t)w & 15) || tiles <= 0) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int k_iters = (K + TC_BK - 1) / TC_BK;
     const int bn = N >= 256 ? 256 : 128;
@@ -208,10 +226,14 @@ extern "C" int illm_moe_gemm_tc_ex(const void* xs, const void* w, void* y, int P
     int rc;
     if ((rc = mt_make_map(&ma, xs, P, K, TC_BM)) != 0) return rc;
     if ((rc = mt_make_map(&mb, w, (long long)E * N, K, bn)) != 0) return rc;
-    if (gated) {
-        if (bn == 256) return mt_launch<256, bf16, true>(ma, mb, (bf16*)y, N / 2, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
-        return mt_launch<128, bf16, true>(ma, mb, (bf16*)y, N / 2, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
+    if (gated == 2) {
+        if (bn == 256) return mt_launch<256, bf16, MT_PLAIN>(ma, mb, (bf16*)y, N, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
+        return mt_launch<128, bf16, MT_PLAIN>(ma, mb, (bf16*)y, N, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
     }
-    if (bn == 256) return mt_launch<256, float, false>(ma, mb, (float*)y, N, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
-    return mt_launch<128, float, false>(ma, mb, (float*)y, N, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
+    if (gated) {
+        if (bn == 256) return mt_launch<256, bf16, MT_GATED>(ma, mb, (bf16*)y, N / 2, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
+        return mt_launch<128, bf16, MT_GATED>(ma, mb, (bf16*)y, N / 2, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
+    }
+    if (bn == 256) return mt_launch<256, float, MT_DOWN>(ma, mb, (float*)y, N, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
+    return mt_launch<128, float, MT_DOWN>(ma, mb, (float*)y, N, N, k_iters, tiles, act, act_limit, tile_expert, tile_row0, tile_rows, err, s);
 }

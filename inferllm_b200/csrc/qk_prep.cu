@@ -4,6 +4,7 @@
 //   q = x[q_off : q_off + nh d] + bq;   k = x[k_off : ...] + bk;   v = x[v_off : ...] + bv     (biases optional)
 //   q = q / sqrt(mean(q^2) + eps) * wq,  the mean over the WHOLE projection of the token, all heads
 //       together; likewise k with wk                                                            (optional)
+//   or: every head of q is normed by itself, q_h / sqrt(mean(q_h^2) + eps) * wq with wq of one head's size; likewise k
 //   the first `rot` channels of every q and k head are rotated by the token's position, either in the
 //       interleaved layout (channel 2j with 2j + 1) or the rotate-half one (j with j + rot / 2), with
 //       (cos, sin) from a float32 table [positions, rot / 2, 2] that may carry a magnitude factor
@@ -36,6 +37,7 @@ struct QkPrepArgs {
     int v_first_ld;
     const float* v_lambda;
     float* v_keep;              // [T, nkv dv] or nullptr
+    int head_norm;              // wq, wk: of one head's size, every head normed by itself
 };
 
 __device__ __forceinline__ float rotated(const float* buf, int e, int rot, int pairs, const float* cs) {
@@ -85,12 +87,24 @@ __global__ void __launch_bounds__(256) qk_prep_kernel(QkPrepArgs a) {
         buf[nq + c] = v;
         ssk += v * v;
     }
-    if (a.wq) {
+    if (a.head_norm) {
+        __syncthreads();
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, heads = a.nh + (nk ? a.nkv : 0);
+        for (int hd = warp; hd < heads; hd += 8) {          // a warp per head, the sum in the order of the lanes' channels
+            float* row = buf + (size_t)hd * a.d;
+            const float* w = hd < a.nh ? a.wq : a.wk;
+            float ss = 0.f;
+            for (int c = lane; c < a.d; c += 32) ss = fmaf(row[c], row[c], ss);
+            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.d + a.eps);
+            for (int c = lane; c < a.d; c += 32) row[c] = (row[c] * inv) * w[c];
+        }
+    }
+    if (a.wq && !a.head_norm) {
         ssq = block_sum(ssq, scratch);
         const float inv = 1.0f / sqrtf(ssq / (float)nq + a.eps);
         for (int c = threadIdx.x; c < nq; c += blockDim.x) buf[c] = (buf[c] * inv) * a.wq[c];
     }
-    if (a.wk && nk) {
+    if (a.wk && nk && !a.head_norm) {
         ssk = block_sum(ssk, scratch);
         const float inv = 1.0f / sqrtf(ssk / (float)nk + a.eps);
         for (int c = threadIdx.x; c < nk; c += blockDim.x) buf[nq + c] = (buf[nq + c] * inv) * a.wk[c];
@@ -140,6 +154,12 @@ extern "C" int illm_qk_prep_mix(const void* x, int x_dtype, int ld, int q_off, i
                                 int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
                                 int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
                                 const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, void* stream);
+// the same with norms per head (head_norm != 0: wq and wk have one head's size)
+extern "C" int illm_qk_prep_heads(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq,
+                                  const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot,
+                                  int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
+                                  int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
+                                  const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, int head_norm, void* stream);
 extern "C" int illm_qk_prep(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq,
                             const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot,
                             int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
@@ -160,13 +180,23 @@ extern "C" int illm_qk_prep_mix(const void* x, int x_dtype, int ld, int q_off, i
                                 int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
                                 int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
                                 const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, void* stream) {
+    return illm_qk_prep_heads(x, x_dtype, ld, q_off, k_off, v_off, nh, nkv, d, dv, bq, bk, bv, wq, wk, eps, cos_sin, rot, pairs, n_pos, token_pos, token_seq,
+                              block_table, max_pages, page_size, q_out, kc, vc, act_dtype, T, err, qt_coef, qt_every, v_first, v_first_ld, v_lambda, v_keep, 0,
+                              stream);
+}
+extern "C" int illm_qk_prep_heads(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq,
+                                  const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot,
+                                  int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages,
+                                  int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every,
+                                  const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, int head_norm, void* stream) {
     if (T <= 0) return 0;
+    if (head_norm && (!wq || (k_off >= 0 && !wk))) return ILLM_ERR_BAD_ARG;
     if (qt_every < 0 || (v_first && (!v_lambda || v_first_ld < nkv * dv)) || ((v_first || v_keep) && (k_off < 0 || v_off < 0 || !vc))) return ILLM_ERR_BAD_ARG;
     if (nh <= 0 || d <= 0 || rot < 0 || rot > d || (rot & 1) || (rot && !cos_sin) || !x || !q_out) return ILLM_ERR_BAD_ARG;
     if (k_off >= 0 && (nkv <= 0 || dv <= 0)) return ILLM_ERR_BAD_ARG;      // v_off < 0 with k_off >= 0: keys alone are stored
     QkPrepArgs a{x, ld, q_off, k_off, v_off, nh, nkv, d, dv, bq, bk, bv, wq, wk, eps, cos_sin, rot, pairs, n_pos,
                  token_pos, token_seq, block_table, max_pages, page_size, q_out, kc, vc, err, qt_coef, qt_every,
-                 v_first, v_first_ld, v_lambda, v_keep};
+                 v_first, v_first_ld, v_lambda, v_keep, head_norm};
     const size_t smem = (size_t)(nh * d + (k_off >= 0 ? nkv * d : 0)) * sizeof(float);
     if (smem > 200 * 1024) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;

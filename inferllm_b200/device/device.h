@@ -87,7 +87,7 @@ public:
     // input or output is the head of a wider piece: rows x_ld / out_ld elements apart, heads x_head_stride / out_head_stride
     // (0: the packed layout).
     void library_gemm_bf16_heads(const void* x, const void* w, void* out, int M, int N, int K, int batch, bool transposed, int x_ld = 0,
-                                 long long x_head_stride = 0, int out_ld = 0, long long out_head_stride = 0);
+                                 long long x_head_stride = 0, int out_ld = 0, long long out_head_stride = 0, DType out_dtype = DType::BF16);
 
     // Copy a small host array to the device without making the host wait for the work already queued:
     // through a ring of pinned staging buffers, each reused only when its copy has left.

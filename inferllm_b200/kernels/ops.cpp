@@ -463,6 +463,36 @@ Mat scale_add_rmsnorm(Device& dev, const Mat& resid, const MatOrPartials* delta,
     return y;
 }
 
+Mat join_rmsnorm(Device& dev, const Mat& resid, const MatOrPartials& y, const Mat& w, float eps, DType out_dtype, bool want_rows) {
+    need(resid, "resid", true, DType::F32);
+    need(w, "norm weight", true, DType::F32);
+    const long long H = resid.cols;
+    if (w.rows * w.cols != H || y.rows() != resid.rows || y.cols() != H) throw KernelError("join_rmsnorm: the addition and the weight must have the stream's shape and width");
+    if (H > kMaxNormWidth) throw KernelError("join_rmsnorm: width " + std::to_string(H) + " exceeds what one block's shared memory holds");
+    Mat d;
+    if (!y.is_partials()) d = cast(dev, y.m, DType::F32);
+    Mat h;
+    if (want_rows) h = new_mat(dev, resid.rows, H, out_dtype);
+    check_kernel(illm_join_rmsnorm((float*)resid.p, y.is_partials() ? y.part.ws : (const float*)d.p, y.is_partials() ? y.part.splits : 1,
+                                   y.is_partials() ? y.part.rows * y.part.cols : 0, (const float*)w.p, want_rows ? h.p : nullptr,
+                                   want_rows ? code_of(out_dtype, "join_rmsnorm") : 0, (int)resid.rows, (int)H, eps, dev.stream()),
+                 "join_rmsnorm");
+    return h;
+}
+
+Mat embedding_normed(Device& dev, const StepView& ctx, const Mat& table, const Mat& w, float eps, DType dtype, Mat* rows) {
+    need(table, "table", true, dtype);
+    need(w, "norm weight", true, DType::F32);
+    if (w.rows * w.cols != table.cols) throw KernelError("embedding_normed: the norm's weight must have the table's width");
+    Mat out = new_mat_exact(dev, ctx.T, table.cols, DType::F32);
+    const bool copy = dtype != DType::F32;
+    *rows = copy ? new_mat(dev, ctx.T, table.cols, dtype) : out;
+    check_kernel(illm_embedding_normed(ctx.ids, table.p, code_of(table.dtype, "embedding_normed"), (const float*)w.p, (float*)out.p, copy ? rows->p : nullptr,
+                                       code_of(dtype, "embedding_normed"), ctx.T, (int)table.cols, (int)table.rows, eps, ctx.err, dev.stream()),
+                 "embedding_normed");
+    return out;
+}
+
 Mat qk_prep(Device& dev, const Mat& x, const QkPrep& p, Geometry g, const StepView& ctx, const KVView& kv, DType act_dtype) {
     need(x, "the packed projection");
     if (x.dtype != DType::F32 && x.dtype != act_dtype) throw KernelError("qk_prep: the projection must be float32 or the activation dtype");
@@ -474,11 +504,11 @@ Mat qk_prep(Device& dev, const Mat& x, const QkPrep& p, Geometry g, const StepVi
     Mat q = new_mat(dev, x.rows, (long long)g.n_heads * g.head_dim, act_dtype);
     if (p.q_temp_every < 0) throw KernelError("qk_prep: the query temperature's period must not be negative");
     if (p.v_first && (!p.v_lambda || p.v_first_ld < g.n_kv_heads * dv)) throw KernelError("qk_prep: mixed values need their factor and rows of the values' width");
-    check_kernel(illm_qk_prep_mix(x.p, code_of(x.dtype, "qk_prep"), (int)x.cols, p.q_off, has_kv ? p.k_off : -1, p.v_off, g.n_heads, g.n_kv_heads, g.head_dim, dv,
+    check_kernel(illm_qk_prep_heads(x.p, code_of(x.dtype, "qk_prep"), (int)x.cols, p.q_off, has_kv ? p.k_off : -1, p.v_off, g.n_heads, g.n_kv_heads, g.head_dim, dv,
                                  p.q_bias, p.k_bias, p.v_bias, p.q_norm, p.k_norm, p.eps, p.cos_sin, p.rot_dim, p.pairs ? 1 : 0, (int)p.n_pos,
                                  ctx.token_pos, ctx.token_seq, kv.block_table, kv.width, kv.page_size, q.p, store ? kv.k : nullptr,
                                  store ? kv.v : nullptr, code_of(act_dtype, "qk_prep"), (int)x.rows, ctx.err, p.q_temp_coef, p.q_temp_every, p.v_first, p.v_first_ld, p.v_lambda,
-                                  p.v_keep, dev.stream()),
+                                  p.v_keep, p.head_norm ? 1 : 0, dev.stream()),
                  "qk_prep");
     return q;
 }
@@ -851,6 +881,7 @@ int gate_act_from_name(const std::string& name) {
     if (name == "relu") return kActRelu;
     if (name == "gelu_tanh") return kActGeluTanh;
     if (name == "swish_clamped") return kActSwishClamped;
+    if (name == "relu_squared") return kActReluSquared;
     return -1;
 }
 
@@ -949,6 +980,106 @@ Mat delta_rule(Device& dev, const Mat& x, const Mat* a, const DeltaRule& p, cons
                                  (float*)st.state, st.elements, st.slots, ctx.cu_q, ctx.token_pos, ctx.token_seq, ctx.seq_lens, (float*)qkv.p,
                                  (float*)g.p, (float*)beta.p, (float*)out.p, ctx.B, ctx.max_q, chunks, dev.stream()),
                  "delta_rule");
+    return out;
+}
+
+Mat token_mix(Device& dev, const Mat& x, const float* mu, int n_mix, const StepView& ctx, const StateView& st, long long prev_off, DType dtype,
+              long long* group_rows) {
+    need(x, "the stream", true, DType::F32);
+    const long long T = x.rows, H = x.cols;
+    if (!st.state || st.dtype != DType::F32 || prev_off < 0 || prev_off + H > st.elements) throw KernelError("token_mix: the cache entry does not hold the previous row");
+    const long long held = dtype == DType::BF16 && T > kLibraryRowBucket ? ceil_div(T, kLibraryRowBucket) * kLibraryRowBucket : T;
+    Mat out = new_mat_exact(dev, n_mix * held, H, dtype);
+    *group_rows = held;
+    check_kernel(illm_token_mix((const float*)x.p, (int)T, (int)H, n_mix, mu, (float*)st.state + prev_off, st.elements, st.slots, ctx.cu_q, ctx.token_seq, ctx.B,
+                                ctx.is_decode ? 1 : 0, out.p, code_of(dtype, "token_mix"), held * H, dev.stream()),
+                 "token_mix");
+    return out;
+}
+
+MatOrPartials group_linear(Device& dev, GemmBackend backend, const Mat& x, long long group_rows, long long M, const Mat& w, const std::vector<int>& n,
+                           bool defer_reduce) {
+    need(x, "x");
+    need(w, "w");
+    const long long K = x.cols, G = (long long)n.size();
+    long long N = 0;
+    for (int v : n) N += v;
+    if (w.cols != K || w.rows != N || w.dtype != x.dtype || x.rows != G * group_rows || group_rows < M)
+        throw KernelError("group_linear: the stacked inputs and weights do not fit the groups");
+    MatOrPartials r;
+    if (M <= 0) {
+        r.m = new_mat_exact(dev, 0, N, DType::F32);
+        return r;
+    }
+    if (x.dtype == DType::F32) {
+        r.m = new_mat_exact(dev, M, N, DType::F32);
+        long long row = 0;
+        for (long long g = 0; g < G; row += n[g++])
+            for (long long m0 = 0; m0 < M; m0 += 65535LL * 64)
+                check_kernel(illm_gemm_f32_nt((const float*)row_ptr(x, g * group_rows + m0), (const float*)row_ptr(w, row), (float*)row_ptr(r.m, m0) + row,
+                                              (int)std::min(M - m0, 65535LL * 64), n[g], (int)K, (int)K, (int)K, (int)N, dev.tc_error_word(), dev.stream()),
+                             "gemm_f32");
+        return r;
+    }
+    need(x, "x", true, DType::BF16);
+    if (M <= 64 && K % 8 == 0 && G <= 8 && backend != GemmBackend::Library) {
+        r.m = new_mat_exact(dev, M, N, DType::F32);
+        const int splits = gemm_tc_splits(M, N, K, dev.n_sms());
+        float* ws = splits > 1 ? dev.alloc_n<float>((size_t)splits * M * N) : nullptr;
+        const bool defer = defer_reduce && splits > 1;
+        check_kernel(illm_gemm_bf16_tc_grouped(x.p, (int)group_rows, w.p, n.data(), (int)G, (float*)r.m.p, (int)M, (int)K, ws, splits, dev.tc_error_word(),
+                                               dev.stream(), defer ? 1 : 0),
+                     "gemm_bf16_tc_grouped");
+        if (defer) {
+            r.part.ws = ws;
+            r.part.splits = splits;
+            r.part.rows = M;
+            r.part.cols = N;
+        }
+        return r;
+    }
+    // whole buckets of rows for the library, as in linear()
+    const long long Mlib = M > kLibraryRowBucket ? std::min(ceil_div(M, kLibraryRowBucket) * kLibraryRowBucket, group_rows) : M;
+    r.m = new_mat_exact(dev, Mlib, N, DType::F32);
+    r.m.rows = M;
+    long long row = 0;
+    for (long long g = 0; g < G;) {
+        long long e = g + 1;
+        while (e < G && n[e] == n[g]) e++;
+        dev.library_gemm_bf16_heads(row_ptr(x, g * group_rows), row_ptr(w, row), (float*)r.m.p + row, (int)Mlib, n[g], (int)K, (int)(e - g), false, (int)K,
+                                    group_rows * K, (int)N, n[g], DType::F32);
+        row += (e - g) * n[g];
+        g = e;
+    }
+    return r;
+}
+
+bool wkv_supported(int d, int dv) { return illm_wkv_supported(d, dv) != 0; }
+
+int wkv_segments(int B, int n_heads, int v_head_dim, int max_q, int n_sms) {
+    const long long blocks = (long long)B * n_heads * ceil_div(v_head_dim, 64);
+    long long P = std::min<long long>(16, (8LL * n_sms) / std::max<long long>(blocks, 1));
+    P = std::min<long long>(P, max_q / 64);
+    return P < 2 ? 1 : (int)P;
+}
+
+Mat wkv_scan(Device& dev, const Mat& y, const WkvScan& p, const StepView& ctx, const StateView& st) {
+    need(y, "the projections", true, DType::F32);
+    const long long HD = (long long)p.n_heads * p.head_dim, HV = (long long)p.n_heads * p.v_head_dim;
+    if (!st.state || st.dtype != DType::F32 || st.elements < HD * p.v_head_dim) throw KernelError("wkv_scan: the cache entry does not hold the state");
+    if (!wkv_supported(p.head_dim, p.v_head_dim)) throw KernelError("wkv_scan: the head size is beyond the kernel (up to 1024)");
+    if (!p.w2 || p.w2->rows != HD || p.w2->cols != p.rank || p.rank <= 0) throw KernelError("wkv_scan: the decay's outer map must be [heads * head size, rank]");
+    if (p.r_off < 0 || p.r_off + HD > y.cols || p.k_off < 0 || p.k_off + HD > y.cols || p.v_off < 0 || p.v_off + HV > y.cols || p.z_off < 0 || p.z_off + p.rank > y.cols)
+        throw KernelError("wkv_scan: the projections do not lie inside the rows");
+    Mat out = new_mat_exact(dev, y.rows, HV, DType::F32);
+    float *w = dev.alloc_n<float>((size_t)y.rows * HD), *bonus = dev.alloc_n<float>((size_t)y.rows * p.n_heads);
+    const int segments = (p.in_order || ctx.is_decode) ? 1 : wkv_segments(ctx.B, p.n_heads, p.v_head_dim, ctx.max_q, dev.n_sms());
+    float* seg_state = segments > 1 ? dev.alloc_n<float>((size_t)ctx.B * segments * HD * p.v_head_dim) : nullptr;
+    float* seg_decay = segments > 1 ? dev.alloc_n<float>((size_t)ctx.B * segments * HD) : nullptr;
+    check_kernel(illm_wkv_scan((const float*)y.p, (int)y.rows, (int)y.cols, p.r_off, p.k_off, p.v_off, p.z_off, p.rank, p.n_heads, p.head_dim, p.v_head_dim,
+                               p.w2->p, code_of(p.w2->dtype, "wkv_scan"), p.w0, p.u, (float*)st.state, st.elements, st.slots, ctx.cu_q, w, bonus, (float*)out.p,
+                               ctx.B, segments, seg_state, seg_decay, dev.stream()),
+                 "wkv_scan");
     return out;
 }
 
@@ -1059,8 +1190,10 @@ Mat moe_forward_ex(Device& dev, const Mat& h, const Mat& logits, const MoeRoutin
     need(h, "h");
     need(logits, "the router's logits", true, DType::F32);
     const long long T = h.rows, D = h.cols;
-    if (logits.rows != T || logits.cols != E || top <= 0 || top > E) throw KernelError("moe: the router's logits must be [T, experts] and top within the experts");
-    if (w_gu.dtype != h.dtype || w_down.dtype != h.dtype || w_gu.cols != D || w_gu.rows % (2 * E) || w_down.cols * 2 * E != w_gu.rows ||
+    const int all = E + r.identity, per = r.plain ? 1 : 2;         // experts the router knows; matrix rows per hidden channel
+    if (r.identity < 0 || logits.rows != T || logits.cols != all || top <= 0 || top > all)
+        throw KernelError("moe: the router's logits must be [T, experts] and top within the experts");
+    if (w_gu.dtype != h.dtype || w_down.dtype != h.dtype || w_gu.cols != D || w_gu.rows % (per * E) || w_down.cols * per * E != w_gu.rows ||
         w_down.rows != (long long)E * D)
         throw KernelError("moe: the experts' matrices do not match the input");
     const long long F = w_down.cols, P = T * top;
@@ -1077,12 +1210,14 @@ Mat moe_forward_ex(Device& dev, const Mat& h, const Mat& logits, const MoeRoutin
     int* tile_expert = dev.alloc_n<int>((size_t)tiles);
     int* tile_row0 = dev.alloc_n<int>((size_t)tiles);
     int* tile_rows = dev.alloc_n<int>((size_t)tiles);
-    if (r.scoring >= 1 && (r.groups < 1 || r.groups > 32 || E % r.groups || r.keep < 1 || r.keep > r.groups || (long long)r.keep * (E / r.groups) < top))
+    if (r.scoring >= 1 && (r.groups < 1 || r.groups > 32 || all % r.groups || r.keep < 1 || r.keep > r.groups || (long long)r.keep * (all / r.groups) < top))
         throw KernelError("moe: the experts must form up to 32 equal groups, and the groups kept must hold at least `top` experts");
     if (r.plus && (r.plus->dtype != DType::F32 || r.plus->rows != T || r.plus->cols != D)) throw KernelError("moe: the addend must be float32 [T, hidden]");
     if (r.scoring < 0 || r.scoring > 2 || r.group_top < 1 || r.group_top > 4) throw KernelError("moe: unknown scoring, or a group score of more than 4 experts");
     if (act == kActSwishClamped && !(r.act_limit > 0.f)) throw KernelError("moe: the clamped activation needs a positive limit");
-    check_kernel(illm_moe_route_ex2((const float*)logits.p, r.bias, (int)T, E, top, bm, r.scoring, r.groups, r.keep, r.renorm ? 1 : 0, r.group_top, r.sum_eps,
+    if (act == kActReluSquared && !r.plain) throw KernelError("moe: the square of relu is an activation of experts without a gate");
+    if (act == kActSwishClamped && r.plain) throw KernelError("moe: the clamped activation needs experts with a gate");
+    check_kernel(illm_moe_route_ex2((const float*)logits.p, r.bias, (int)T, E, r.identity, top, bm, r.scoring, r.groups, r.keep, r.renorm ? 1 : 0, r.group_top, r.sum_eps,
                                     r.weight_scale, expert, weight, row_of_pair, pair_of_row, tile_expert, tile_row0, tile_rows, dev.stream()),
                  "moe_route");
     const int code = code_of(h.dtype, "moe");
@@ -1090,22 +1225,22 @@ Mat moe_forward_ex(Device& dev, const Mat& h, const Mat& logits, const MoeRoutin
     if (tc5) {
         Mat xs = new_mat_exact(dev, P, D, DType::BF16);
         check_kernel(illm_moe_gather_rows(h.p, xs.p, pair_of_row, (int)P, (int)D, top, dev.stream()), "moe_gather_rows");
-        check_kernel(illm_moe_gemm_tc_ex(xs.p, w_gu.p, hid.p, (int)P, E, (int)(2 * F), (int)D, 1, act, r.act_limit, tiles, tile_expert, tile_row0, tile_rows,
+        check_kernel(illm_moe_gemm_tc_ex(xs.p, w_gu.p, hid.p, (int)P, E, (int)(per * F), (int)D, r.plain ? 2 : 1, act, r.act_limit, tiles, tile_expert, tile_row0, tile_rows,
                                       dev.tc_error_word(), dev.stream()),
                      "moe_gemm_tc (gate/up)");
         check_kernel(illm_moe_gemm_tc(hid.p, w_down.p, rows.p, (int)P, E, (int)D, (int)F, 0, 0, tiles, tile_expert, tile_row0, tile_rows,
                                       dev.tc_error_word(), dev.stream()),
                      "moe_gemm_tc (down)");
     } else {
-        check_kernel(illm_moe_gemm_ex(h.p, code, w_gu.p, code, hid.p, (int)T, top, E, (int)(2 * F), (int)D, 1, act, r.act_limit, bm, tc, pair_of_row, tile_expert, tile_row0,
+        check_kernel(illm_moe_gemm_ex(h.p, code, w_gu.p, code, hid.p, (int)T, top, E, (int)(per * F), (int)D, r.plain ? 2 : 1, act, r.act_limit, bm, tc, pair_of_row, tile_expert, tile_row0,
                                    tile_rows, dev.stream()),
                      "moe_gemm (gate/up)");
         check_kernel(illm_moe_gemm(hid.p, code, w_down.p, code, rows.p, (int)T, top, E, (int)D, (int)F, 0, 0, bm, tc, pair_of_row, tile_expert, tile_row0,
                                    tile_rows, dev.stream()),
                      "moe_gemm (down)");
     }
-    check_kernel(illm_moe_combine_plus((const float*)rows.p, row_of_pair, weight, r.plus ? (const float*)r.plus->p : nullptr, (float*)out.p, (int)T, (int)D, top,
-                                       dev.stream()),
+    check_kernel(illm_moe_combine_ex((const float*)rows.p, row_of_pair, weight, r.plus ? (const float*)r.plus->p : nullptr, r.identity ? h.p : nullptr, code,
+                                     (float*)out.p, (int)T, (int)D, top, dev.stream()),
                  "moe_combine");
     return out;
 }

@@ -9,6 +9,7 @@
 #pragma once
 #include <cstdint>
 #include <string>
+#include <vector>
 
 #include "cache/cache.h"
 #include "device/device.h"
@@ -235,6 +236,12 @@ Mat attention(Device& dev, const Mat& qkv, const KVView& kv, const StepView& ctx
 // in `out_dtype` as well (what the next sublayer reads).
 Mat scale_add_rmsnorm(Device& dev, const Mat& resid, const MatOrPartials* delta, const Mat& weight_f32, float alpha, float eps, DType out_dtype);
 
+// stream.x += rmsnorm(y) * w (w float32, y a float32 matrix or unreduced slices, added up by the kernel): a sublayer's output
+// normed on its way into the stream.  With want_rows the new rows come back in `out_dtype`, else an empty matrix.
+Mat join_rmsnorm(Device& dev, const Mat& resid, const MatOrPartials& y, const Mat& weight_f32, float eps, DType out_dtype, bool want_rows);
+// The embedding's rows through an RMS norm with a float32 weight: the float32 stream, and (bfloat16 mode) its rows in `dtype` in *rows.
+Mat embedding_normed(Device& dev, const StepView& ctx, const Mat& table, const Mat& weight_f32, float eps, DType dtype, Mat* rows);
+
 // Between the packed projection x [T, ld] (float32 or the activation dtype) of an attention layer and its attention kernel:
 // optional biases, optional RMS norms over a token's whole q and whole k projection, rotation of the
 // first `rot_dim` channels of every head (interleaved pairs or rotate-half) from a (cos, sin) table,
@@ -243,6 +250,7 @@ struct QkPrep {
     int q_off = 0, k_off = -1, v_off = -1;
     const float *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr;
     const float *q_norm = nullptr, *k_norm = nullptr;
+    bool head_norm = false;     // the norms are over every head by itself, their weights of one head's size
     float eps = 0.f;
     const float* cos_sin = nullptr;
     int rot_dim = 0;
@@ -328,7 +336,8 @@ Mat group_norm_gate(Device& dev, const Mat& o_f32, int group, const float* w, fl
 
 // Activations of the gated feed-forward: act(gate) * up.
 // kActSwishClamped: g = min(gate, limit), u = clamp(up, -limit, limit); g sigmoid(1.702 g) (u + 1)
-enum GateAct { kActSilu = 1, kActRelu = 2, kActGeluTanh = 3, kActSwishClamped = 4 };
+// kActReluSquared: for experts without a gate only (max(x, 0)^2)
+enum GateAct { kActSilu = 1, kActRelu = 2, kActGeluTanh = 3, kActSwishClamped = 4, kActReluSquared = 5 };
 int gate_act_from_name(const std::string& name);        // ConfigError-free: -1 for an unknown name
 // resid += d1 (+ d2), all float32 [T, H], and the RMS norm of the new rows times w (float32 [H]) in `out_dtype`: one kernel
 Mat add2_rmsnorm(Device& dev, const Mat& resid, const Mat& d1, const Mat* d2, const Mat& weight_f32, float eps, DType out_dtype);
@@ -368,6 +377,33 @@ constexpr int kDeltaChunkMinTokens = 16;      // the most tokens of a sequence i
 long long delta_rule_state_elements(int n_heads, int n_kv_heads, int head_dim, int v_head_dim, int taps);
 bool delta_rule_supported(int head_dim, int v_head_dim, int taps);
 Mat delta_rule(Device& dev, const Mat& x_f32, const Mat* a_f32, const DeltaRule& p, const StepView& ctx, const StateView& st);
+
+// Blends of every token's row and the one before it, x + (x' - x) * mu_s, for s = 0 .. n_mix - 1 (csrc/wkv_state.cu): x float32
+// [T, H], mu float32 [n_mix, H]; the rows before a step's first tokens are `width` floats at `prev_off` of the slot's elements,
+// which are renewed.  Returns the n_mix matrices stacked, [n_mix * rows_held of one, H] in `dtype`; *group_rows gets the rows
+// from one to the next.
+Mat token_mix(Device& dev, const Mat& x_f32, const float* mu, int n_mix, const StepView& ctx, const StateView& st, long long prev_off, DType dtype,
+              long long* group_rows);
+// Products with inputs of their own, side by side: group g's inputs are rows [g * group_rows, g * group_rows + M) of x, its
+// weights the next n[g] rows of w, its outputs the next n[g] columns of the float32 result [M, sum of n].  Up to 64 rows in
+// bfloat16 in one launch of gemm_tc.cu (the result may then come back as unreduced slices), more rows through the library (equal
+// groups that follow one another as one batched product), float32 on the plain kernels.
+MatOrPartials group_linear(Device& dev, GemmBackend backend, const Mat& x, long long group_rows, long long M, const Mat& w, const std::vector<int>& n,
+                           bool defer_reduce);
+// The recurrence with a decay per head and key channel made by the token itself, and a bonus for the token's own contribution
+// (csrc/wkv_state.cu).  y: float32 [T, ld] with r, k, v and the decay's inner products z (rank columns) at their offsets;
+// w2 [heads * d, rank]; w0, u float32 [heads * d].  The state S [heads, dv, d] stands at the start of the slot's elements.
+// Returns float32 [T, heads * v_head_dim].  in_order as in DecayScan.
+struct WkvScan {
+    int r_off = 0, k_off = 0, v_off = 0, z_off = 0, rank = 0;
+    int n_heads = 0, head_dim = 0, v_head_dim = 0;
+    const Mat* w2 = nullptr;
+    const float *w0 = nullptr, *u = nullptr;
+    bool in_order = true;
+};
+bool wkv_supported(int head_dim, int v_head_dim);
+int wkv_segments(int B, int n_heads, int v_head_dim, int max_q, int n_sms);
+Mat wkv_scan(Device& dev, const Mat& y_f32, const WkvScan& p, const StepView& ctx, const StateView& st);
 
 // Attention through latents (csrc/latent_attention.cu): the two norms and the cache write; returns the normed
 // query latent [T, q_rank] in `act_dtype`.  kv: a keys-only entry of one head of kv_rank channels.
@@ -423,6 +459,11 @@ struct MoeRouting {
     bool renorm = true;
     const float* bias = nullptr;
     const Mat* plus = nullptr;
+    // experts beyond those with matrices that the router can choose and whose output is their input (the logits have
+    // experts + identity columns, the identity experts last)
+    int identity = 0;
+    // experts without a gate: w_gate_up is [experts * ff, hidden], a row per output, and the activation is applied to it
+    bool plain = false;
 };
 Mat moe_forward_ex(Device& dev, const Mat& h, const Mat& logits_f32, const MoeRouting& r, int experts, int top, const Mat& w_gate_up,
                    const Mat& w_down, int act);

@@ -77,6 +77,13 @@ std::map<int, CacheRequest> DecoderModel::cache_requests() const {
             if (aux.kind == CacheRequest::FixedState) out[kAuxCacheEntryBase + e.cache] = aux;
             else if (aux.kind != CacheRequest::None) throw ConfigError("a mixer's second cache entry must be fixed state");
         }
+    // an entry that other layers read too keeps what the farthest-reaching of them sees (those mask for themselves)
+    for (const ScheduleEntry& e : spec.schedule) {
+        if (e.writes) continue;
+        const Mixer::Reach r = layers_[(size_t)e.layer].mixer->reach();
+        auto it = out.find(e.cache);
+        if (r.known && it != out.end() && it->second.kind == CacheRequest::PagedKV) it->second = it->second.reaching(r.window, r.chunk);
+    }
     const CacheRequest er = embedding_->cache_request();
     if (er.kind != CacheRequest::None) out[kEmbeddingCacheEntry] = er;
     return out;

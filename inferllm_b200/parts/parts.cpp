@@ -9,6 +9,7 @@ void register_delta_parts(std::map<std::string, PartFactory<Mixer>>& mixers);   
 void register_latent_parts(std::map<std::string, PartFactory<Mixer>>& mixers);     // parts/latent_mixer.cpp
 void register_routed_parts(std::map<std::string, PartFactory<FeedForward>>& ffs);  // parts/routed_mlp.cpp
 void register_gated_state_parts(std::map<std::string, PartFactory<Mixer>>& mixers);   // parts/gated_mixers.cpp
+void register_wkv_parts(std::map<std::string, PartFactory<Mixer>>& mixers);           // parts/wkv_mixer.cpp
 void register_sandwich_parts(std::map<std::string, PartFactory<Norm>>& norms, std::map<std::string, PartFactory<Mixer>>& mixers,
                              std::map<std::string, BlockKind>& blocks);               // parts/sandwich.cpp
 
@@ -119,6 +120,21 @@ std::vector<double> rotary_frequencies(double theta, int rot_dim, const Json* sc
         if (!scaling->has(key) || !scaling->at(key).is_number()) throw ConfigError(std::string("rotary scaling: '") + key + "' must be a number");
         return scaling->at(key).as_double();
     };
+    if (scaling->has("low") || scaling->has("high")) {
+        const double factor = num("factor"), original = num("original"), low = num("low"), high = num("high");
+        if (!(factor > 0) || !(original > 0) || !(low > 0) || !(high > 0)) throw ConfigError("rotary scaling: all four numbers must be positive");
+        for (double& v : f) {
+            const double wave = 2.0 * M_PI / v;
+            if (wave < original / high) continue;
+            if (wave > original / low) {
+                v /= factor;
+            } else {
+                const double s = high > low ? (original / wave - low) / (high - low) : 1.0;
+                v = (1.0 - s) * v / factor + s * v;
+            }
+        }
+        return f;
+    }
     const double factor = num("factor"), original = num("original"), fast = num("fast"), slow = num("slow");
     if (!(factor > 0) || !(original > 0) || !(fast > 0) || !(slow > 0)) throw ConfigError("rotary scaling: all four numbers must be positive");
     // the (real-valued) pair index whose wave turns `turns` times within `original` positions
@@ -232,9 +248,22 @@ struct RMSNorm : Norm {
         ops::norm_sandwich(*rt->dev, stream.x, &y, &weight.m, nullptr, eps, DType::F32, nullptr, 0, false, post_scale);
         stream.has_pending = false;
     }
+    Mat join_stream(ResidualStream& stream, bool want_rows) override {
+        if (stream.has_pending2 || post_scale != 1.f || weight.m.dtype != DType::F32)
+            throw EngineError("rmsnorm: only one addition, with a float32 weight and no factor, joins the stream this way");
+        const bool copy = want_rows && rt->dtype != DType::F32;
+        Mat h = ops::join_rmsnorm(*rt->dev, stream.x, stream.pending, weight.m, eps, copy ? rt->dtype : DType::F32, copy);
+        stream.has_pending = false;
+        stream.pending_post = nullptr;
+        return want_rows && !copy ? stream.x : h;
+    }
     Mat forward(ResidualStream& stream, const int* rows, long long n_rows) override {
         // an addition that passes an RMS norm of its own on its way into the stream: both norms in one kernel
         if (RMSNorm* post = stream.has_pending && !stream.has_pending2 ? dynamic_cast<RMSNorm*>(stream.pending_post) : nullptr) {
+            if (stream.pending.is_partials() && rows != nullptr) {
+                stream.pending.m = ops::materialize(*rt->dev, stream.pending.part, DType::F32);
+                stream.pending.part = Partials();
+            }
             if (!stream.pending.is_partials() && stream.pending.m.dtype == DType::F32 && post->eps == eps && post->weight.m.dtype == DType::F32 &&
                 weight.m.dtype == DType::F32) {
                 Mat y = ops::norm_sandwich(*rt->dev, stream.x, &stream.pending.m, &post->weight.m, &weight.m, eps, rt->dtype, rows, n_rows, false,
@@ -304,8 +333,8 @@ struct LayerScale : Norm {
 // writes K and V into the cache.  theta (fixed to 10000 in the reference) and rot_dim are parameters.
 //
 // "rope_pairs" is the same rotation with channel 2j paired with 2j + 1 (the interleaved layout).  Both
-// take an optional `scaling` {factor, original, fast, slow}: the frequencies are blended with the
-// stretched ones and cos and sin carry a magnitude factor (rotary_frequencies).
+// take an optional `scaling`, {factor, original, fast, slow} or {factor, original, low, high}: the frequencies are blended
+// with the stretched ones and, in the first form, cos and sin carry a magnitude factor (rotary_frequencies).
 struct RopeTable : PositionEncoding {
     int head_dim, rot_dim;
     double theta, magnitude = 1.0;
@@ -382,7 +411,8 @@ struct NoPosition : PositionEncoding {
 // Options beyond the reference's attention, each a parameter that is off unless given: `v_head_dim`
 // (values of another size than keys), `qkv_bias` (biases on the three projections), `qk_norm` =
 // "projection" (an RMS norm with a weight over the token's whole q projection, all heads together, and
-// likewise over k, before the rotation; `norm_eps`), `sink` (one learned number per head whose
+// likewise over k, before the rotation; `norm_eps`) or "head" (an RMS norm over every head's q and every head's k, with one
+// weight of a head's size shared by all heads), `sink` (one learned number per head whose
 // exponential joins the softmax denominator without a value), `out_gate` = "head_sigmoid" (a
 // projection of the mixer's input to one number per head; the head's output is multiplied by its
 // sigmoid before the output projection), `own_kv` = false (the layer has no key and value
@@ -427,7 +457,7 @@ struct Attention : Mixer {
     int q_temp_every = 0;
     int chunk = 0;
     float softcap = 0.f;
-    bool unit_sink = false, keeps_values = false, mixes_values = false;
+    bool unit_sink = false, keeps_values = false, mixes_values = false, head_norm = false;
     std::map<std::string, std::string> names;
     std::unique_ptr<PositionEncoding> position;
     DeviceBuffer qkv_buf, o_buf;
@@ -446,7 +476,8 @@ struct Attention : Mixer {
             throw ConfigError("attention: sizes must be positive");
         if (n_heads % n_kv_heads) throw ConfigError("attention: n_heads must be a multiple of n_kv_heads");
         const std::string qn = s.get_string("qk_norm", "none"), og = s.get_string("out_gate", "none");
-        if (qn != "none" && qn != "projection") throw ConfigError("attention: qk_norm '" + qn + "' is not supported (none, projection)");
+        if (qn != "none" && qn != "projection" && qn != "head") throw ConfigError("attention: qk_norm '" + qn + "' is not supported (none, projection, head)");
+        head_norm = qn == "head";
         if (og != "none" && og != "head_sigmoid" && og != "sigmoid")
             throw ConfigError("attention: out_gate '" + og + "' is not supported (none, head_sigmoid, sigmoid)");
         const std::string vs = s.get_string("values", "own"), db = s.get_string("distance_bias", "none");
@@ -454,14 +485,14 @@ struct Attention : Mixer {
         if (db != "none" && db != "log1p") throw ConfigError("attention: distance_bias '" + db + "' is not supported (none, log1p)");
         if ((log_distance || head_mix) && !values_are_keys)
             throw ConfigError("attention: distance_bias and head_mix run on the kernel for values = keys only");
-        if (values_are_keys && (v_head_dim != head_dim || !own_kv || qkv_bias || proj_norm || has_sink || has_gate))
+        if (values_are_keys && (v_head_dim != head_dim || !own_kv || qkv_bias || proj_norm || head_norm || has_sink || has_gate))
             throw ConfigError("attention: values = keys needs key and value heads of one size and takes no biases, projection norms, sinks or head gates");
         maps = (int)s.get_int("score_maps", 1);
         o_bias = s.get_bool("o_bias", false);
         if (maps != 1 && maps != 2) throw ConfigError("attention: score_maps must be 1 or 2");
         if (maps == 2) {
             diff = (float)s.get_double("diff");
-            if (values_are_keys || has_sink || has_gate || !own_kv)
+            if (values_are_keys || has_sink || has_gate || head_norm || !own_kv)
                 throw ConfigError("attention: two score maps take no sinks and no head gates, and need keys and values of their own");
         }
         if (s.has("q_temperature")) {
@@ -507,7 +538,7 @@ struct Attention : Mixer {
     }
     // true if the layer needs the general path (see above)
     bool general() const {
-        return v_head_dim != head_dim || qkv_bias || proj_norm || has_sink || has_gate || !own_kv || out_f32 || maps == 2 || q_temp_every > 0 || o_bias ||
+        return v_head_dim != head_dim || qkv_bias || proj_norm || head_norm || has_sink || has_gate || !own_kv || out_f32 || maps == 2 || q_temp_every > 0 || o_bias ||
                chunk > 0 || softcap > 0.f || unit_sink || keeps_values || mixes_values || wide_gate;
     }
     long long gate_rows() const { return has_gate ? n_heads : wide_gate ? (long long)n_heads * v_head_dim : 0; }
@@ -534,9 +565,9 @@ struct Attention : Mixer {
             if (!values_are_keys) d.push_back({nm("v"), TensorDecl{{v, hidden}}});
             if (qkv_bias) d.push_back({nm("v_bias"), TensorDecl{{v}}});
         }
-        if (proj_norm) {
-            d.push_back({nm("q_norm"), TensorDecl{{q}, "norm"}});
-            if (own_kv) d.push_back({nm("k_norm"), TensorDecl{{k}, "norm"}});
+        if (proj_norm || head_norm) {
+            d.push_back({nm("q_norm"), TensorDecl{{head_norm ? (long long)head_dim : q}, "norm"}});
+            if (own_kv) d.push_back({nm("k_norm"), TensorDecl{{head_norm ? (long long)head_dim : k}, "norm"}});
         }
         if (has_sink) d.push_back({nm("sink"), TensorDecl{{(long long)n_heads}}});
         if (has_gate || wide_gate) d.push_back({nm("gate"), TensorDecl{{gate_rows(), hidden}}});
@@ -580,7 +611,7 @@ struct Attention : Mixer {
                 b_v = fetch_owned(rt, src, names.at("v_bias"), DType::F32, "an attention bias");
             }
         }
-        if (proj_norm) {
+        if (proj_norm || head_norm) {
             n_q = fetch_owned(rt, src, names.at("q_norm"), DType::F32, "a projection norm's weight");
             if (own_kv) n_k = fetch_owned(rt, src, names.at("k_norm"), DType::F32, "a projection norm's weight");
         }
@@ -618,6 +649,14 @@ struct Attention : Mixer {
     CacheRequest cache_request() const override {
         if (values_are_keys) return CacheRequest::paged_keys_only(n_kv_heads, head_dim, window);
         return own_kv ? CacheRequest::paged(n_kv_heads, maps * head_dim, window, v_head_dim).in_chunks(chunk) : CacheRequest();
+    }
+
+    Reach reach() const override {
+        Reach r;
+        r.known = true;
+        r.window = window;
+        r.chunk = chunk;
+        return r;
     }
 
     // values = keys: one float32 product for q, k and the gate; q out and k into the pages (with the table rotation,
@@ -671,6 +710,7 @@ struct Attention : Mixer {
         p.v_bias = (const float*)b_v.m.p;
         p.q_norm = (const float*)n_q.m.p;
         p.k_norm = (const float*)n_k.m.p;
+        p.head_norm = head_norm;
         p.eps = norm_eps;
         const float* table = nullptr;
         int rot = 0;
@@ -726,6 +766,9 @@ struct Attention : Mixer {
         Device& dev = *rt->dev;
         KVView kv = cache.kv;
         kv.writes = writes;
+        // the mask is this layer's own: the cache entry may keep more positions, for other layers that read it
+        kv.window = window;
+        kv.chunk = chunk;
         if (values_are_keys) return forward_mixed(h, ctx, kv, may_defer);
         if (general()) return forward_general(h, ctx, kv, may_defer);
         const ops::Geometry g{n_heads, n_kv_heads, head_dim};
@@ -770,7 +813,7 @@ struct GatedMLP : FeedForward {
             : FeedForward(s, rt), hidden(s.get_int("hidden_size")), inter(s.get_int("intermediate_size")),
               out_f32(s.get_string("output_dtype", "compute") == "float32") {
         act = ops::gate_act_from_name(s.get_string("activation", "silu"));
-        if (act < 0) throw ConfigError("gated_mlp: activation '" + s.get_string("activation", "silu") + "' is not supported (silu, relu, gelu_tanh, swish_clamped)");
+        if (act < 0 || act == ops::kActReluSquared) throw ConfigError("gated_mlp: activation '" + s.get_string("activation", "silu") + "' is not supported (silu, relu, gelu_tanh, swish_clamped)");
         act_limit = (float)s.get_double("activation_limit", 0.0);
         if (act == ops::kActSwishClamped && !(act_limit > 0.f)) throw ConfigError("gated_mlp: swish_clamped needs a positive activation_limit");
         if (hidden <= 0 || inter <= 0) throw ConfigError("gated_mlp: sizes must be positive");
@@ -805,21 +848,35 @@ struct GatedMLP : FeedForward {
 // written as the float32 residual stream.
 // Two parameters beyond the gather: `scale` (the row times a constant) and `sinusoid_base` (a position vector is added:
 // entry 2i is sin(p base^(-2i / hidden)) and entry 2i + 1 the cosine of the same angle; the frequencies are made in
-// float64 once, angle and functions are float32).  A tied head still reads the table itself, without the scale.
+// float64 once, angle and functions are float32).  A third, `norm` {tensor, eps}: the row passes an RMS norm with a weight
+// (float32) on its way into the stream, without the other two.  A tied head still reads the table itself.
 struct Embedding : EmbeddingPart {
     long long vocab, hidden;
     std::string tensor;         // the table's name below the part's prefix
-    double scale, sinusoid_base;
-    OwnedMat weight;
+    double scale, sinusoid_base, norm_eps = 0.0;
+    std::string norm_tensor;    // empty: no norm
+    OwnedMat weight, norm_w;
     DeviceBuffer freq_buf;
     Embedding(const PartSpec& s, Runtime* rt)
             : EmbeddingPart(s, rt), vocab(s.get_int("vocab_size")), hidden(s.get_int("hidden_size")), tensor(s.get_string("tensor", "weight")),
               scale(s.get_double("scale", 1.0)), sinusoid_base(s.get_double("sinusoid_base", 0.0)) {
         if (sinusoid_base < 0 || (s.has("sinusoid_base") && !(sinusoid_base > 0))) throw ConfigError("embedding: sinusoid_base must be positive");
+        if (s.has("norm")) {
+            const PartSpec n("embedding's norm", s.params.at("norm"));
+            norm_tensor = n.get_string("tensor", "norm.weight");
+            norm_eps = n.get_double("eps");
+            if (!(norm_eps > 0)) throw ConfigError("embedding: the norm's eps must be positive");
+            if (scale != 1.0 || sinusoid_base > 0) throw ConfigError("embedding: the norm goes with neither scale nor sinusoid_base");
+        }
     }
-    TensorDecls tensors() const override { return {{tensor, TensorDecl{{vocab, hidden}}}}; }
+    TensorDecls tensors() const override {
+        TensorDecls d = {{tensor, TensorDecl{{vocab, hidden}}}};
+        if (!norm_tensor.empty()) d.push_back({norm_tensor, TensorDecl{{hidden}, "norm"}});
+        return d;
+    }
     void load(TensorSource& src) override {
         weight = fetch_owned(rt, src, tensor, rt->dtype, "the embedding table");
+        if (!norm_tensor.empty()) norm_w = fetch_owned(rt, src, norm_tensor, DType::F32, "the embedding's norm weight");
         if (sinusoid_base > 0) {
             std::vector<float> f((size_t)(hidden + 1) / 2);
             for (size_t i = 0; i < f.size(); i++) f[i] = (float)std::pow(sinusoid_base, -2.0 * (double)i / (double)hidden);
@@ -831,7 +888,9 @@ struct Embedding : EmbeddingPart {
     ResidualStream forward(const StepContext& ctx) override {
         ResidualStream s;
         s.dev = rt->dev;
-        if (scale != 1.0 || sinusoid_base > 0)
+        if (!norm_tensor.empty())
+            s.x = ops::embedding_normed(*rt->dev, ctx, weight.m, norm_w.m, (float)norm_eps, rt->dtype, &s.h);
+        else if (scale != 1.0 || sinusoid_base > 0)
             s.x = ops::embedding_scaled(*rt->dev, ctx, weight.m, (float)scale, (const float*)freq_buf.get());
         else
             s.x = ops::embedding(*rt->dev, ctx.ids, ctx.T, weight.m, ctx.err);
@@ -986,6 +1045,33 @@ struct PostNormBlock : Block {
     }
 };
 
+// "outnorm": a norm on every sublayer's output and none in front; the sublayers read the stream as it is:
+//     x = x + norm1(mixer(x));  x = x + norm2(ffn(x))
+// ("outnorm_mixer": without the feed-forward.)  One kernel norms a sublayer's output (which may come as unreduced K slices)
+// into the float32 stream and leaves the new rows in the compute dtype for the sublayer that reads them next; a mixer that
+// asks for it (reads_stream) gets the float32 stream itself.
+struct OutNormBlock : Block {
+    // the stream's rows with everything pending folded in; in the compute dtype if `want`
+    static Mat rows(ResidualStream& stream, DType dtype, bool want) {
+        if (stream.has_pending && stream.pending_post && !stream.has_pending2) {
+            stream.h = stream.pending_post->join_stream(stream, want);
+        } else if (stream.has_pending || stream.has_pending2) {
+            stream.flush();
+            stream.h = Mat();
+        }
+        if (want && !stream.h.p) stream.h = ops::cast(*stream.dev, stream.x, dtype);
+        return stream.h;
+    }
+    void forward(ResidualStream& stream, const StepContext& ctx, const CacheView& cache, bool writes) override {
+        const bool as_is = mixer->reads_stream();
+        Mat h = rows(stream, ctx.rt->dtype, !as_is);
+        stream.add_normed(mixer->forward(as_is ? stream.x : h, ctx, cache, writes, true), norms.at("norm1"));
+        if (!ffn) return;
+        h = rows(stream, ctx.rt->dtype, true);
+        stream.add_normed(ffn->forward(h, ctx, true), norms.at("norm2"));
+    }
+};
+
 // "parallel": one norm, and both sublayers read its output:
 //     h = norm1(x);  x = x + mixer(h) + ffn(h)
 // (a layer without a feed-forward adds the mixer alone).  The sublayers' outputs stay pending in the stream, and the next
@@ -1005,10 +1091,13 @@ void register_builtin_parts() {
     register_latent_parts(reg<Mixer>());
     register_routed_parts(reg<FeedForward>());
     register_gated_state_parts(reg<Mixer>());
+    register_wkv_parts(reg<Mixer>());
     register_sandwich_parts(reg<Norm>(), reg<Mixer>(), block_reg());
     block_reg()["parallel"] = BlockKind{{"norm1"}, [] { return std::unique_ptr<Block>(new ParallelBlock); }};
     reg<FeedForward>()["linear"] = [](const PartSpec& s, Runtime* rt) { return std::unique_ptr<FeedForward>(new LinearMap(s, rt)); };
     reg<EmbeddingPart>()["bigram_embedding"] = [](const PartSpec& s, Runtime* rt) { return std::unique_ptr<EmbeddingPart>(new BigramEmbedding(s, rt)); };
+    block_reg()["outnorm"] = BlockKind{{"norm1", "norm2"}, [] { return std::unique_ptr<Block>(new OutNormBlock); }};
+    block_reg()["outnorm_mixer"] = BlockKind{{"norm1"}, [] { return std::unique_ptr<Block>(new OutNormBlock); }};
     block_reg()["postnorm"] = BlockKind{{"norm1", "norm2"}, [] { return std::unique_ptr<Block>(new PostNormBlock); }};
     block_reg()["postnorm_mixer"] = BlockKind{{"norm1", "norm2"}, [] { return std::unique_ptr<Block>(new PostNormBlock); }};
     reg<Norm>()["rmsnorm"] = [](const PartSpec& s, Runtime* rt) { return std::unique_ptr<Norm>(new RMSNorm(s, rt)); };

@@ -193,6 +193,9 @@ public:
     // stream.x += norm(stream.pending), for the norm a sublayer's output passes before it joins the stream
     // (ResidualStream::add_normed); only norms that can stand there override it.
     virtual void add_normed_pending(ResidualStream& stream) { throw EngineError("norm '" + spec.kind + "' cannot norm a sublayer's output into the stream"); }
+    // The same, and the new rows of the stream in the compute dtype, for a block whose sublayers read the stream as it is
+    // (nothing comes back unless `want_rows`; in the float32 mode it is the stream itself).
+    virtual Mat join_stream(ResidualStream& stream, bool want_rows) { throw EngineError("norm '" + spec.kind + "' cannot norm a sublayer's output into the stream"); }
     // A part that stands behind a sublayer and is nothing but a factor per channel (a layer scale) gives its float32
     // factors [size] here, so that the next norm can fold x + factors * pending into its own kernel.
     virtual const Mat* channel_scale() const { return nullptr; }
@@ -254,6 +257,13 @@ public:
     // A second cache entry, of fixed per-sequence state, beside the first (a mixer with keys and values AND a few
     // rows of state, say): the decoder gives it an entry number of its own and hands it over as CacheView::aux.
     virtual CacheRequest aux_cache_request() const { return CacheRequest(); }
+    // Which earlier positions the mixer's queries see (0, 0: all; as in CacheRequest), for a mixer that attends to keys and
+    // values which another layer wrote: the cache keeps every position that one of the entry's readers still needs.
+    struct Reach { bool known = false; int window = 0, chunk = 0; };
+    virtual Reach reach() const { return Reach(); }
+    // true: in a block whose sublayers read the stream as it is, forward() gets the float32 stream instead of its rows in
+    // the compute dtype
+    virtual bool reads_stream() const { return false; }
     // h [T, H] in the compute dtype -> [T, H].  `may_defer`: the result may be the unreduced slices of
     // a split matrix product, for a caller that only adds it to the residual stream.
     virtual MatOrPartials forward(const Mat& h, const StepContext& ctx, const CacheView& cache, bool writes, bool may_defer) = 0;
@@ -334,10 +344,13 @@ struct PositionTable {
 std::shared_ptr<PositionTable> shared_position_table(Runtime* rt, double theta, int rot_dim, long long positions);
 // The general form: entry (p, j) = magnitude * (cos, sin)(p * freqs[j]), freqs of rot_dim / 2 pairs.
 std::shared_ptr<PositionTable> shared_position_table(Runtime* rt, const std::vector<double>& freqs, double magnitude, long long positions);
-// Frequencies theta^(-2j / rot_dim), optionally blended with the ones stretched by `factor` along a
-// linear ramp over the pair index (the "YaRN" scaling: pairs that turn more than `fast` times within
-// `original` positions keep their frequency, pairs that turn less than `slow` times are stretched);
-// *magnitude gets the factor 0.1 ln(factor) + 1 that goes with it (1 without scaling).
+// Frequencies theta^(-2j / rot_dim), optionally blended with the ones stretched by `factor`: along a
+// linear ramp over the pair index (the "YaRN" scaling {factor, original, fast, slow}: pairs that turn more than `fast` times
+// within `original` positions keep their frequency, pairs that turn less than `slow` times are stretched;
+// *magnitude gets the factor 0.1 ln(factor) + 1 that goes with it), or along a ramp over the turns themselves (the scaling of
+// Llama 3.1, {factor, original, low, high}: pairs that turn more than `high` times within `original` positions keep their
+// frequency, pairs that turn less than `low` times are stretched, linear in the number of turns between; *magnitude is 1, as
+// it is without scaling).
 std::vector<double> rotary_frequencies(double theta, int rot_dim, const Json* scaling, double* magnitude);
 
 }  // namespace illm

@@ -23,6 +23,10 @@
 // choice scores; 1 if not given), `weight_scale` (the weights are multiplied by it at the end) and `sum_eps` (added to the
 // sum the weights are divided by).  And one more activation of the experts, "swish_clamped" with `activation_limit` L:
 // g = min(W_gate h, L), u = clamp(W_up h, -L, L), y = g sigmoid(1.702 g) (u + 1).
+//
+// Two more parameters: `expert_kind` = "plain" (experts without a gate, y = W_down act(W_up h); activations silu, relu,
+// gelu_tanh and "relu_squared", max(z, 0)^2) and `identity_experts` I (the router has I outputs more than there are experts
+// with matrices; the last I are experts whose output is their input h, and which have no tensors).
 #include "parts/parts.h"
 
 namespace illm {
@@ -33,7 +37,8 @@ struct RoutedMLP : FeedForward {
     long long hidden, inter;
     int experts, top, act;
     bool has_bias;
-    bool score_all, score_sigmoid, has_correction, renorm;
+    bool score_all, score_sigmoid, has_correction, renorm, plain;
+    int identity;
     int groups = 1, keep = 1, group_top = 1;
     float weight_scale = 1.f, sum_eps = 0.f, act_limit = 0.f;
     std::unique_ptr<FeedForward> shared;
@@ -49,11 +54,15 @@ struct RoutedMLP : FeedForward {
               top((int)s.get_int("top")), act(ops::gate_act_from_name(s.get_string("activation", "silu"))), has_bias(s.get_bool("router_bias", false)),
               score_all(s.get_string("scoring", "softmax_chosen") == "softmax_all"), score_sigmoid(s.get_string("scoring", "softmax_chosen") == "sigmoid"),
               has_correction(s.get_bool("choice_correction", false)),
-              renorm(s.get_bool("renormalize", false)), shared_prefix(s.get_string("shared_prefix", "shared.")) {
+              renorm(s.get_bool("renormalize", false)), plain(s.get_string("expert_kind", "gated") == "plain"), identity((int)s.get_int("identity_experts", 0)),
+              shared_prefix(s.get_string("shared_prefix", "shared.")) {
         const std::string sc = s.get_string("scoring", "softmax_chosen");
         if (sc != "softmax_chosen" && sc != "softmax_all" && sc != "sigmoid")
             throw ConfigError("routed_mlp: scoring '" + sc + "' is not supported (softmax_chosen, softmax_all, sigmoid)");
         const bool scored = score_all || score_sigmoid;
+        if (!plain && s.get_string("expert_kind", "gated") != "gated")
+            throw ConfigError("routed_mlp: expert_kind '" + s.get_string("expert_kind", "") + "' is not supported (gated, plain)");
+        if (identity < 0) throw ConfigError("routed_mlp: identity_experts must not be negative");
         if (!scored && (has_correction || s.has("groups") || s.has("group_score_top") || s.has("weight_scale") || s.has("sum_eps")))
             throw ConfigError("routed_mlp: a choice correction, groups, weight_scale and sum_eps need scoring = softmax_all or sigmoid");
         if (scored && has_bias) throw ConfigError("routed_mlp: scoring = " + sc + " takes a choice correction, not a router bias");
@@ -71,8 +80,7 @@ struct RoutedMLP : FeedForward {
                 throw ConfigError("routed_mlp: groups must be {count, keep}");
             groups = (int)g.at("count").as_int();
             keep = (int)g.at("keep").as_int();
-            if (groups < 1 || groups > 32 || s.get_int("experts") % groups || keep < 1 || keep > groups ||
-                (long long)keep * (s.get_int("experts") / groups) < s.get_int("top"))
+            if (groups < 1 || groups > 32 || all() % groups || keep < 1 || keep > groups || (long long)keep * (all() / groups) < top)
                 throw ConfigError("routed_mlp: the experts must form 1 to 32 equal groups, and the groups kept must hold at least `top` experts");
         }
         if (s.has("shared")) {
@@ -81,21 +89,24 @@ struct RoutedMLP : FeedForward {
             sh.params.set("output_dtype", std::string("float32"));
             shared = build_feed_forward(sh, rt);
         }
-        if (hidden <= 0 || inter <= 0 || experts <= 0 || top <= 0 || top > experts)
+        if (hidden <= 0 || inter <= 0 || experts <= 0 || top <= 0 || top > all())
             throw ConfigError("routed_mlp: sizes must be positive and top at most the number of experts");
-        if (act < 0) throw ConfigError("routed_mlp: activation '" + s.get_string("activation", "silu") + "' is not supported (silu, relu, gelu_tanh, swish_clamped)");
+        if (act < 0 || (act == ops::kActReluSquared && !plain) || (act == ops::kActSwishClamped && plain))
+            throw ConfigError("routed_mlp: activation '" + s.get_string("activation", "silu") +
+                              "' is not supported (silu, relu, gelu_tanh, swish_clamped; without a gate silu, relu, gelu_tanh, relu_squared)");
         names = {{"router", "router.weight"}, {"router_bias", "router.bias"}, {"correction", "correction"}, {"expert", "experts."}, {"gate", "gate_proj.weight"},
                  {"up", "up_proj.weight"}, {"down", "down_proj.weight"}};
         if (s.has("names"))
             for (auto& m : s.params.at("names").members()) names[m.first] = m.second.as_string();
     }
+    int all() const { return experts + identity; }          // what the router chooses from
     std::string expert_tensor(int e, const char* role) const { return names.at("expert") + std::to_string(e) + "." + names.at(role); }
     TensorDecls tensors() const override {
-        TensorDecls d = {{names.at("router"), TensorDecl{{(long long)experts, hidden}}}};
-        if (has_bias) d.push_back({names.at("router_bias"), TensorDecl{{(long long)experts}}});
-        if (has_correction) d.push_back({names.at("correction"), TensorDecl{{(long long)experts}}});
+        TensorDecls d = {{names.at("router"), TensorDecl{{(long long)all(), hidden}}}};
+        if (has_bias) d.push_back({names.at("router_bias"), TensorDecl{{(long long)all()}}});
+        if (has_correction) d.push_back({names.at("correction"), TensorDecl{{(long long)all()}}});
         for (int e = 0; e < experts; e++) {
-            d.push_back({expert_tensor(e, "gate"), TensorDecl{{inter, hidden}}});
+            if (!plain) d.push_back({expert_tensor(e, "gate"), TensorDecl{{inter, hidden}}});
             d.push_back({expert_tensor(e, "up"), TensorDecl{{inter, hidden}}});
             d.push_back({expert_tensor(e, "down"), TensorDecl{{hidden, inter}}});
         }
@@ -120,14 +131,19 @@ struct RoutedMLP : FeedForward {
             } below(src, shared_prefix);
             shared->load(below);
         }
-        gu_buf = DeviceBuffer(rt->dev, (size_t)experts * 2 * inter * hidden * es, "the experts' packed gate/up matrices");
+        const int per = plain ? 1 : 2;          // matrix rows per hidden channel of an expert
+        gu_buf = DeviceBuffer(rt->dev, (size_t)experts * per * inter * hidden * es, "the experts' packed gate/up matrices");
         down_buf = DeviceBuffer(rt->dev, (size_t)experts * hidden * inter * es, "the experts' down matrices");
-        w_gate_up = Mat{gu_buf.get(), (long long)experts * 2 * inter, hidden, rt->dtype, (long long)experts * 2 * inter};
+        w_gate_up = Mat{gu_buf.get(), (long long)experts * per * inter, hidden, rt->dtype, (long long)experts * per * inter};
         w_down = Mat{down_buf.get(), (long long)experts * hidden, inter, rt->dtype, (long long)experts * hidden};
         for (int e = 0; e < experts; e++) {
-            char* gu = (char*)w_gate_up.p + (size_t)e * 2 * inter * hidden * es;
-            src.fetch_into(expert_tensor(e, "gate"), gu, rt->dtype, 2 * hidden);              // rows 2i
-            src.fetch_into(expert_tensor(e, "up"), gu + (size_t)hidden * es, rt->dtype, 2 * hidden);  // rows 2i + 1
+            char* gu = (char*)w_gate_up.p + (size_t)e * per * inter * hidden * es;
+            if (plain) {
+                src.fetch_into(expert_tensor(e, "up"), gu, rt->dtype);
+            } else {
+                src.fetch_into(expert_tensor(e, "gate"), gu, rt->dtype, 2 * hidden);              // rows 2i
+                src.fetch_into(expert_tensor(e, "up"), gu + (size_t)hidden * es, rt->dtype, 2 * hidden);  // rows 2i + 1
+            }
             src.fetch_into(expert_tensor(e, "down"), (char*)w_down.p + (size_t)e * hidden * inter * es, rt->dtype);
         }
     }
@@ -142,6 +158,8 @@ struct RoutedMLP : FeedForward {
         route.weight_scale = weight_scale;
         route.sum_eps = sum_eps;
         route.act_limit = act_limit;
+        route.identity = identity;
+        route.plain = plain;
         route.renorm = (score_all || score_sigmoid) ? renorm : true;
         route.bias = has_bias ? (const float*)b_router.m.p : has_correction ? (const float*)correction.m.p : nullptr;
         Mat plus;
