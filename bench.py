@@ -260,8 +260,32 @@ def fifotar_config(z, vocab=32000, max_positions=4096):
                 embedding=dict(scale=8.0), residual_mult=0.5, logit_softcap=30.0, vocab=vocab, width=z["width"], max_positions=max_positions)
 
 
+ZELUZEN_LAYERS = (("wkv", "dense"), ("attention", "moe"), ("wkv", "moe"), ("wkv", "dense"), ("attention_shared", "moe"), ("wkv", "moe"))
+
+
+def zeluzen_config(z, vocab=32000, max_positions=4096):
+    """Six layers of the Zeluzen design at the size z: time-mixing layers with the linear layers' head count and 128 x 128
+    state per head and a decay map of rank 64, attention with the size's head counts in chunks of 1,024 positions (the second
+    such layer on the first one's keys and values), dense feed-forwards of the size's width, routed ones with 8 ungated experts
+    of three quarters of that width (the matrix elements of a gated expert of half of it) and 4 identity experts, of which a
+    token uses 2."""
+    layers = []
+    for t, kind in ZELUZEN_LAYERS:
+        if t == "wkv":
+            m = dict(heads=z["lin_heads"], dim=z["lin_d"], decay_rank=64)
+        else:
+            m = dict(heads=z["heads"], kv_heads=z["kv"], dim=z["d"], vdim=z["d"], scale=z["d"] ** -0.5, mask=dict(size=1024),
+                     rot=dict(base=500000.0, dims=z["d"] // 2, scaling=dict(factor=4.0, low=1.0, high=8.0, original=2048)))
+            if t == "attention_shared":
+                m["kv_from"] = 1
+        mlp = dict(kind="dense", ff=z["ff"]) if kind == "dense" else \
+            dict(kind="moe", expert=dict(ff=z["ff"] // 4 * 3), router=dict(experts=8, identity=4, top=2))
+        layers.append(dict(type="wkv" if t == "wkv" else "attention", mixer=m, mlp=mlp))
+    return dict(architecture="Zeluzen", layers=layers, norm=dict(eps=1e-5), vocab=vocab, width=z["width"], max_positions=max_positions)
+
+
 DESIGN_LAYER_NAMES = {"vokelix": list(DESIGN_LAYERS), "vizosun": ["/".join(x) for x in VIZOSUN_LAYERS], "kudonex": list(KUDONEX_LAYERS),
-                      "tukulorn": ["/".join(x) for x in TUKULORN_LAYERS], "fifotar": ["/".join(x) for x in FIFOTAR_LAYERS], "llama": len(DESIGN_LAYERS)}
+                      "tukulorn": ["/".join(x) for x in TUKULORN_LAYERS], "fifotar": ["/".join(x) for x in FIFOTAR_LAYERS], "zeluzen": ["/".join(x) for x in ZELUZEN_LAYERS], "llama": len(DESIGN_LAYERS)}
 
 
 def llama_twin(z, vocab=32000, max_positions=4096):
@@ -275,7 +299,7 @@ def run_design(args):
     """Prompt and decode throughput of a design at a few layer sizes, each beside the closest other
     model of the same width, feed-forward, head counts and number of layers (Vokelix beside LLaMA;
     Vizosun beside Vokelix and LLaMA; Kudonex and Tukulorn beside all three; Fifotar beside Vizosun, Tukulorn
-    and LLaMA), through Engine.step; and
+    and LLaMA; Zeluzen beside Vizosun, Fifotar, Vokelix and LLaMA), through Engine.step; and
     where each of the two spends its time, kernel by kernel (the driver's activity records of one step).
     One JSON line per (size, model)."""
     import torch
@@ -320,6 +344,10 @@ def run_design(args):
             arms = (("tukulorn", tukulorn_config(z)), ("vizosun", vizosun_config(z))) + arms
         if args.design == "fifotar":
             arms = (("fifotar", fifotar_config(z)), ("vizosun", vizosun_config(z)), ("tukulorn", tukulorn_config(z)), arms[1])
+        if args.design == "zeluzen":
+            arms = (("zeluzen", zeluzen_config(z)), ("vizosun", vizosun_config(z)), ("fifotar", fifotar_config(z))) + arms
+        if args.design_only:
+            arms = tuple(a for a in arms if a[0] in args.design_only.split(","))
         for which, cfgd in arms:
             eng = Engine.from_config(config_from_dict(cfgd), EngineOptions(dtype="bfloat16", max_tokens=max(B * (C + 64), NP * (T + 64)) + 64,
                                                                            max_seq_len=4096, max_batch=max(B, NP, 8)), seed=0)
@@ -582,9 +610,10 @@ def main():
                     "lengths uniform in [MIN, MAX] (seeded) prefilled in one step of unequal lengths, then NEW tokens "
                     "each (or 'toN': until position N), through the Python entry point; 'config' = the workload of --model "
                     "(8b: 16:64:2048:256, 13b: 32:128:1024:to4096)")
-    ap.add_argument("--design", choices=["vokelix", "vizosun", "kudonex", "tukulorn", "fifotar"], help="beside the default workload: prompt and decode throughput of this design "
+    ap.add_argument("--design", choices=["vokelix", "vizosun", "kudonex", "tukulorn", "fifotar", "zeluzen"], help="beside the default workload: prompt and decode throughput of this design "
                     "at a few layer sizes, each next to LLaMA layers of equal size, with the time per kernel")
     ap.add_argument("--design-size", default="1k,2k,4k", help="with --design: sizes to run (1k, 2k, 4k: the width)")
+    ap.add_argument("--design-only", help="with --design: only these of its models, with commas between them")
     ap.add_argument("--design-tokens", type=int, default=2048, help="with --design: tokens of the prompt")
     ap.add_argument("--design-context", type=int, default=2048, help="with --design: position at which the timed decode steps end")
     ap.add_argument("--design-prompts", type=int, default=1, help="with --design: prompts of --design-tokens tokens each in the prompt step")

@@ -80,6 +80,8 @@ ModelSpec ZeluzenConfig::model_spec() const {
                                            {"output_dtype", std::string("float32")},
                                            {"names", name_map({{"r", "r"}, {"k", "k"}, {"v", "v"}, {"gate", "g"}, {"mu", "mu."}, {"mu_gate", "g"}, {"w1", "w1"},
                                                                {"w2", "w2"}, {"w0", "w0"}, {"bonus", "u"}, {"norm", "norm"}, {"o", "o"}})}}));
+            // the inner size of the decay's map is the file's (the shape of w1); a model made from random numbers names it
+            if (given(m, "decay_rank")) l.mixer.params.set("decay_rank", take_int(m, "decay_rank"));
         } else if (type == "attention") {
             // softmax attention inside chunks of the sequence, one added to the softmax denominator; an RMS norm per query and
             // key head in front of an interleaved-pair rotation
