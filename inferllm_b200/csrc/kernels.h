@@ -180,7 +180,12 @@ int illm_embedding_normed(const int* ids, const void* table, int table_dtype, co
 // wkv_state.cu
 int illm_token_mix(const float* x, int T, int H, int n_mix, const float* mu, float* prev, long long prev_stride, const int* slots, const int* cu_q, const int* token_seq, int B, int single, void* out, int act_dtype, long long group_stride, void* stream);
 int illm_wkv_supported(int d, int dv);
-int illm_wkv_scan(const float* y, int T, int ld, int r_off, int k_off, int v_off, int z_off, int rank, int nh, int d, int dv, const void* w2, int w2_dtype, const float* w0, const float* u, float* state, long long state_stride, const int* slots, const int* cu_q, float* w, float* bonus, float* out, int B, int segments, float* seg_state, float* seg_decay, void* stream);
+int illm_wkv_scan(const float* y, int T, int ld, int r_off, int k_off, int v_off, int z_off, int rank, int nh, int d, int dv, const void* w2, int w2_dtype, const float* w0, const float* u, float* state, long long state_stride, const int* slots, const int* cu_q, float* w, float* bonus, float* out, int B, void* stream);
+long long illm_wkv_chunk_places(int T, int B);
+int illm_wkv_chunk_supported(int d, int dv, int ld, int r_off, int k_off, int v_off);
+int illm_wkv_chunks(float* y, int T, int ld, int r_off, int k_off, int v_off, int z_off, int rank, int nh, int d, int dv, const void* w2, const float* w0, const float* u, float* state, long long state_stride, const int* slots, const int* cu_q, float* A, float* P, float* out, int B, int max_q, int segments, float* seg_state, float* seg_decay, void* stream);
+int illm_wkv_step_supported(int d, int dv);
+int illm_wkv_step(const float* y, int splits, long long stride, int T, int ld, int r_off, int k_off, int v_off, int g_off, int z_off, int rank, int nh, int d, int dv, const void* w2, const float* w0, const float* u, float* state, long long state_stride, const int* slots, const float* norm_w, float eps, void* out, void* stream);
 
 // gemm_tc.cu, qk_prep.cu, moe.cu: further forms
 int illm_gemm_bf16_tc_grouped(const void* X, int x_rows, const void* W, const int* n, int n_groups, float* out, int M, int K, float* ws, int splits, int* err, void* stream, int skip_reduce);

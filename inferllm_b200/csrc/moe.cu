@@ -439,6 +439,35 @@ __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __
     out[i] = plus ? acc + plus[i] : acc;
 }
 
+// the same, four neighbouring channels per thread (D a multiple of four), a block per token
+template <typename TX>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const float* __restrict__ rows, const int* __restrict__ row_of_pair, const float* __restrict__ weight, const float* __restrict__ plus,
+                       const TX* __restrict__ x, float* __restrict__ out, int D, int top) {
+    pdl_grid_sync();
+    const int t = blockIdx.x;
+    for (int c = threadIdx.x * 4; c < D; c += 1024) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < top; k++) {
+            const int row = row_of_pair[t * top + k];
+            const float w = weight[t * top + k];
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (row >= 0) {
+                v = *reinterpret_cast<const float4*>(rows + (size_t)row * D + c);
+            } else if (x) {
+                const TX* xr = x + (size_t)t * D + c;
+                v = make_float4(to_f32(xr[0]), to_f32(xr[1]), to_f32(xr[2]), to_f32(xr[3]));
+            }
+            acc.x = fmaf(w, v.x, acc.x), acc.y = fmaf(w, v.y, acc.y), acc.z = fmaf(w, v.z, acc.z), acc.w = fmaf(w, v.w, acc.w);
+        }
+        if (plus) {
+            const float4 p = *reinterpret_cast<const float4*>(plus + (size_t)t * D + c);
+            acc.x += p.x, acc.y += p.y, acc.z += p.z, acc.w += p.w;
+        }
+        *reinterpret_cast<float4*>(out + (size_t)t * D + c) = acc;
+    }
+}
+
 extern "C" int illm_moe_max_tiles(int T, int top, int E, int bm) { return (int)(((long long)T * top + bm - 1) / bm) + E; }
 // rows per tile: the tensor-core kernel takes 64; the plain one 16 for steps of few tokens, else 64
 extern "C" int illm_moe_row_tile(int T, int top, int tensor_cores) { return tensor_cores || (long long)T * top > 1024 ? 64 : 16; }
@@ -580,6 +609,12 @@ extern "C" int illm_moe_combine_ex(const float* rows, const int* row_of_pair, co
     const long long n = (long long)T * D;
     const dim3 grid((unsigned)((n + 255) / 256));
     cudaStream_t s = (cudaStream_t)stream;
+    if (!(D & 3) && !(((uintptr_t)rows | (uintptr_t)plus | (uintptr_t)out) & 15)) {
+        if (x && x_dtype == ILLM_BF16) illm_launch(moe_combine_vec_kernel<bf16>, dim3(T), dim3(256), 0, s, rows, row_of_pair, weight, plus, (const bf16*)x, out, D, top);
+        else if (!x || x_dtype == ILLM_F32) illm_launch(moe_combine_vec_kernel<float>, dim3(T), dim3(256), 0, s, rows, row_of_pair, weight, plus, (const float*)x, out, D, top);
+        else return ILLM_ERR_BAD_ARG;
+        return illm_launch_status();
+    }
     if (x && x_dtype == ILLM_BF16) illm_launch(moe_combine_kernel<bf16>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const bf16*)x, out, D, top, n);
     else if (!x || x_dtype == ILLM_F32) illm_launch(moe_combine_kernel<float>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const float*)x, out, D, top, n);
     else return ILLM_ERR_BAD_ARG;

@@ -15,18 +15,31 @@
 //                        does it in the first kernel)
 // wkv_prep_kernel        w = exp(-exp(w2 tanh(z) + w0)) from the inner products z of a low-rank map, and the bonus
 //                        r . (u * k) per token and head
-// wkv_scan_kernel        the recurrence for steps of any length
-// wkv_step_kernel        the recurrence, the decay, the bonus, the per-head unit norm and the gate for one token per sequence
-//                        in one kernel, reading the projections as unreduced K slices (the bfloat16 mode's decoding)
+// wkv_scan_kernel        the recurrence token by token, for steps of any length (the float32 mode; short steps)
+// wkv_chunk_prep_kernel, wkv_chunk_kernel
+//                        the recurrence sixteen tokens at a time, for prompts in the bfloat16 mode (w2 in bfloat16)
+// wkv_step_kernel        decay, bonus, recurrence, per-head unit norm and gate for one token per sequence in one kernel that
+//                        also adds up the projections' K slices (the bfloat16 mode's decoding)
 //
-// wkv_scan_kernel: the columns of S never meet, so a block owns (sequence, head, 64 columns or what the head size leaves) and a
-// thread keeps 16 rows of four columns in registers for the whole step, the rows of a column group over LI neighbouring
-// lanes, as the scan with one decay per head does (decay_state.cu); here r, k and w of a token are three staged rows, and two
-// rows of the state share one instruction (fma.rn.f32x2).  A long prompt of few sequences may be cut into segments that run
-// side by side: pass 0 runs each from zero (the first from the sequence's state) and leaves its final state and the product of
-// its decays per channel; pass 1 folds the earlier segments' states into the state at the segment's start and adds what that
-// state gives its tokens, o_t += S_in^T (r_t * product of the segment's decays before t).  Products of decays are never
-// divided by one another.  The sums then have another order than token by token, so the float32 mode never asks for segments.
+// wkv_scan_kernel: the columns of S never meet, so a block owns (sequence, head, a run of columns) and a thread keeps 16 rows
+// of four columns in registers for the whole step, the rows of a column group over LI neighbouring lanes, as the scan with one
+// decay per head does (decay_state.cu); here r, k and w of a token are three staged rows, and two rows of the state share one
+// instruction (fma.rn.f32x2).
+//
+// Sixteen tokens at a time.  With the state S in front of a chunk, P_t the product of the decays of the chunk's tokens before
+// t, Q_t that of those behind t, and P all of them (per key channel; products of decays are never divided by one another):
+//
+//   o_t = S^T (r_t * P_t) + sum over s <= t of A[t, s] v_s
+//   A[t, s] = sum_i r_t,i k_s,i (product of w_i over the tokens between s and t),   A[t, t] = sum_i r_t,i u_i k_t,i
+//   S <- diag(P) S + sum_s (k_s * Q_s) v_s^T
+//
+// wkv_chunk_prep_kernel makes w (the low-rank map's outer product on warp-level MMA, tanh as two bfloat16 terms), the scaled
+// rows r_t * P_t and k_t * Q_t in place of r and k, A and P, a block per chunk and head; wkv_chunk_kernel runs the chunks with
+// the state in registers: its products take one multiply-add per state element instead of three, and a chunk's tokens do
+// not wait for one another.  A long prompt of few sequences is cut into segments that run side by side: pass 0 runs every
+// segment but the last for its state alone, from zero (the first from the sequence's state), and leaves that state and the
+// product of its decays; pass 1 folds the earlier segments' states into the one its segment starts from and runs the segment
+// in full.  The sums have another order than token by token, so the float32 mode never takes this form.
 #include <type_traits>
 
 #include "common.cuh"
@@ -191,7 +204,7 @@ __global__ void __launch_bounds__(128) wkv_prep_kernel(WkvPrepArgs a, const TW* 
     }
 }
 
-// ---- the recurrence over a step's tokens
+// ---- the recurrence over a step's tokens, one by one
 
 #define WS_THREADS 128
 #define WS_MAX_TILE 16
@@ -207,9 +220,6 @@ struct WkvScanArgs {
     const int *slots, *cu_q;
     float* out;                     // [T, nh * dv]
     int tile, vec;
-    int segments;
-    float* seg_state;               // [B, segments, nh, dv, d]
-    float* seg_decay;               // [B, segments, nh, d]
 };
 
 __device__ __forceinline__ void ws_cp_async16(float* dst, const float* src) {
@@ -217,8 +227,90 @@ __device__ __forceinline__ void ws_cp_async16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
 }
 
+// A thread's piece of a state [dv][d] at `src`: R = 4 M rows of C columns as pairs of rows; row of pair (m, p): m * 4 LI + 4 g +
+// 2 p and the one behind it, so that the LI lanes of a column group touch 16-byte pieces that lie side by side.  `mul` (or
+// nullptr): what the thread holds already times the rows' factors is added.
+template <int C, int M, int LI>
+__device__ __forceinline__ void wkv_load_state(f2 (&s)[C][M][2], const float* src, const float* mul, int j, int g, int d, int dv, bool vec) {
+#pragma unroll
+    for (int m = 0; m < M; m++) {
+        const int i = m * 4 * LI + 4 * g;
+        f2 f0 = 0, f1 = 0;
+        if (mul) {
+            f0 = f2_pack(i < d ? mul[i] : 0.f, i + 1 < d ? mul[i + 1] : 0.f);
+            f1 = f2_pack(i + 2 < d ? mul[i + 2] : 0.f, i + 3 < d ? mul[i + 3] : 0.f);
+        }
+#pragma unroll
+        for (int c = 0; c < C; c++) {
+            float v[4];
+            if (vec && j + c < dv && i < d) {
+                const float4 v4 = *reinterpret_cast<const float4*>(src + (size_t)(j + c) * d + i);
+                v[0] = v4.x; v[1] = v4.y; v[2] = v4.z; v[3] = v4.w;
+            } else {
+#pragma unroll
+                for (int r = 0; r < 4; r++) v[r] = (j + c < dv && i + r < d) ? src[(size_t)(j + c) * d + i + r] : 0.f;
+            }
+            s[c][m][0] = mul ? f2_fma(s[c][m][0], f0, f2_pack(v[0], v[1])) : f2_pack(v[0], v[1]);
+            s[c][m][1] = mul ? f2_fma(s[c][m][1], f1, f2_pack(v[2], v[3])) : f2_pack(v[2], v[3]);
+        }
+    }
+}
+template <int C, int M, int LI>
+__device__ __forceinline__ void wkv_store_state(const f2 (&s)[C][M][2], float* dst, int j, int g, int d, int dv, bool vec) {
+#pragma unroll
+    for (int c = 0; c < C; c++)
+#pragma unroll
+        for (int m = 0; m < M; m++) {
+            const int i = m * 4 * LI + 4 * g;
+            float v[4];
+            f2_unpack(s[c][m][0], v[0], v[1]);
+            f2_unpack(s[c][m][1], v[2], v[3]);
+            if (vec && j + c < dv && i < d) {
+                *reinterpret_cast<float4*>(dst + (size_t)(j + c) * d + i) = make_float4(v[0], v[1], v[2], v[3]);
+            } else {
+#pragma unroll
+                for (int r = 0; r < 4; r++)
+                    if (j + c < dv && i + r < d) dst[(size_t)(j + c) * d + i + r] = v[r];
+            }
+        }
+}
+
+// The sums of p[u][c] over the LI lanes of a column group, a fixed tree: while a lane holds several columns, each step halves
+// them (a lane keeps the lower half if its bit is clear and gets the partner's part of it); with one column left the
+// steps are plain.  *first: the first column this lane still holds, *held: how many; false for a lane whose sums another holds too.
+template <int U, int C, int LI>
+__device__ __forceinline__ bool wkv_lane_sums(float (&p)[U][C], int lane, int* first, int* held) {
+    int at = 0, nc = C, plain_bits = 0;
+#pragma unroll
+    for (int o = LI / 2; o >= 1; o >>= 1) {
+        const bool up = (lane & o) != 0;
+        if (nc > 1) {
+            const int hf = nc / 2;
+#pragma unroll
+            for (int u = 0; u < U; u++)
+#pragma unroll
+                for (int c = 0; c < C / 2; c++) {
+                    if (c < hf) {
+                        const float mine = up ? p[u][c + hf] : p[u][c];
+                        const float theirs = up ? p[u][c] : p[u][c + hf];
+                        p[u][c] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
+                    }
+                }
+            if (up) at += hf;
+            nc = hf;
+        } else {
+#pragma unroll
+            for (int u = 0; u < U; u++) p[u][0] += __shfl_xor_sync(0xffffffffu, p[u][0], o);
+            plain_bits |= o;
+        }
+    }
+    *first = at;
+    *held = nc;
+    return (lane & plain_bits) == 0;
+}
+
 // R rows x C columns of the state per thread, the rows of a column group over LI lanes
-template <int R, int C, int LI, int PASS>
+template <int R, int C, int LI>
 __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(WkvScanArgs a) {
     pdl_grid_sync();
     extern __shared__ __align__(16) float sm[];
@@ -227,97 +319,17 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(WkvScanArgs a) {
     constexpr int DP = R * LI;                      // rows with padding
     constexpr int ROW = 3 * DP + JB + 4;            // floats of one staged token: r, k, w, v, the bonus
     constexpr int V_AT = 3 * DP, B_AT = 3 * DP + JB;
-    const int P = a.segments;
-    const int b = blockIdx.x / P, seg = blockIdx.x % P, h = blockIdx.y, j0 = blockIdx.z * JB;
+    const int b = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * JB;
     const int d = a.d, dv = a.dv;
-    const int q0 = a.cu_q[b], q1 = a.cu_q[b + 1];
-    const int seg_len = P > 1 ? (((q1 - q0 + P - 1) / P + 15) & ~15) : q1 - q0;      // whole tiles
-    const int t0 = q0 + seg * seg_len, t1 = t0 + seg_len < q1 ? t0 + seg_len : q1;
-    if (t0 >= t1) return;                                                           // a short sequence fills fewer segments
-    const bool last_seg = t1 == q1;
+    const int t0 = a.cu_q[b], t1 = a.cu_q[b + 1];
+    if (t0 >= t1) return;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane % LI;
     const int jl = (warp * (32 / LI) + lane / LI) * C;      // first of this thread's columns within the block
     const int jn = dv - j0 < JB ? dv - j0 : JB;     // columns of this block that exist
     float* Sg = a.state + (size_t)a.slots[b] * a.state_stride + (size_t)h * d * dv;       // [dv][d]
-    // row of register pair (m, p): m * 4 LI + 4 g + 2 p and the one behind it
     f2 s[C][M][2];
-    f2 cum[M][2];                   // pass 0: the product of the segment's decays so far; pass 1: of those before the token at hand
-    const bool keep_cum = PASS == 1 || P > 1;
-    // s = (accumulate ? s * mul : 0) + src, per element; mul: the rows' factors or nullptr (1)
-    auto load_state = [&](const float* src, const float* mul, bool accumulate) {
-#pragma unroll
-        for (int c = 0; c < C; c++) {
-            const int j = j0 + jl + c;
-#pragma unroll
-            for (int m = 0; m < M; m++) {
-                const int i = m * 4 * LI + 4 * g;
-                float v[4], f[4];
-                if (a.vec && j < dv && i < d) {
-                    const float4 v4 = *reinterpret_cast<const float4*>(src + (size_t)j * d + i);
-                    v[0] = v4.x; v[1] = v4.y; v[2] = v4.z; v[3] = v4.w;
-                } else {
-#pragma unroll
-                    for (int r = 0; r < 4; r++) v[r] = (j < dv && i + r < d) ? src[(size_t)j * d + i + r] : 0.f;
-                }
-                if (accumulate) {
-#pragma unroll
-                    for (int r = 0; r < 4; r++) f[r] = i + r < d ? mul[i + r] : 0.f;
-                    s[c][m][0] = f2_fma(s[c][m][0], f2_pack(f[0], f[1]), f2_pack(v[0], v[1]));
-                    s[c][m][1] = f2_fma(s[c][m][1], f2_pack(f[2], f[3]), f2_pack(v[2], v[3]));
-                } else {
-                    s[c][m][0] = f2_pack(v[0], v[1]);
-                    s[c][m][1] = f2_pack(v[2], v[3]);
-                }
-            }
-        }
-    };
-    auto store_state = [&](float* dst) {
-#pragma unroll
-        for (int c = 0; c < C; c++) {
-            const int j = j0 + jl + c;
-#pragma unroll
-            for (int m = 0; m < M; m++) {
-                const int i = m * 4 * LI + 4 * g;
-                float v[4];
-                f2_unpack(s[c][m][0], v[0], v[1]);
-                f2_unpack(s[c][m][1], v[2], v[3]);
-                if (a.vec && j < dv && i < d) {
-                    *reinterpret_cast<float4*>(dst + (size_t)j * d + i) = make_float4(v[0], v[1], v[2], v[3]);
-                } else {
-#pragma unroll
-                    for (int r = 0; r < 4; r++)
-                        if (j < dv && i + r < d) dst[(size_t)j * d + i + r] = v[r];
-                }
-            }
-        }
-    };
-    float* seg_base = a.seg_state + ((size_t)b * P * a.nh + h) * (size_t)d * dv;      // + seg * nh * d * dv per segment
-    const size_t seg_stride = (size_t)a.nh * d * dv;
-    float* dec_base = a.seg_decay + ((size_t)b * P * a.nh + h) * (size_t)d;           // + seg * nh * d per segment
-    const size_t dec_stride = (size_t)a.nh * d;
-#pragma unroll
-    for (int m = 0; m < M; m++) cum[m][0] = cum[m][1] = f2_pack(1.f, 1.f);
-    if (PASS == 0) {
-        if (seg == 0) {
-            load_state(Sg, nullptr, false);
-        } else {
-#pragma unroll
-            for (int c = 0; c < C; c++)
-#pragma unroll
-                for (int m = 0; m < M; m++) s[c][m][0] = s[c][m][1] = f2_pack(0.f, 0.f);
-        }
-    } else {
-        if (seg == 0) {             // nothing to correct; a sequence of one segment still has to get its state
-            if (last_seg) {
-                load_state(seg_base, nullptr, false);
-                store_state(Sg);
-            }
-            return;
-        }
-        load_state(seg_base, nullptr, false);
-        for (int r = 1; r < seg; r++) load_state(seg_base + r * seg_stride, dec_base + r * dec_stride, true);
-    }
+    wkv_load_state<C, M, LI>(s, Sg, nullptr, j0 + jl, g, d, dv, a.vec);
     // rows beyond d and columns beyond dv stay zero in both buffers
     for (int idx = threadIdx.x; idx < 2 * a.tile * ROW; idx += WS_THREADS) sm[idx] = 0.f;
     __syncthreads();
@@ -362,36 +374,18 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(WkvScanArgs a) {
             f2 v[C], acc[C];
 #pragma unroll
             for (int c = 0; c < C; c++) {
-                if (PASS == 0) v[c] = f2_pack(vp[c], vp[c]);
-                acc[c] = f2_pack(0.f, 0.f);
+                v[c] = f2_pack(vp[c], vp[c]);
+                acc[c] = 0;
             }
 #pragma unroll
             for (int m = 0; m < M; m++) {
-                ulonglong2 rr = r4[m * LI];
-                const ulonglong2 ww = w4[m * LI];
-                if (PASS == 1) {
-                    rr.x = f2_mul(rr.x, cum[m][0]);
-                    rr.y = f2_mul(rr.y, cum[m][1]);
-                }
-                if (PASS == 0) {
-                    const ulonglong2 kk = k4[m * LI];
+                const ulonglong2 rr = r4[m * LI], kk = k4[m * LI], ww = w4[m * LI];
 #pragma unroll
-                    for (int c = 0; c < C; c++) {
-                        acc[c] = f2_fma(s[c][m][0], rr.x, acc[c]);
-                        acc[c] = f2_fma(s[c][m][1], rr.y, acc[c]);
-                        s[c][m][0] = f2_fma(ww.x, s[c][m][0], f2_mul(kk.x, v[c]));
-                        s[c][m][1] = f2_fma(ww.y, s[c][m][1], f2_mul(kk.y, v[c]));
-                    }
-                } else {
-#pragma unroll
-                    for (int c = 0; c < C; c++) {
-                        acc[c] = f2_fma(s[c][m][0], rr.x, acc[c]);
-                        acc[c] = f2_fma(s[c][m][1], rr.y, acc[c]);
-                    }
-                }
-                if (keep_cum) {
-                    cum[m][0] = f2_mul(cum[m][0], ww.x);
-                    cum[m][1] = f2_mul(cum[m][1], ww.y);
+                for (int c = 0; c < C; c++) {
+                    acc[c] = f2_fma(s[c][m][0], rr.x, acc[c]);
+                    acc[c] = f2_fma(s[c][m][1], rr.y, acc[c]);
+                    s[c][m][0] = f2_fma(ww.x, s[c][m][0], f2_mul(kk.x, v[c]));
+                    s[c][m][1] = f2_fma(ww.y, s[c][m][1], f2_mul(kk.y, v[c]));
                 }
             }
 #pragma unroll
@@ -401,35 +395,8 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(WkvScanArgs a) {
                 p[u][c] = lo + hi;
             }
         }
-        // the sums over the LI lanes of the column group, a fixed tree: while a lane holds several columns, each step
-        // halves them; with one column left the steps are plain
-        int first = 0;          // first column this lane still holds
-        int nc = C, plain_bits = 0;
-#pragma unroll
-        for (int o = LI / 2; o >= 1; o >>= 1) {
-            const bool up = (lane & o) != 0;
-            if (nc > 1) {
-                const int hf = nc / 2;
-#pragma unroll
-                for (int u = 0; u < U; u++)
-#pragma unroll
-                    for (int c = 0; c < C / 2; c++) {
-                        if (c < hf) {
-                            const float mine = up ? p[u][c + hf] : p[u][c];
-                            const float theirs = up ? p[u][c] : p[u][c + hf];
-                            p[u][c] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
-                        }
-                    }
-                if (up) first += hf;
-                nc = hf;
-            } else {
-#pragma unroll
-                for (int u = 0; u < U; u++) p[u][0] += __shfl_xor_sync(0xffffffffu, p[u][0], o);
-                plain_bits |= o;
-            }
-        }
-        // lanes that differ only in the bits of the plain steps hold the same sum: one of them writes
-        if ((lane & plain_bits) == 0) {
+        int first, held;
+        if (wkv_lane_sums<U, C, LI>(p, lane, &first, &held)) {
 #pragma unroll
             for (int u = 0; u < U; u++) {
                 float* orow = a.out + (size_t)(t + u) * a.nh * dv + (size_t)h * dv + j0 + jl + first;
@@ -437,10 +404,7 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(WkvScanArgs a) {
                 const float bonus = rowp[u * ROW + B_AT];
 #pragma unroll
                 for (int c = 0; c < C; c++)
-                    if (c < nc && j0 + jl + first + c < dv) {
-                        if (PASS == 0) orow[c] = fmaf(bonus, vp[c], p[u][c]);
-                        else orow[c] += p[u][c];
-                    }
+                    if (c < held && j0 + jl + first + c < dv) orow[c] = fmaf(bonus, vp[c], p[u][c]);
             }
         }
     };
@@ -461,26 +425,7 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(WkvScanArgs a) {
         for (; tt < n; tt++) tokens(std::integral_constant<int, 1>(), base + tt * ROW, tb + tt);
         __syncthreads();        // the buffer is filled again by the tile after the next
     }
-    if (PASS == 0) {
-        store_state(P > 1 ? seg_base + seg * seg_stride : Sg);
-        if (P > 1 && blockIdx.z == 0 && warp == 0 && lane < LI) {
-            float* dst = dec_base + seg * dec_stride;
-#pragma unroll
-            for (int m = 0; m < M; m++) {
-                const int i = m * 4 * LI + 4 * g;
-                float v[4];
-                f2_unpack(cum[m][0], v[0], v[1]);
-                f2_unpack(cum[m][1], v[2], v[3]);
-#pragma unroll
-                for (int r = 0; r < 4; r++)
-                    if (i + r < d) dst[i + r] = v[r];
-            }
-        }
-    } else if (last_seg) {
-        // the sequence's state: what came in, decayed over this segment, plus what the segment added
-        load_state(seg_base + seg * seg_stride, dec_base + seg * dec_stride, true);
-        store_state(Sg);
-    }
+    wkv_store_state<C, M, LI>(s, Sg, j0 + jl, g, d, dv, a.vec);
 }
 
 // head sizes up to 1024 (the rows of a column group over at most 32 lanes), any value size
@@ -492,20 +437,15 @@ static void wkv_scan_launch(WkvScanArgs a, int B, cudaStream_t s) {
     int tile = (int)(48 * 1024 / sizeof(float) / (2 * ROW));
     a.tile = tile > WS_MAX_TILE ? WS_MAX_TILE : (tile < 1 ? 1 : tile);
     if (a.tile > WS_U) a.tile -= a.tile % WS_U;
-    const size_t smem = (size_t)2 * a.tile * ROW * sizeof(float);
-    const dim3 grid(B * a.segments, a.nh, (a.dv + JB - 1) / JB);
-    illm_launch(wkv_scan_kernel<R, C, LI, 0>, grid, dim3(WS_THREADS), smem, s, a);
-    if (a.segments > 1) illm_launch(wkv_scan_kernel<R, C, LI, 1>, grid, dim3(WS_THREADS), smem, s, a);
+    illm_launch(wkv_scan_kernel<R, C, LI>, dim3(B, a.nh, (a.dv + JB - 1) / JB), dim3(WS_THREADS), (size_t)2 * a.tile * ROW * sizeof(float), s, a);
 }
 
 // y: the projections [T, ld] with r, k, v and the decay's inner products z at their offsets; w2 [nh * d, rank] (w2_dtype), w0, u
-// float32 [nh * d].  Scratch: w [T, nh * d], bonus [T, nh]; with segments > 1 seg_state [B, segments, nh, dv, d] and seg_decay
-// [B, segments, nh, d].  out: float32 [T, nh * dv].
+// float32 [nh * d].  Scratch: w [T, nh * d], bonus [T, nh].  out: float32 [T, nh * dv].
 extern "C" int illm_wkv_scan(const float* y, int T, int ld, int r_off, int k_off, int v_off, int z_off, int rank, int nh, int d, int dv, const void* w2,
                              int w2_dtype, const float* w0, const float* u, float* state, long long state_stride, const int* slots, const int* cu_q,
-                             float* w, float* bonus, float* out, int B, int segments, float* seg_state, float* seg_decay, void* stream) {
+                             float* w, float* bonus, float* out, int B, void* stream) {
     if (B <= 0 || T <= 0) return 0;
-    if (segments < 1 || (segments > 1 && (!seg_state || !seg_decay)) || (long long)B * segments > 0x7fffffff) return ILLM_ERR_BAD_ARG;
     if (nh <= 0 || nh > 65535 || d <= 0 || d > 1024 || dv <= 0 || rank <= 0 || !y || !w2 || !w0 || !u || !state || !w || !bonus || !out ||
         state_stride < (long long)nh * d * dv)
         return ILLM_ERR_BAD_ARG;
@@ -515,7 +455,7 @@ extern "C" int illm_wkv_scan(const float* y, int T, int ld, int r_off, int k_off
     if (w2_dtype == ILLM_BF16) illm_launch(wkv_prep_kernel<bf16>, pgrid, dim3(128), 0, s, p, (const bf16*)w2);
     else if (w2_dtype == ILLM_F32) illm_launch(wkv_prep_kernel<float>, pgrid, dim3(128), 0, s, p, (const float*)w2);
     else return ILLM_ERR_BAD_ARG;
-    WkvScanArgs a{y, ld, r_off, k_off, v_off, nh, d, dv, w, bonus, state, state_stride, slots, cu_q, out, 0, 0, segments, seg_state, seg_decay};
+    WkvScanArgs a{y, ld, r_off, k_off, v_off, nh, d, dv, w, bonus, state, state_stride, slots, cu_q, out, 0, 0};
     a.vec = !((d | dv | ld | r_off | k_off | v_off) & 3) && !((uintptr_t)y & 15) && !((uintptr_t)state & 15) && !((uintptr_t)w & 15) && !(state_stride & 3);
     if (d <= 16) wkv_scan_launch<16, 4, 1>(a, B, s);
     else if (d <= 32) wkv_scan_launch<16, 4, 2>(a, B, s);
@@ -524,5 +464,586 @@ extern "C" int illm_wkv_scan(const float* y, int T, int ld, int r_off, int k_off
     else if (d <= 256) wkv_scan_launch<16, 4, 16>(a, B, s);
     else if (d <= 512) wkv_scan_launch<16, 4, 32>(a, B, s);
     else wkv_scan_launch<32, 2, 32>(a, B, s);
+    return illm_launch_status();
+}
+
+// ---- sixteen tokens at a time
+
+#define WC_L 16                     // tokens of a chunk
+#define WC_CH 128                   // channels that the preparation takes at a time
+#define WC_LD (WC_CH + 4)
+#define WC_RK 64                    // columns of the low-rank map at a time
+#define WC_TLD (WC_RK + 8)
+
+struct WkvChunkPrepArgs {
+    float* y;                       // [T, ld]: r and k are replaced by r * P_t and k * Q_t
+    int ld, r_off, k_off, z_off, rank;
+    int nh, d;
+    const bf16* w2;                 // [nh * d, rank]
+    const float *w0, *u;
+    const int* cu_q;
+    float* A;                       // [chunk places, nh, 16, 16]
+    float* P;                       // [chunk places, nh, d]
+};
+
+// a sequence's chunks have neighbouring places, and no two sequences share one
+__device__ __forceinline__ int wc_place(int first_token, int b) { return first_token / WC_L + b; }
+extern "C" long long illm_wkv_chunk_places(int T, int B) { return (long long)T / WC_L + B + 1; }
+
+__device__ __forceinline__ void wc_ldsm4(unsigned* r, const void* p) {
+    const unsigned addr = (unsigned)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void wc_mma(float* c, const unsigned* a, unsigned b0, unsigned b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// grid (most chunks of a sequence, heads, sequences)
+__global__ void __launch_bounds__(128) wkv_chunk_prep_kernel(WkvChunkPrepArgs a) {
+    pdl_grid_sync();
+    __shared__ __align__(16) bf16 th[2][WC_L][WC_TLD];             // tanh of the inner products, two bfloat16 terms
+    __shared__ __align__(16) float ws[WC_L][WC_LD], rs[WC_L][WC_LD], ks[WC_L][WC_LD];
+    __shared__ __align__(16) float us[WC_CH];
+    __shared__ float As[WC_L][WC_L];
+    const int b = blockIdx.z, h = blockIdx.y, q0 = a.cu_q[b], q1 = a.cu_q[b + 1];
+    const int t0 = q0 + blockIdx.x * WC_L, n = q1 - t0 < WC_L ? q1 - t0 : WC_L;
+    if (n <= 0) return;
+    const size_t place = (size_t)(wc_place(q0, b) + blockIdx.x) * a.nh + h;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = a.d;
+    for (int i = tid; i < WC_L * WC_L; i += 128) (&As[0][0])[i] = 0.f;
+    // A: this thread takes columns s1 and s2 of sixteen rows, of every 128 channels eight (its slice)
+    const int slice = tid & 15, s1 = tid >> 4, s2 = WC_L - 1 - s1;
+    float av[WC_L + 1];
+#pragma unroll
+    for (int j = 0; j <= WC_L; j++) av[j] = 0.f;
+    for (int c0 = 0; c0 < d; c0 += WC_CH) {
+        float acc[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+            for (int k = 0; k < 4; k++) acc[i][k] = 0.f;
+        for (int r0 = 0; r0 < a.rank; r0 += WC_RK) {
+            __syncthreads();
+            for (int i = tid; i < WC_L * WC_RK; i += 128) {
+                const int tt = i / WC_RK, r = i % WC_RK;
+                const float v = tt < n && r0 + r < a.rank ? tanhf(a.y[(size_t)(t0 + tt) * a.ld + a.z_off + r0 + r]) : 0.f;
+                const bf16 hi = __float2bfloat16_rn(v);
+                th[0][tt][r] = hi;
+                th[1][tt][r] = __float2bfloat16_rn(v - __bfloat162float(hi));
+            }
+            __syncthreads();
+            const int steps = ((a.rank - r0 < WC_RK ? a.rank - r0 : WC_RK) + 15) / 16;
+            for (int kk = 0; kk < steps; kk++) {
+                unsigned hi[4], lo[4];
+                wc_ldsm4(hi, &th[0][lane & 15][kk * 16 + (lane >> 4) * 8]);
+                wc_ldsm4(lo, &th[1][lane & 15][kk * 16 + (lane >> 4) * 8]);
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    const int c = c0 + (warp * 4 + i) * 8 + (lane >> 2);
+                    unsigned bb[2] = {0, 0};
+                    if (c < d) {
+                        const bf16* row = a.w2 + (size_t)(h * d + c) * a.rank;
+#pragma unroll
+                        for (int x = 0; x < 2; x++) {
+                            const int k = r0 + kk * 16 + (lane & 3) * 2 + 8 * x;
+                            if (!(a.rank & 1)) {
+                                if (k < a.rank) bb[x] = *reinterpret_cast<const unsigned*>(row + k);
+                            } else {
+                                const unsigned e0 = k < a.rank ? __bfloat16_as_ushort(row[k]) : 0, e1 = k + 1 < a.rank ? __bfloat16_as_ushort(row[k + 1]) : 0;
+                                bb[x] = e0 | (e1 << 16);
+                            }
+                        }
+                    }
+                    wc_mma(acc[i], hi, bb[0], bb[1]);
+                    wc_mma(acc[i], lo, bb[0], bb[1]);
+                }
+            }
+        }
+        __syncthreads();        // the rows of the channels before are no longer read
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int e = (warp * 4 + i) * 8 + (lane & 3) * 2, c = c0 + e;
+            const float b0 = c < d ? a.w0[h * d + c] : 0.f, b1 = c + 1 < d ? a.w0[h * d + c + 1] : 0.f;
+#pragma unroll
+            for (int x = 0; x < 2; x++) {
+                const int tt = (lane >> 2) + 8 * x;
+                // tokens and channels that are not there leave every product as it is
+                ws[tt][e] = tt < n && c < d ? wkv_decay(acc[i][2 * x] + b0) : 1.f;
+                ws[tt][e + 1] = tt < n && c + 1 < d ? wkv_decay(acc[i][2 * x + 1] + b1) : 1.f;
+            }
+        }
+        __syncthreads();
+        {
+            const int c = c0 + tid;
+            us[tid] = c < d ? a.u[h * d + c] : 0.f;
+            float kr[WC_L], rr[WC_L];
+            float* yr = a.y + (size_t)t0 * a.ld + a.r_off + h * d + c;
+            float* yk = a.y + (size_t)t0 * a.ld + a.k_off + h * d + c;
+#pragma unroll
+            for (int t = 0; t < WC_L; t++) {
+                rr[t] = t < n && c < d ? yr[(size_t)t * a.ld] : 0.f;
+                kr[t] = t < n && c < d ? yk[(size_t)t * a.ld] : 0.f;
+                rs[t][tid] = rr[t];
+                ks[t][tid] = kr[t];
+            }
+            float cum = 1.f;
+#pragma unroll
+            for (int t = 0; t < WC_L; t++) {
+                if (t < n && c < d) yr[(size_t)t * a.ld] = rr[t] * cum;
+                cum *= ws[t][tid];
+            }
+            if (c < d) a.P[place * d + c] = cum;
+            float suf = 1.f;
+#pragma unroll
+            for (int t = WC_L - 1; t >= 0; t--) {
+                if (t < n && c < d) yk[(size_t)t * a.ld] = kr[t] * suf;
+                suf *= ws[t][tid];
+            }
+        }
+        __syncthreads();
+        f2 q[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) q[i] = 0;
+#pragma unroll
+        for (int j = 0; j <= WC_L; j++) {       // rows s1 .. 15 of column s1, then rows s2 .. 15 of column s2
+            const bool second = j >= WC_L - s1;
+            const int s = second ? s2 : s1, t = second ? s2 + j - (WC_L - s1) : s1 + j;
+            const ulonglong2* rp = reinterpret_cast<const ulonglong2*>(&rs[t][slice * 8]);
+            const ulonglong2 ra = rp[0], rb = rp[1];
+            f2 sum;
+            if (t == s) {
+                const ulonglong2* kp = reinterpret_cast<const ulonglong2*>(&ks[t][slice * 8]);
+                const ulonglong2* up = reinterpret_cast<const ulonglong2*>(&us[slice * 8]);
+                const ulonglong2 ka = kp[0], kb = kp[1], ua = up[0], ub = up[1];
+                q[0] = ka.x, q[1] = ka.y, q[2] = kb.x, q[3] = kb.y;
+                sum = f2_mul(f2_mul(ra.x, ua.x), q[0]);
+                sum = f2_fma(f2_mul(ra.y, ua.y), q[1], sum);
+                sum = f2_fma(f2_mul(rb.x, ub.x), q[2], sum);
+                sum = f2_fma(f2_mul(rb.y, ub.y), q[3], sum);
+            } else {
+                const ulonglong2* wp = reinterpret_cast<const ulonglong2*>(&ws[t][slice * 8]);
+                const ulonglong2 wa = wp[0], wb = wp[1];
+                sum = f2_mul(ra.x, q[0]);
+                sum = f2_fma(ra.y, q[1], sum);
+                sum = f2_fma(rb.x, q[2], sum);
+                sum = f2_fma(rb.y, q[3], sum);
+                q[0] = f2_mul(q[0], wa.x), q[1] = f2_mul(q[1], wa.y), q[2] = f2_mul(q[2], wb.x), q[3] = f2_mul(q[3], wb.y);
+            }
+            float lo, hi;
+            f2_unpack(sum, lo, hi);
+            av[j] += lo + hi;
+        }
+    }
+#pragma unroll
+    for (int j = 0; j <= WC_L; j++) {
+        float v = av[j];
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        const bool second = j >= WC_L - s1;
+        if (slice == 0) As[second ? s2 + j - (WC_L - s1) : s1 + j][second ? s2 : s1] = v;
+    }
+    __syncthreads();
+    for (int i = tid; i < WC_L * WC_L; i += 128) a.A[place * WC_L * WC_L + i] = (&As[0][0])[i];
+}
+
+struct WkvChunkArgs {
+    const float* y;                 // [T, ld] as the preparation left it, v untouched
+    int ld, r_off, k_off, v_off;
+    int nh, d, dv;
+    const float *A, *P;
+    float* state;
+    long long state_stride;
+    const int *slots, *cu_q;
+    float* out;                     // [T, nh * dv]
+    int segments;
+    float* seg_state;               // [B, segments, nh, dv, d]; the last place keeps the state that came in
+    float* seg_decay;               // [B, segments, nh, d]
+};
+
+template <int R, int C, int LI, int PASS>
+__global__ void __launch_bounds__(128) wkv_chunk_kernel(WkvChunkArgs a) {
+    pdl_grid_sync();
+    extern __shared__ __align__(16) float sm[];
+    constexpr int M = R / 4, DP = R * LI, JB = C * (32 / LI) * 4;
+    constexpr int U = C >= 8 ? 2 : 4;               // tokens whose sums are interleaved
+    constexpr int R_AT = 0, K_AT = PASS ? WC_L * DP : 0, V_AT = K_AT + WC_L * DP, P_AT = V_AT + WC_L * JB, A_AT = P_AT + DP;
+    constexpr int TILE = A_AT + (PASS ? WC_L * WC_L : 0);
+    constexpr int NP = LI >= 8 ? 1 : 8 / LI;        // pairs of a chunk's tokens per lane in the sum over A
+    const int S = a.segments;
+    const int b = blockIdx.x / S, seg = blockIdx.x % S, h = blockIdx.y, j0 = blockIdx.z * JB, d = a.d, dv = a.dv;
+    const int q0 = a.cu_q[b], q1 = a.cu_q[b + 1], chunks = (q1 - q0 + WC_L - 1) / WC_L, per = (chunks + S - 1) / S;
+    const int first_chunk = seg * per, end_chunk = first_chunk + per < chunks ? first_chunk + per : chunks;
+    if (first_chunk >= end_chunk) return;           // a short sequence fills fewer segments
+    const bool last = end_chunk == chunks;
+    if (PASS == 0 && last) return;                  // nobody starts from the last segment's state
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane % LI;
+    const int jl = (warp * (32 / LI) + lane / LI) * C;
+    const int jn = dv - j0 < JB ? dv - j0 : JB;
+    float* Sg = a.state + (size_t)a.slots[b] * a.state_stride + (size_t)h * d * dv;       // [dv][d]
+    float* seg_base = a.seg_state + ((size_t)b * S * a.nh + h) * (size_t)d * dv;          // + segment * nh * d * dv
+    const size_t seg_stride = (size_t)a.nh * d * dv;
+    float* dec_base = a.seg_decay + ((size_t)b * S * a.nh + h) * (size_t)d;
+    const size_t dec_stride = (size_t)a.nh * d;
+    const size_t place0 = (size_t)wc_place(q0, b);
+    for (int idx = threadIdx.x; idx < 2 * TILE; idx += 128) sm[idx] = 0.f;          // rows beyond d, columns beyond dv, tokens that are not there
+    __syncthreads();
+    auto stage = [&](int buf, int chunk) {
+        const int t0 = q0 + chunk * WC_L, n = q1 - t0 < WC_L ? q1 - t0 : WC_L;
+        float* base = sm + buf * TILE;
+        const int cq = d >> 2, cv = jn >> 2;
+        const float* row0 = a.y + (size_t)t0 * a.ld;
+        for (int tt = warp; tt < n; tt += 4) {
+            const float* row = row0 + (size_t)tt * a.ld;
+            for (int c = lane; c < cq; c += 32) {
+                if (PASS == 1) ws_cp_async16(base + R_AT + tt * DP + 4 * c, row + a.r_off + h * d + 4 * c);
+                ws_cp_async16(base + K_AT + tt * DP + 4 * c, row + a.k_off + h * d + 4 * c);
+            }
+            for (int c = lane; c < cv; c += 32) ws_cp_async16(base + V_AT + tt * JB + 4 * c, row + a.v_off + h * dv + j0 + 4 * c);
+        }
+        const size_t place = (place0 + chunk) * a.nh + h;
+        for (int c = threadIdx.x; c < cq; c += 128) ws_cp_async16(base + P_AT + 4 * c, a.P + place * d + 4 * c);
+        if (PASS == 1 && threadIdx.x < WC_L * WC_L / 4) ws_cp_async16(base + A_AT + 4 * threadIdx.x, a.A + place * WC_L * WC_L + 4 * threadIdx.x);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage(0, first_chunk);
+    f2 s[C][M][2], cum[M][2];
+    if (PASS == 0) {
+#pragma unroll
+        for (int m = 0; m < M; m++) cum[m][0] = cum[m][1] = f2_pack(1.f, 1.f);
+        if (seg == 0) {
+            // what came in is kept for pass 1, whose last segment renews the state while its first may not have begun
+            wkv_load_state<C, M, LI>(s, Sg, nullptr, j0 + jl, g, d, dv, true);
+            wkv_store_state<C, M, LI>(s, seg_base + (size_t)(S - 1) * seg_stride, j0 + jl, g, d, dv, true);
+        } else {
+#pragma unroll
+            for (int c = 0; c < C; c++)
+#pragma unroll
+                for (int m = 0; m < M; m++) s[c][m][0] = s[c][m][1] = 0;
+        }
+    } else if (seg == 0) {
+        wkv_load_state<C, M, LI>(s, last ? Sg : seg_base + (size_t)(S - 1) * seg_stride, nullptr, j0 + jl, g, d, dv, true);
+    } else {
+        wkv_load_state<C, M, LI>(s, seg_base, nullptr, j0 + jl, g, d, dv, true);
+        for (int r = 1; r < seg; r++) wkv_load_state<C, M, LI>(s, seg_base + r * seg_stride, dec_base + r * dec_stride, j0 + jl, g, d, dv, true);
+    }
+    int buf = 0;
+    for (int chunk = first_chunk; chunk < end_chunk; chunk++, buf ^= 1) {
+        const int t0 = q0 + chunk * WC_L, n = q1 - t0 < WC_L ? q1 - t0 : WC_L;
+        if (chunk + 1 < end_chunk) {
+            stage(buf ^ 1, chunk + 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const float* base = sm + buf * TILE;
+        if (PASS == 1) {
+            // a lane's share of the sum over the chunk's own tokens: pairs (2 i, 2 i + 1), i = g, g + LI, ..
+            f2 vp[NP][C];
+#pragma unroll
+            for (int i = 0; i < NP; i++)
+#pragma unroll
+                for (int c = 0; c < C; c++) {
+                    const int s0 = 2 * ((g & 7) + i * LI);
+                    vp[i][c] = LI <= 8 || g < 8 ? f2_pack(base[V_AT + s0 * JB + jl + c], base[V_AT + (s0 + 1) * JB + jl + c]) : 0;
+                }
+            for (int tt = 0; tt < n; tt += U) {
+                float p[U][C];
+#pragma unroll
+                for (int u = 0; u < U; u++) {
+                    const ulonglong2* r4 = reinterpret_cast<const ulonglong2*>(base + R_AT + (tt + u) * DP) + g;
+                    f2 acc[C];
+#pragma unroll
+                    for (int i = 0; i < NP; i++) {
+                        const f2 av = *reinterpret_cast<const f2*>(base + A_AT + (tt + u) * WC_L + 2 * ((g & 7) + i * LI));
+#pragma unroll
+                        for (int c = 0; c < C; c++) acc[c] = i == 0 ? f2_mul(av, vp[i][c]) : f2_fma(av, vp[i][c], acc[c]);
+                    }
+#pragma unroll
+                    for (int m = 0; m < M; m++) {
+                        const ulonglong2 rr = r4[m * LI];
+#pragma unroll
+                        for (int c = 0; c < C; c++) {
+                            acc[c] = f2_fma(s[c][m][0], rr.x, acc[c]);
+                            acc[c] = f2_fma(s[c][m][1], rr.y, acc[c]);
+                        }
+                    }
+#pragma unroll
+                    for (int c = 0; c < C; c++) {
+                        float lo, hi;
+                        f2_unpack(acc[c], lo, hi);
+                        p[u][c] = lo + hi;
+                    }
+                }
+                int first, held;
+                if (wkv_lane_sums<U, C, LI>(p, lane, &first, &held)) {
+#pragma unroll
+                    for (int u = 0; u < U; u++) {
+                        float* orow = a.out + (size_t)(t0 + tt + u) * a.nh * dv + (size_t)h * dv + j0 + jl + first;
+#pragma unroll
+                        for (int c = 0; c < C; c++)
+                            if (c < held && tt + u < n && j0 + jl + first + c < dv) orow[c] = p[u][c];
+                    }
+                }
+            }
+        }
+        const ulonglong2* p4 = reinterpret_cast<const ulonglong2*>(base + P_AT) + g;
+#pragma unroll
+        for (int m = 0; m < M; m++) {
+            const ulonglong2 pp = p4[m * LI];
+#pragma unroll
+            for (int c = 0; c < C; c++) {
+                s[c][m][0] = f2_mul(s[c][m][0], pp.x);
+                s[c][m][1] = f2_mul(s[c][m][1], pp.y);
+            }
+            if (PASS == 0) {
+                cum[m][0] = f2_mul(cum[m][0], pp.x);
+                cum[m][1] = f2_mul(cum[m][1], pp.y);
+            }
+        }
+#pragma unroll 2
+        for (int tt = 0; tt < n; tt++) {
+            const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(base + K_AT + tt * DP) + g;
+            const float* vr = base + V_AT + tt * JB + jl;
+            f2 v[C];
+#pragma unroll
+            for (int c = 0; c < C; c++) v[c] = f2_pack(vr[c], vr[c]);
+#pragma unroll
+            for (int m = 0; m < M; m++) {
+                const ulonglong2 kk = k4[m * LI];
+#pragma unroll
+                for (int c = 0; c < C; c++) {
+                    s[c][m][0] = f2_fma(kk.x, v[c], s[c][m][0]);
+                    s[c][m][1] = f2_fma(kk.y, v[c], s[c][m][1]);
+                }
+            }
+        }
+        __syncthreads();        // the buffer is filled again by the chunk after the next
+    }
+    if (PASS == 0) {
+        wkv_store_state<C, M, LI>(s, seg_base + seg * seg_stride, j0 + jl, g, d, dv, true);
+        if (blockIdx.z == 0 && warp == 0 && lane < LI) {
+            float* dst = dec_base + seg * dec_stride;
+#pragma unroll
+            for (int m = 0; m < M; m++) {
+                const int i = m * 4 * LI + 4 * g;
+                float v[4];
+                f2_unpack(cum[m][0], v[0], v[1]);
+                f2_unpack(cum[m][1], v[2], v[3]);
+                if (i < d) *reinterpret_cast<float4*>(dst + i) = make_float4(v[0], v[1], v[2], v[3]);
+            }
+        }
+    } else if (last) {
+        wkv_store_state<C, M, LI>(s, Sg, j0 + jl, g, d, dv, true);
+    }
+}
+
+template <int R, int C, int LI>
+static int wkv_chunk_launch(const WkvChunkArgs& a, int B, cudaStream_t s) {
+    constexpr int DP = R * LI, JB = C * (32 / LI) * 4;
+    constexpr size_t smem0 = 2 * sizeof(float) * (WC_L * DP + WC_L * JB + DP), smem1 = smem0 + 2 * sizeof(float) * (WC_L * DP + WC_L * WC_L);
+    static bool raised = false;
+    if (!raised) {
+        cudaError_t e = cudaFuncSetAttribute(wkv_chunk_kernel<R, C, LI, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem0);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(wkv_chunk_kernel<R, C, LI, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        if (e != cudaSuccess) return (int)e;
+        raised = true;
+    }
+    const dim3 grid(B * a.segments, a.nh, (a.dv + JB - 1) / JB);
+    if (a.segments > 1) illm_launch(wkv_chunk_kernel<R, C, LI, 0>, grid, dim3(128), smem0, s, a);
+    illm_launch(wkv_chunk_kernel<R, C, LI, 1>, grid, dim3(128), smem1, s, a);
+    return illm_launch_status();
+}
+
+// rows of whole 16-byte pieces and up to 512 key channels; ld and the offsets are multiples of four too
+extern "C" int illm_wkv_chunk_supported(int d, int dv, int ld, int r_off, int k_off, int v_off) {
+    return d > 0 && d <= 512 && dv > 0 && !((d | dv | ld | r_off | k_off | v_off) & 3) ? 1 : 0;
+}
+
+// The prompts' form: as illm_wkv_scan with w2 in bfloat16; y's r and k columns are scratch afterwards.  A [places, nh, 16, 16] and
+// P [places, nh, d] are scratch (places = illm_wkv_chunk_places), with segments > 1 also seg_state [B, segments, nh, dv, d] and
+// seg_decay [B, segments, nh, d].  max_q: the most tokens of a sequence.
+extern "C" int illm_wkv_chunks(float* y, int T, int ld, int r_off, int k_off, int v_off, int z_off, int rank, int nh, int d, int dv, const void* w2,
+                               const float* w0, const float* u, float* state, long long state_stride, const int* slots, const int* cu_q, float* A, float* P,
+                               float* out, int B, int max_q, int segments, float* seg_state, float* seg_decay, void* stream) {
+    if (B <= 0 || T <= 0) return 0;
+    if (segments < 1 || (segments > 1 && (!seg_state || !seg_decay)) || (long long)B * segments > 0x7fffffff || B > 65535 || max_q <= 0) return ILLM_ERR_BAD_ARG;
+    if (nh <= 0 || nh > 65535 || rank <= 0 || !y || !w2 || !w0 || !u || !state || !A || !P || !out || state_stride < (long long)nh * d * dv ||
+        !illm_wkv_chunk_supported(d, dv, ld, r_off, k_off, v_off) || (state_stride & 3) ||
+        (((uintptr_t)y | (uintptr_t)state | (uintptr_t)A | (uintptr_t)P | (uintptr_t)seg_state | (uintptr_t)seg_decay) & 15) || ((uintptr_t)w2 & 3))
+        return ILLM_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    WkvChunkPrepArgs p{y, ld, r_off, k_off, z_off, rank, nh, d, (const bf16*)w2, w0, u, cu_q, A, P};
+    illm_launch(wkv_chunk_prep_kernel, dim3((max_q + WC_L - 1) / WC_L, nh, B), dim3(128), 0, s, p);
+    WkvChunkArgs a{y, ld, r_off, k_off, v_off, nh, d, dv, A, P, state, state_stride, slots, cu_q, out, segments, seg_state, seg_decay};
+    if (d <= 16) return wkv_chunk_launch<16, 4, 1>(a, B, s);
+    if (d <= 32) return wkv_chunk_launch<16, 4, 2>(a, B, s);
+    if (d <= 64) return wkv_chunk_launch<16, 4, 4>(a, B, s);
+    if (d <= 128) return wkv_chunk_launch<16, 8, 8>(a, B, s);
+    if (d <= 256) return wkv_chunk_launch<16, 8, 16>(a, B, s);
+    return wkv_chunk_launch<16, 8, 32>(a, B, s);
+}
+
+// ---- one token per sequence
+
+struct WkvStepArgs {
+    const float* y;                 // the projections [T, ld], finished or as `splits` slices `stride` floats apart
+    int splits;
+    long long stride;
+    int ld, r_off, k_off, v_off, g_off, z_off, rank;
+    int nh, d, dv;
+    const bf16* w2;                 // [nh * d, rank]
+    const float *w0, *u;
+    float* state;
+    long long state_stride;
+    const int* slots;
+    const float* norm_w;            // [nh * dv]
+    float eps;
+};
+
+// grid (tokens, heads), 256 threads: token t is the only one of sequence t.  A column of the state lies over LI lanes, NV pieces
+// of four rows each; a warp has CB columns per lane group on their way at a time.
+template <int LI, int NV, int CB>
+__global__ void __launch_bounds__(256) wkv_step_kernel(WkvStepArgs a, bf16* __restrict__ out) {
+    pdl_grid_sync();
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float scratch[32];
+    constexpr int GW = 32 / LI;                     // column groups of a warp
+    const int t = blockIdx.x, h = blockIdx.y, d = a.d, dv = a.dv, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane % LI;
+    float *r = sm, *k = r + d, *w = k + d, *v = w + d, *gt = v + dv, *o = gt + dv, *th = o + dv;
+    float* Sg = a.state + (size_t)a.slots[t] * a.state_stride + (size_t)h * d * dv;
+    float4 s[CB][NV];
+    auto column = [&](int batch, int c) { return ((batch * CB + c) * 8 + warp) * GW + lane / LI; };
+    auto load = [&](int batch) {
+#pragma unroll
+        for (int c = 0; c < CB; c++) {
+            const int j = column(batch, c);
+#pragma unroll
+            for (int m = 0; m < NV; m++) {
+                const int i = 4 * (g + m * LI);
+                s[c][m] = j < dv && i < d ? *reinterpret_cast<const float4*>(Sg + (size_t)j * d + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        }
+    };
+    load(0);
+    const float* row = a.y + (size_t)t * a.ld;
+    auto projected = [&](int col) {                 // the slices in ascending order, their loads in flight together
+        float x = row[col];
+        int sl = 1;
+        for (; sl + 4 <= a.splits; sl += 4) {
+            float f[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) f[i] = row[(size_t)(sl + i) * a.stride + col];
+#pragma unroll
+            for (int i = 0; i < 4; i++) x += f[i];
+        }
+        for (; sl < a.splits; sl++) x += row[(size_t)sl * a.stride + col];
+        return x;
+    };
+    for (int i = tid; i < 2 * d + 2 * dv + a.rank; i += 256) {
+        if (i < d) r[i] = projected(a.r_off + h * d + i);
+        else if (i < 2 * d) k[i - d] = projected(a.k_off + h * d + i - d);
+        else if (i < 2 * d + dv) v[i - 2 * d] = projected(a.v_off + h * dv + i - 2 * d);
+        else if (i < 2 * d + 2 * dv) gt[i - 2 * d - dv] = projected(a.g_off + h * dv + i - 2 * d - dv);
+        else th[i - 2 * d - 2 * dv] = tanhf(projected(a.z_off + i - 2 * d - 2 * dv));
+    }
+    __syncthreads();
+    float bonus = 0.f;
+    for (int c = tid; c < d; c += 256) bonus = fmaf(r[c] * a.u[h * d + c], k[c], bonus);
+    bonus = block_sum(bonus, scratch);
+    // two lanes per channel, each half of the low-rank map's columns
+    const int half = (a.rank + 15) / 16 * 8;
+    for (int i = tid; i < (2 * d + 31) / 32 * 32; i += 256) {
+        const int c = i >> 1, r0 = (i & 1) * half, r1 = r0 + half < a.rank ? r0 + half : a.rank;
+        float acc = 0.f;
+        if (c < d) {
+            const bf16* wr = a.w2 + (size_t)(h * d + c) * a.rank;
+            if (!(a.rank & 7)) {
+                for (int q = r0; q < r1; q += 8) {
+                    float f[8];
+                    load8(wr + q, f);
+#pragma unroll
+                    for (int e = 0; e < 8; e++) acc = fmaf(f[e], th[q + e], acc);
+                }
+            } else {
+                for (int q = r0; q < r1; q++) acc = fmaf(to_f32(wr[q]), th[q], acc);
+            }
+        }
+        acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+        if (c < d && !(i & 1)) w[c] = wkv_decay(acc + a.w0[h * d + c]);
+    }
+    __syncthreads();
+    float4 r4[NV], k4[NV], w4[NV];
+#pragma unroll
+    for (int m = 0; m < NV; m++) {
+        const int i = 4 * (g + m * LI);
+        const bool ok = i < d;
+        r4[m] = ok ? *reinterpret_cast<const float4*>(r + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        k4[m] = ok ? *reinterpret_cast<const float4*>(k + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        w4[m] = ok ? *reinterpret_cast<const float4*>(w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const int batches = (dv + 8 * GW * CB - 1) / (8 * GW * CB);
+    for (int batch = 0; batch < batches; batch++) {
+        if (batch) load(batch);
+        float p[1][CB];
+#pragma unroll
+        for (int c = 0; c < CB; c++) {
+            const int j = column(batch, c);
+            const float vj = j < dv ? v[j] : 0.f;
+            float x = 0.f;
+#pragma unroll
+            for (int m = 0; m < NV; m++) {
+                float4 q = s[c][m];
+                x = fmaf(q.x, r4[m].x, x), x = fmaf(q.y, r4[m].y, x), x = fmaf(q.z, r4[m].z, x), x = fmaf(q.w, r4[m].w, x);
+                q.x = fmaf(w4[m].x, q.x, k4[m].x * vj);
+                q.y = fmaf(w4[m].y, q.y, k4[m].y * vj);
+                q.z = fmaf(w4[m].z, q.z, k4[m].z * vj);
+                q.w = fmaf(w4[m].w, q.w, k4[m].w * vj);
+                const int i = 4 * (g + m * LI);
+                if (j < dv && i < d) *reinterpret_cast<float4*>(Sg + (size_t)j * d + i) = q;
+            }
+            p[0][c] = x;
+        }
+        int first, held;
+        if (wkv_lane_sums<1, CB, LI>(p, lane, &first, &held)) {
+#pragma unroll
+            for (int c = 0; c < CB; c++) {
+                const int j = column(batch, first + c);
+                if (c < held && j < dv) o[j] = fmaf(bonus, v[j], p[0][c]);
+            }
+        }
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int c = tid; c < dv; c += 256) ss = fmaf(o[c], o[c], ss);
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + a.eps);
+    bf16* orow = out + (size_t)t * a.nh * dv + (size_t)h * dv;
+    for (int c = tid; c < dv; c += 256) orow[c] = __float2bfloat16_rn(((o[c] * inv) * a.norm_w[h * dv + c]) * (gt[c] / (1.0f + expf(-gt[c]))));
+}
+
+extern "C" int illm_wkv_step_supported(int d, int dv) { return d > 0 && d <= 512 && !(d & 3) && dv > 0 && dv <= 1024 && !(dv & 3) ? 1 : 0; }
+
+// One token per sequence (T = B tokens in the order of the sequences), bfloat16 mode: y [T, ld] float32 with r, k, v, the gate's and
+// the decay's inner projections, finished (splits 1) or as slices `stride` floats apart; w2 [nh * d, rank] bfloat16.  out: bfloat16
+// [T, nh * dv] = o / rms(o) per head * norm_w * silu(gate).
+extern "C" int illm_wkv_step(const float* y, int splits, long long stride, int T, int ld, int r_off, int k_off, int v_off, int g_off, int z_off, int rank,
+                             int nh, int d, int dv, const void* w2, const float* w0, const float* u, float* state, long long state_stride,
+                             const int* slots, const float* norm_w, float eps, void* out, void* stream) {
+    if (T <= 0) return 0;
+    if (splits < 1 || nh <= 0 || nh > 65535 || rank <= 0 || rank > 4096 || !y || !w2 || !w0 || !u || !state || !norm_w || !out ||
+        !illm_wkv_step_supported(d, dv) || state_stride < (long long)nh * d * dv || (state_stride & 3) || ((uintptr_t)state & 15) || ((uintptr_t)w2 & 15))
+        return ILLM_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    WkvStepArgs a{y, splits, stride, ld, r_off, k_off, v_off, g_off, z_off, rank, nh, d, dv, (const bf16*)w2, w0, u, state, state_stride, slots, norm_w, eps};
+    const size_t smem = (size_t)(3 * d + 3 * dv + rank) * sizeof(float);
+    const dim3 grid(T, nh);
+    if (d <= 16) illm_launch((wkv_step_kernel<4, 1, 4>), grid, dim3(256), smem, s, a, (bf16*)out);
+    else if (d <= 32) illm_launch((wkv_step_kernel<8, 1, 4>), grid, dim3(256), smem, s, a, (bf16*)out);
+    else if (d <= 64) illm_launch((wkv_step_kernel<16, 1, 8>), grid, dim3(256), smem, s, a, (bf16*)out);
+    else if (d <= 128) illm_launch((wkv_step_kernel<32, 1, 16>), grid, dim3(256), smem, s, a, (bf16*)out);
+    else if (d <= 256) illm_launch((wkv_step_kernel<32, 2, 8>), grid, dim3(256), smem, s, a, (bf16*)out);
+    else illm_launch((wkv_step_kernel<32, 4, 4>), grid, dim3(256), smem, s, a, (bf16*)out);
     return illm_launch_status();
 }

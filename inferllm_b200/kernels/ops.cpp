@@ -1057,8 +1057,8 @@ MatOrPartials group_linear(Device& dev, GemmBackend backend, const Mat& x, long 
 bool wkv_supported(int d, int dv) { return illm_wkv_supported(d, dv) != 0; }
 
 int wkv_segments(int B, int n_heads, int v_head_dim, int max_q, int n_sms) {
-    const long long blocks = (long long)B * n_heads * ceil_div(v_head_dim, 64);
-    long long P = std::min<long long>(16, (8LL * n_sms) / std::max<long long>(blocks, 1));
+    const long long blocks = (long long)B * n_heads * ceil_div(v_head_dim, 128);
+    long long P = std::min<long long>(16, (4LL * n_sms) / std::max<long long>(blocks, 1));
     P = std::min<long long>(P, max_q / 64);
     return P < 2 ? 1 : (int)P;
 }
@@ -1072,14 +1072,46 @@ Mat wkv_scan(Device& dev, const Mat& y, const WkvScan& p, const StepView& ctx, c
     if (p.r_off < 0 || p.r_off + HD > y.cols || p.k_off < 0 || p.k_off + HD > y.cols || p.v_off < 0 || p.v_off + HV > y.cols || p.z_off < 0 || p.z_off + p.rank > y.cols)
         throw KernelError("wkv_scan: the projections do not lie inside the rows");
     Mat out = new_mat_exact(dev, y.rows, HV, DType::F32);
+    if (!p.in_order && ctx.max_q >= kWkvChunkMinTokens && p.w2->dtype == DType::BF16 && st.elements % 4 == 0 &&
+        illm_wkv_chunk_supported(p.head_dim, p.v_head_dim, (int)y.cols, p.r_off, p.k_off, p.v_off)) {
+        const long long places = illm_wkv_chunk_places((int)y.rows, ctx.B);
+        float *A = dev.alloc_n<float>((size_t)places * p.n_heads * 256), *P = dev.alloc_n<float>((size_t)places * HD);
+        const int segments = wkv_segments(ctx.B, p.n_heads, p.v_head_dim, ctx.max_q, dev.n_sms());
+        float* seg_state = segments > 1 ? dev.alloc_n<float>((size_t)ctx.B * segments * HD * p.v_head_dim) : nullptr;
+        float* seg_decay = segments > 1 ? dev.alloc_n<float>((size_t)ctx.B * segments * HD) : nullptr;
+        check_kernel(illm_wkv_chunks((float*)y.p, (int)y.rows, (int)y.cols, p.r_off, p.k_off, p.v_off, p.z_off, p.rank, p.n_heads, p.head_dim, p.v_head_dim,
+                                     p.w2->p, p.w0, p.u, (float*)st.state, st.elements, st.slots, ctx.cu_q, A, P, (float*)out.p, ctx.B, ctx.max_q, segments,
+                                     seg_state, seg_decay, dev.stream()),
+                     "wkv_chunks");
+        return out;
+    }
     float *w = dev.alloc_n<float>((size_t)y.rows * HD), *bonus = dev.alloc_n<float>((size_t)y.rows * p.n_heads);
-    const int segments = (p.in_order || ctx.is_decode) ? 1 : wkv_segments(ctx.B, p.n_heads, p.v_head_dim, ctx.max_q, dev.n_sms());
-    float* seg_state = segments > 1 ? dev.alloc_n<float>((size_t)ctx.B * segments * HD * p.v_head_dim) : nullptr;
-    float* seg_decay = segments > 1 ? dev.alloc_n<float>((size_t)ctx.B * segments * HD) : nullptr;
     check_kernel(illm_wkv_scan((const float*)y.p, (int)y.rows, (int)y.cols, p.r_off, p.k_off, p.v_off, p.z_off, p.rank, p.n_heads, p.head_dim, p.v_head_dim,
                                p.w2->p, code_of(p.w2->dtype, "wkv_scan"), p.w0, p.u, (float*)st.state, st.elements, st.slots, ctx.cu_q, w, bonus, (float*)out.p,
-                               ctx.B, segments, seg_state, seg_decay, dev.stream()),
+                               ctx.B, dev.stream()),
                  "wkv_scan");
+    return out;
+}
+
+bool wkv_step_supported(const WkvScan& p, const StateView& st) {
+    return p.w2 && p.w2->dtype == DType::BF16 && illm_wkv_step_supported(p.head_dim, p.v_head_dim) && st.elements % 4 == 0 && p.rank <= 4096;
+}
+
+Mat wkv_step(Device& dev, const MatOrPartials& y, const WkvScan& p, int gate_off, const float* norm_w, float eps, const StepView& ctx, const StateView& st) {
+    const long long HD = (long long)p.n_heads * p.head_dim, HV = (long long)p.n_heads * p.v_head_dim, N = y.cols();
+    if (!ctx.is_decode || y.rows() != ctx.B) throw KernelError("wkv_step: a step of one token per sequence only");
+    if (!wkv_step_supported(p, st)) throw KernelError("wkv_step: the head size is beyond the kernel");
+    if (!y.is_partials()) need(y.m, "the projections", true, DType::F32);
+    if (!st.state || st.dtype != DType::F32 || st.elements < HD * p.v_head_dim) throw KernelError("wkv_step: the cache entry does not hold the state");
+    if (p.w2->rows != HD || p.w2->cols != p.rank || p.rank <= 0) throw KernelError("wkv_step: the decay's outer map must be [heads * head size, rank]");
+    if (p.r_off < 0 || p.r_off + HD > N || p.k_off < 0 || p.k_off + HD > N || p.v_off < 0 || p.v_off + HV > N || gate_off < 0 || gate_off + HV > N || p.z_off < 0 ||
+        p.z_off + p.rank > N)
+        throw KernelError("wkv_step: the projections do not lie inside the rows");
+    Mat out = new_mat(dev, y.rows(), HV, DType::BF16);
+    check_kernel(illm_wkv_step(y.is_partials() ? y.part.ws : (const float*)y.m.p, y.is_partials() ? y.part.splits : 1, y.is_partials() ? y.part.rows * N : 0,
+                               (int)y.rows(), (int)N, p.r_off, p.k_off, p.v_off, gate_off, p.z_off, p.rank, p.n_heads, p.head_dim, p.v_head_dim, p.w2->p, p.w0,
+                               p.u, (float*)st.state, st.elements, st.slots, norm_w, eps, out.p, dev.stream()),
+                 "wkv_step");
     return out;
 }
 

@@ -393,17 +393,27 @@ MatOrPartials group_linear(Device& dev, GemmBackend backend, const Mat& x, long 
 // The recurrence with a decay per head and key channel made by the token itself, and a bonus for the token's own contribution
 // (csrc/wkv_state.cu).  y: float32 [T, ld] with r, k, v and the decay's inner products z (rank columns) at their offsets;
 // w2 [heads * d, rank]; w0, u float32 [heads * d].  The state S [heads, dv, d] stands at the start of the slot's elements.
-// Returns float32 [T, heads * v_head_dim].  in_order as in DecayScan.
+// Returns float32 [T, heads * v_head_dim].
 struct WkvScan {
     int r_off = 0, k_off = 0, v_off = 0, z_off = 0, rank = 0;
     int n_heads = 0, head_dim = 0, v_head_dim = 0;
     const Mat* w2 = nullptr;
     const float *w0 = nullptr, *u = nullptr;
+    // false: prompts may go sixteen tokens at a time, in segments that run side by side (the order of the sums then differs from
+    // token by token; y's r and k columns are overwritten); true: always token by token, bit for bit
     bool in_order = true;
 };
+constexpr int kWkvChunkMinTokens = 16;       // the most tokens of a sequence in a step from which prompts go sixteen at a time
 bool wkv_supported(int head_dim, int v_head_dim);
+// In how many segments the chunks of a prompt step's sequences are cut: enough blocks for the GPU, at most 16, none of fewer
+// than 64 tokens.
 int wkv_segments(int B, int n_heads, int v_head_dim, int max_q, int n_sms);
 Mat wkv_scan(Device& dev, const Mat& y_f32, const WkvScan& p, const StepView& ctx, const StateView& st);
+// One token per sequence in the bfloat16 mode: the recurrence and what surrounds it in one kernel, from the projections (finished or
+// unreduced slices) with the gate's columns at gate_off to the bfloat16 rows o / rms(o) per head * norm_w * silu(gate), [T, heads *
+// v_head_dim].
+bool wkv_step_supported(const WkvScan& p, const StateView& st);
+Mat wkv_step(Device& dev, const MatOrPartials& y, const WkvScan& p, int gate_off, const float* norm_w, float eps, const StepView& ctx, const StateView& st);
 
 // Attention through latents (csrc/latent_attention.cu): the two norms and the cache write; returns the normed
 // query latent [T, q_rank] in `act_dtype`.  kv: a keys-only entry of one head of kv_rank channels.

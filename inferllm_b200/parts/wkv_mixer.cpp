@@ -21,7 +21,7 @@ namespace {
 
 struct WkvMixer : Mixer {
     long long hidden;
-    int n_heads, head_dim, rank = 0;
+    int n_heads, head_dim, rank = 0, rank_rows = 0;      // rank_rows: the rank in whole pieces of eight rows (the rest zeros)
     float norm_eps;
     bool out_f32;
     std::map<std::string, std::string> names;
@@ -67,12 +67,14 @@ struct WkvMixer : Mixer {
         const std::vector<long long> s1 = src.shape(names.at("w1")), s2 = src.shape(names.at("w2"));
         if (s1.size() != 2 || s2.size() != 2 || s1[0] != s2[1] || s1[0] <= 0) throw WeightError("wkv: the two matrices of the decay's map do not fit together");
         rank = (int)s1[0];
+        rank_rows = (rank + 7) / 8 * 8;
         mu_buf = DeviceBuffer(rt->dev, (size_t)5 * hidden * sizeof(float), "a mixer's blends");
         int i = 0;
         for (const char* s : {"r", "k", "v", "g", "w"}) src.fetch_into(blend(s), (float*)mu_buf.get() + (size_t)(i++) * hidden, DType::F32);
-        const long long rows = 4 * n + rank;
+        const long long rows = 4 * n + rank_rows;
         in_buf = DeviceBuffer(rt->dev, (size_t)rows * hidden * es, "the stacked projections of a time-mixing layer");
         w_in = Mat{in_buf.get(), rows, hidden, rt->dtype, rows};
+        check_cuda(cudaMemsetAsync(in_buf.get(), 0, in_buf.bytes(), rt->dev->stream()), "clearing the stacked projections");
         i = 0;
         for (const char* s : {"r", "k", "v", "gate"}) src.fetch_into(names.at(s), (char*)in_buf.get() + (size_t)(i++) * n * hidden * es, rt->dtype);
         src.fetch_into(names.at("w1"), (char*)in_buf.get() + (size_t)4 * n * hidden * es, rt->dtype);
@@ -90,7 +92,6 @@ struct WkvMixer : Mixer {
         Mat xf = ops::cast(dev, x, DType::F32);
         long long group_rows = 0;
         Mat mixed = ops::token_mix(dev, xf, (const float*)mu_buf.get(), 5, ctx, cache.st, prev_off(), rt->dtype, &group_rows);
-        MatOrPartials y = ops::group_linear(dev, rt->gemm, mixed, group_rows, xf.rows, w_in, {n, n, n, n, rank}, false);
         ops::WkvScan p;
         p.r_off = 0;
         p.k_off = n;
@@ -103,6 +104,11 @@ struct WkvMixer : Mixer {
         p.w0 = (const float*)w0.m.p;
         p.u = (const float*)u.m.p;
         p.in_order = rt->is_f32();      // the float32 mode gives the same bits however a prompt is cut
+        const bool one = ctx.is_decode && !rt->is_f32() && ops::wkv_step_supported(p, cache.st);
+        MatOrPartials y = ops::group_linear(dev, rt->gemm, mixed, group_rows, xf.rows, w_in, {n, n, n, n, rank_rows}, one);
+        if (one)        // one token per sequence: everything up to the gated row in one kernel, which also adds up the slices
+            return ops::linear(dev, rt->gemm, ops::wkv_step(dev, y, p, 3 * n, (const float*)norm_w.m.p, norm_eps, ctx, cache.st), w_o.m,
+                               out_f32 ? DType::F32 : rt->dtype, may_defer);
         Mat o = ops::wkv_scan(dev, y.m, p, ctx, cache.st);
         Mat g = ops::group_norm_gate(dev, o, head_dim, (const float*)norm_w.m.p, norm_eps, (const float*)y.m.p + 3 * n, (int)y.m.cols, 1, rt->dtype);
         return ops::linear(dev, rt->gemm, g, w_o.m, out_f32 ? DType::F32 : rt->dtype, may_defer);
