@@ -47,7 +47,7 @@ join_rmsnorm_kernel(float* __restrict__ x, const float* __restrict__ y, int spli
         v[i] = c < H ? on_load4(yr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
         xv[i] = c < H ? on_load4(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    constexpr int K = NV <= 2 ? 4 : NV == 4 ? 2 : 1;         // slices on their way at a time, added in their order
+    constexpr int K = NV <= 4 ? 4 : 1;         // slices on their way at a time, added in their order
     for (int s = 1; s < splits; s += K) {
         float4 q[K][NV];
 #pragma unroll
@@ -152,7 +152,7 @@ embedding_normed_any_kernel(const int* __restrict__ ids, const TW* __restrict__ 
 }
 
 // threads of a row of H channels, and how many pieces of four channels a thread then holds (1, 2, 4 or 8; 0: too wide)
-static int on_threads(int H) { return H <= 512 ? 128 : H <= 1024 ? 256 : 512; }
+static int on_threads(int H) { return H <= 512 ? 128 : H <= 4096 ? 256 : 512; }
 static int on_pieces(int H) {
     if (H % 4 || H > 16384) return 0;
     const int n = (H / 4 + on_threads(H) - 1) / on_threads(H);

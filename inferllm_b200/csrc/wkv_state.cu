@@ -38,8 +38,8 @@
 // the state in registers: its products take one multiply-add per state element instead of three, and a chunk's tokens do
 // not wait for one another.  A long prompt of few sequences is cut into segments that run side by side: pass 0 runs every
 // segment but the last for its state alone, from zero (the first from the sequence's state), and leaves that state and the
-// product of its decays; pass 1 folds the earlier segments' states into the one its segment starts from and runs the segment
-// in full.  The sums have another order than token by token, so the float32 mode never takes this form.
+// product of its decays; wkv_fold_kernel turns these into the states that the later segments start from, and pass 1 runs
+// every segment in full.  The sums have another order than token by token, so the float32 mode never takes this form.
 #include <type_traits>
 
 #include "common.cuh"
@@ -228,20 +228,14 @@ __device__ __forceinline__ void ws_cp_async16(float* dst, const float* src) {
 }
 
 // A thread's piece of a state [dv][d] at `src`: R = 4 M rows of C columns as pairs of rows; row of pair (m, p): m * 4 LI + 4 g +
-// 2 p and the one behind it, so that the LI lanes of a column group touch 16-byte pieces that lie side by side.  `mul` (or
-// nullptr): what the thread holds already times the rows' factors is added.
+// 2 p and the one behind it, so that the LI lanes of a column group touch 16-byte pieces that lie side by side.
 template <int C, int M, int LI>
-__device__ __forceinline__ void wkv_load_state(f2 (&s)[C][M][2], const float* src, const float* mul, int j, int g, int d, int dv, bool vec) {
+__device__ __forceinline__ void wkv_load_state(f2 (&s)[C][M][2], const float* src, int j, int g, int d, int dv, bool vec) {
 #pragma unroll
-    for (int m = 0; m < M; m++) {
-        const int i = m * 4 * LI + 4 * g;
-        f2 f0 = 0, f1 = 0;
-        if (mul) {
-            f0 = f2_pack(i < d ? mul[i] : 0.f, i + 1 < d ? mul[i + 1] : 0.f);
-            f1 = f2_pack(i + 2 < d ? mul[i + 2] : 0.f, i + 3 < d ? mul[i + 3] : 0.f);
-        }
+    for (int c = 0; c < C; c++)
 #pragma unroll
-        for (int c = 0; c < C; c++) {
+        for (int m = 0; m < M; m++) {
+            const int i = m * 4 * LI + 4 * g;
             float v[4];
             if (vec && j + c < dv && i < d) {
                 const float4 v4 = *reinterpret_cast<const float4*>(src + (size_t)(j + c) * d + i);
@@ -250,10 +244,9 @@ __device__ __forceinline__ void wkv_load_state(f2 (&s)[C][M][2], const float* sr
 #pragma unroll
                 for (int r = 0; r < 4; r++) v[r] = (j + c < dv && i + r < d) ? src[(size_t)(j + c) * d + i + r] : 0.f;
             }
-            s[c][m][0] = mul ? f2_fma(s[c][m][0], f0, f2_pack(v[0], v[1])) : f2_pack(v[0], v[1]);
-            s[c][m][1] = mul ? f2_fma(s[c][m][1], f1, f2_pack(v[2], v[3])) : f2_pack(v[2], v[3]);
+            s[c][m][0] = f2_pack(v[0], v[1]);
+            s[c][m][1] = f2_pack(v[2], v[3]);
         }
-    }
 }
 template <int C, int M, int LI>
 __device__ __forceinline__ void wkv_store_state(const f2 (&s)[C][M][2], float* dst, int j, int g, int d, int dv, bool vec) {
@@ -329,7 +322,7 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(WkvScanArgs a) {
     const int jn = dv - j0 < JB ? dv - j0 : JB;     // columns of this block that exist
     float* Sg = a.state + (size_t)a.slots[b] * a.state_stride + (size_t)h * d * dv;       // [dv][d]
     f2 s[C][M][2];
-    wkv_load_state<C, M, LI>(s, Sg, nullptr, j0 + jl, g, d, dv, a.vec);
+    wkv_load_state<C, M, LI>(s, Sg, j0 + jl, g, d, dv, a.vec);
     // rows beyond d and columns beyond dv stay zero in both buffers
     for (int idx = threadIdx.x; idx < 2 * a.tile * ROW; idx += WS_THREADS) sm[idx] = 0.f;
     __syncthreads();
@@ -501,10 +494,13 @@ __device__ __forceinline__ void wc_mma(float* c, const unsigned* a, unsigned b0,
 }
 
 // grid (most chunks of a sequence, heads, sequences)
-__global__ void __launch_bounds__(128) wkv_chunk_prep_kernel(WkvChunkPrepArgs a) {
+__global__ void __launch_bounds__(128, 4) wkv_chunk_prep_kernel(WkvChunkPrepArgs a) {
     pdl_grid_sync();
     __shared__ __align__(16) bf16 th[2][WC_L][WC_TLD];             // tanh of the inner products, two bfloat16 terms
-    __shared__ __align__(16) float ws[WC_L][WC_LD], rs[WC_L][WC_LD], ks[WC_L][WC_LD];
+    struct Rows { float ws[WC_L][WC_LD], rs[WC_L][WC_LD], ks[WC_L][WC_LD]; };
+    union Shared { Rows rows; bf16 w2[WC_CH][WC_TLD]; };           // the outer map's tile is done with before the rows are made
+    __shared__ __align__(16) Shared sh;
+    float (*ws)[WC_LD] = sh.rows.ws, (*rs)[WC_LD] = sh.rows.rs, (*ks)[WC_LD] = sh.rows.ks;
     __shared__ __align__(16) float us[WC_CH];
     __shared__ float As[WC_L][WC_L];
     const int b = blockIdx.z, h = blockIdx.y, q0 = a.cu_q[b], q1 = a.cu_q[b + 1];
@@ -519,6 +515,16 @@ __global__ void __launch_bounds__(128) wkv_chunk_prep_kernel(WkvChunkPrepArgs a)
 #pragma unroll
     for (int j = 0; j <= WC_L; j++) av[j] = 0.f;
     for (int c0 = 0; c0 < d; c0 += WC_CH) {
+        // this thread's channel of r and k, on its way while the decays are made
+        const int ch = c0 + tid;
+        float kr[WC_L], rr[WC_L];
+        float* yr = a.y + (size_t)t0 * a.ld + a.r_off + h * d + ch;
+        float* yk = a.y + (size_t)t0 * a.ld + a.k_off + h * d + ch;
+#pragma unroll
+        for (int t = 0; t < WC_L; t++) {
+            rr[t] = t < n && ch < d ? yr[(size_t)t * a.ld] : 0.f;
+            kr[t] = t < n && ch < d ? yk[(size_t)t * a.ld] : 0.f;
+        }
         float acc[4][4];
 #pragma unroll
         for (int i = 0; i < 4; i++)
@@ -526,6 +532,22 @@ __global__ void __launch_bounds__(128) wkv_chunk_prep_kernel(WkvChunkPrepArgs a)
             for (int k = 0; k < 4; k++) acc[i][k] = 0.f;
         for (int r0 = 0; r0 < a.rank; r0 += WC_RK) {
             __syncthreads();
+            if (!(a.rank & 7)) {        // rows of whole 16-byte pieces
+                for (int i = tid; i < WC_CH * (WC_RK / 8); i += 128) {
+                    const int e = i / (WC_RK / 8), p = i % (WC_RK / 8) * 8;
+                    bf16* dst = &sh.w2[e][p];
+                    if (c0 + e < d && r0 + p < a.rank)
+                        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)),
+                                     "l"(a.w2 + (size_t)(h * d + c0 + e) * a.rank + r0 + p) : "memory");
+                    else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+                }
+                asm volatile("cp.async.commit_group;" ::: "memory");
+            } else {
+                for (int i = tid; i < WC_CH * WC_RK; i += 128) {
+                    const int e = i / WC_RK, p = i % WC_RK;
+                    sh.w2[e][p] = c0 + e < d && r0 + p < a.rank ? a.w2[(size_t)(h * d + c0 + e) * a.rank + r0 + p] : __float2bfloat16_rn(0.f);
+                }
+            }
             for (int i = tid; i < WC_L * WC_RK; i += 128) {
                 const int tt = i / WC_RK, r = i % WC_RK;
                 const float v = tt < n && r0 + r < a.rank ? tanhf(a.y[(size_t)(t0 + tt) * a.ld + a.z_off + r0 + r]) : 0.f;
@@ -533,6 +555,7 @@ __global__ void __launch_bounds__(128) wkv_chunk_prep_kernel(WkvChunkPrepArgs a)
                 th[0][tt][r] = hi;
                 th[1][tt][r] = __float2bfloat16_rn(v - __bfloat162float(hi));
             }
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
             __syncthreads();
             const int steps = ((a.rank - r0 < WC_RK ? a.rank - r0 : WC_RK) + 15) / 16;
             for (int kk = 0; kk < steps; kk++) {
@@ -540,24 +563,13 @@ __global__ void __launch_bounds__(128) wkv_chunk_prep_kernel(WkvChunkPrepArgs a)
                 wc_ldsm4(hi, &th[0][lane & 15][kk * 16 + (lane >> 4) * 8]);
                 wc_ldsm4(lo, &th[1][lane & 15][kk * 16 + (lane >> 4) * 8]);
 #pragma unroll
-                for (int i = 0; i < 4; i++) {
-                    const int c = c0 + (warp * 4 + i) * 8 + (lane >> 2);
-                    unsigned bb[2] = {0, 0};
-                    if (c < d) {
-                        const bf16* row = a.w2 + (size_t)(h * d + c) * a.rank;
-#pragma unroll
-                        for (int x = 0; x < 2; x++) {
-                            const int k = r0 + kk * 16 + (lane & 3) * 2 + 8 * x;
-                            if (!(a.rank & 1)) {
-                                if (k < a.rank) bb[x] = *reinterpret_cast<const unsigned*>(row + k);
-                            } else {
-                                const unsigned e0 = k < a.rank ? __bfloat16_as_ushort(row[k]) : 0, e1 = k + 1 < a.rank ? __bfloat16_as_ushort(row[k + 1]) : 0;
-                                bb[x] = e0 | (e1 << 16);
-                            }
-                        }
-                    }
-                    wc_mma(acc[i], hi, bb[0], bb[1]);
-                    wc_mma(acc[i], lo, bb[0], bb[1]);
+                for (int i = 0; i < 2; i++) {
+                    unsigned bb[4];
+                    wc_ldsm4(bb, &sh.w2[warp * 32 + i * 16 + (lane & 7) + ((lane >> 4) << 3)][kk * 16 + ((lane >> 3) & 1) * 8]);
+                    wc_mma(acc[2 * i], hi, bb[0], bb[1]);
+                    wc_mma(acc[2 * i], lo, bb[0], bb[1]);
+                    wc_mma(acc[2 * i + 1], hi, bb[2], bb[3]);
+                    wc_mma(acc[2 * i + 1], lo, bb[2], bb[3]);
                 }
             }
         }
@@ -576,15 +588,10 @@ __global__ void __launch_bounds__(128) wkv_chunk_prep_kernel(WkvChunkPrepArgs a)
         }
         __syncthreads();
         {
-            const int c = c0 + tid;
+            const int c = ch;
             us[tid] = c < d ? a.u[h * d + c] : 0.f;
-            float kr[WC_L], rr[WC_L];
-            float* yr = a.y + (size_t)t0 * a.ld + a.r_off + h * d + c;
-            float* yk = a.y + (size_t)t0 * a.ld + a.k_off + h * d + c;
 #pragma unroll
             for (int t = 0; t < WC_L; t++) {
-                rr[t] = t < n && c < d ? yr[(size_t)t * a.ld] : 0.f;
-                kr[t] = t < n && c < d ? yk[(size_t)t * a.ld] : 0.f;
                 rs[t][tid] = rr[t];
                 ks[t][tid] = kr[t];
             }
@@ -714,7 +721,7 @@ __global__ void __launch_bounds__(128) wkv_chunk_kernel(WkvChunkArgs a) {
         for (int m = 0; m < M; m++) cum[m][0] = cum[m][1] = f2_pack(1.f, 1.f);
         if (seg == 0) {
             // what came in is kept for pass 1, whose last segment renews the state while its first may not have begun
-            wkv_load_state<C, M, LI>(s, Sg, nullptr, j0 + jl, g, d, dv, true);
+            wkv_load_state<C, M, LI>(s, Sg, j0 + jl, g, d, dv, true);
             wkv_store_state<C, M, LI>(s, seg_base + (size_t)(S - 1) * seg_stride, j0 + jl, g, d, dv, true);
         } else {
 #pragma unroll
@@ -723,10 +730,9 @@ __global__ void __launch_bounds__(128) wkv_chunk_kernel(WkvChunkArgs a) {
                 for (int m = 0; m < M; m++) s[c][m][0] = s[c][m][1] = 0;
         }
     } else if (seg == 0) {
-        wkv_load_state<C, M, LI>(s, last ? Sg : seg_base + (size_t)(S - 1) * seg_stride, nullptr, j0 + jl, g, d, dv, true);
+        wkv_load_state<C, M, LI>(s, last ? Sg : seg_base + (size_t)(S - 1) * seg_stride, j0 + jl, g, d, dv, true);
     } else {
-        wkv_load_state<C, M, LI>(s, seg_base, nullptr, j0 + jl, g, d, dv, true);
-        for (int r = 1; r < seg; r++) wkv_load_state<C, M, LI>(s, seg_base + r * seg_stride, dec_base + r * dec_stride, j0 + jl, g, d, dv, true);
+        wkv_load_state<C, M, LI>(s, seg_base + (seg - 1) * seg_stride, j0 + jl, g, d, dv, true);
     }
     int buf = 0;
     for (int chunk = first_chunk; chunk < end_chunk; chunk++, buf ^= 1) {
@@ -840,6 +846,36 @@ __global__ void __launch_bounds__(128) wkv_chunk_kernel(WkvChunkArgs a) {
     }
 }
 
+// Between the passes: the state behind segment r from those of the segments by themselves, S_r <- diag(D_r) S_(r-1) + S_r, r from
+// 1 to the last segment but one.  A thread per four rows of a column.  grid (pieces, heads, sequences)
+__global__ void __launch_bounds__(256) wkv_fold_kernel(WkvChunkArgs a) {
+    pdl_grid_sync();
+    const int S = a.segments, b = blockIdx.z, h = blockIdx.y, d = a.d;
+    const int n = a.cu_q[b + 1] - a.cu_q[b], chunks = (n + WC_L - 1) / WC_L, per = (chunks + S - 1) / S;
+    const int used = per > 0 ? (chunks + per - 1) / per : 0;
+    const int i = (blockIdx.x * 256 + threadIdx.x) * 4;
+    if (i >= d * a.dv) return;
+    float* st = a.seg_state + ((size_t)b * S * a.nh + h) * (size_t)d * a.dv + i;
+    const float* dec = a.seg_decay + ((size_t)b * S * a.nh + h) * (size_t)d + i % d;
+    const size_t st_stride = (size_t)a.nh * d * a.dv, dec_stride = (size_t)a.nh * d;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int r0 = 0; r0 < used - 1; r0 += 4) {
+        float4 v[4], f[4];
+#pragma unroll
+        for (int k = 0; k < 4; k++)
+            if (r0 + k < used - 1) {
+                v[k] = *reinterpret_cast<const float4*>(st + (r0 + k) * st_stride);
+                f[k] = *reinterpret_cast<const float4*>(dec + (r0 + k) * dec_stride);
+            }
+#pragma unroll
+        for (int k = 0; k < 4; k++)
+            if (r0 + k < used - 1) {
+                acc.x = fmaf(f[k].x, acc.x, v[k].x), acc.y = fmaf(f[k].y, acc.y, v[k].y), acc.z = fmaf(f[k].z, acc.z, v[k].z), acc.w = fmaf(f[k].w, acc.w, v[k].w);
+                *reinterpret_cast<float4*>(st + (r0 + k) * st_stride) = acc;
+            }
+    }
+}
+
 template <int R, int C, int LI>
 static int wkv_chunk_launch(const WkvChunkArgs& a, int B, cudaStream_t s) {
     constexpr int DP = R * LI, JB = C * (32 / LI) * 4;
@@ -852,7 +888,10 @@ static int wkv_chunk_launch(const WkvChunkArgs& a, int B, cudaStream_t s) {
         raised = true;
     }
     const dim3 grid(B * a.segments, a.nh, (a.dv + JB - 1) / JB);
-    if (a.segments > 1) illm_launch(wkv_chunk_kernel<R, C, LI, 0>, grid, dim3(128), smem0, s, a);
+    if (a.segments > 1) {
+        illm_launch(wkv_chunk_kernel<R, C, LI, 0>, grid, dim3(128), smem0, s, a);
+        if (a.segments > 2) illm_launch(wkv_fold_kernel, dim3((a.d * a.dv / 4 + 255) / 256, a.nh, B), dim3(256), 0, s, a);
+    }
     illm_launch(wkv_chunk_kernel<R, C, LI, 1>, grid, dim3(128), smem1, s, a);
     return illm_launch_status();
 }
@@ -872,7 +911,7 @@ extern "C" int illm_wkv_chunks(float* y, int T, int ld, int r_off, int k_off, in
     if (segments < 1 || (segments > 1 && (!seg_state || !seg_decay)) || (long long)B * segments > 0x7fffffff || B > 65535 || max_q <= 0) return ILLM_ERR_BAD_ARG;
     if (nh <= 0 || nh > 65535 || rank <= 0 || !y || !w2 || !w0 || !u || !state || !A || !P || !out || state_stride < (long long)nh * d * dv ||
         !illm_wkv_chunk_supported(d, dv, ld, r_off, k_off, v_off) || (state_stride & 3) ||
-        (((uintptr_t)y | (uintptr_t)state | (uintptr_t)A | (uintptr_t)P | (uintptr_t)seg_state | (uintptr_t)seg_decay) & 15) || ((uintptr_t)w2 & 3))
+        (((uintptr_t)y | (uintptr_t)state | (uintptr_t)A | (uintptr_t)P | (uintptr_t)seg_state | (uintptr_t)seg_decay) & 15) || ((uintptr_t)w2 & 15))
         return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     WkvChunkPrepArgs p{y, ld, r_off, k_off, z_off, rank, nh, d, (const bf16*)w2, w0, u, cu_q, A, P};

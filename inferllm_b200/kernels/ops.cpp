@@ -1058,7 +1058,7 @@ bool wkv_supported(int d, int dv) { return illm_wkv_supported(d, dv) != 0; }
 
 int wkv_segments(int B, int n_heads, int v_head_dim, int max_q, int n_sms) {
     const long long blocks = (long long)B * n_heads * ceil_div(v_head_dim, 128);
-    long long P = std::min<long long>(16, (4LL * n_sms) / std::max<long long>(blocks, 1));
+    long long P = std::min<long long>(32, (2LL * n_sms) / std::max<long long>(blocks, 1));
     P = std::min<long long>(P, max_q / 64);
     return P < 2 ? 1 : (int)P;
 }

@@ -405,7 +405,7 @@ struct WkvScan {
 };
 constexpr int kWkvChunkMinTokens = 16;       // the most tokens of a sequence in a step from which prompts go sixteen at a time
 bool wkv_supported(int head_dim, int v_head_dim);
-// In how many segments the chunks of a prompt step's sequences are cut: enough blocks for the GPU, at most 16, none of fewer
+// In how many segments the chunks of a prompt step's sequences are cut: two blocks per SM, at most 32, none of fewer
 // than 64 tokens.
 int wkv_segments(int B, int n_heads, int v_head_dim, int max_q, int n_sms);
 Mat wkv_scan(Device& dev, const Mat& y_f32, const WkvScan& p, const StepView& ctx, const StateView& st);
