@@ -70,7 +70,7 @@ _SIGNATURES = {
     "illm_config_to_json": [P, PP], "illm_config_architecture": [P, PP], "illm_config_model_spec": [P, PP],
     "illm_model_spec_validate": [S], "illm_registered_architectures": [PP], "illm_resolve_architecture": [S, PP],
     "illm_registered_parts": [S, PP], "illm_register_architecture": [S, S, P, P], "illm_unregister_architecture": [S],
-    "illm_tensor_decls": [P, PP], "illm_check_model_folder": [P, S], "illm_write_random_model": [P, S, ULL, S],
+    "illm_tensor_decls": [P, PP], "illm_model_cache_requests": [P, PP], "illm_check_model_folder": [P, S], "illm_write_random_model": [P, S, ULL, S],
     "illm_storage_dtype": [S, S, S, PP], "illm_random_values": [ULL, S, LL, S, P], "illm_model_files": [S, PP],
     "illm_model_files_read": [S, S, P, LL], "illm_write_safetensors": [S, S, P, S],
     "illm_pool_create": [I, S, PP], "illm_pool_free_handle": [P], "illm_pool_alloc": [P, I, PI],

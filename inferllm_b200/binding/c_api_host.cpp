@@ -140,6 +140,15 @@ ILLM_API int illm_tensor_decls(void* cfg, char** out) {
         *out = dup_string(a.dump());
     });
 }
+ILLM_API int illm_model_cache_requests(void* cfg, char** out) {
+    return guard([&] {
+        DecoderModel model(((ArchConfig*)cfg)->model_spec(), nullptr);
+        Json o = Json::object();
+        for (auto& r : model.cache_requests())
+            if (r.second.kind != CacheRequest::None) o.set(std::to_string(r.first), r.second.to_json());
+        *out = dup_string(o.dump());
+    });
+}
 ILLM_API int illm_check_model_folder(void* cfg, const char* folder) {
     return guard([&] {
         DecoderModel model(((ArchConfig*)cfg)->model_spec(), nullptr);

@@ -45,6 +45,12 @@ class FixedState:
         return {"kind": "state", "shape": list(self.shape), "dtype": str(self.dtype).replace("torch.", "")}
 
 
+def cache_requests(config) -> Dict[int, dict]:
+    """What the model of a configuration asks of the cache: entry number -> the request as a dictionary (an entry that several
+    layers read is wide enough for all of them)."""
+    return {int(k): v for k, v in _b.call_json(_b.lib().illm_model_cache_requests, config.handle()).items()}
+
+
 class IndexPool:
     def __init__(self, n: int, what: str, _ptr=None, _owner=None):
         self._owner = _owner
