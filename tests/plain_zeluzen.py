@@ -309,6 +309,29 @@ def random_weights(cfg, seed, gain=1.0, rank=7):
     return w
 
 
+def steady_routing(cfg, w, channels=8, margin=0.01):
+    """Edits the weights so that rounding cannot turn a router's choice: the routers read the first few channels alone, which
+    hold the embedding as it is (no sublayer writes there).  Returns the tokens whose choices all have at least this margin."""
+    eps, good = cfg["norm"]["eps"], np.ones(cfg["vocab"], bool)
+    for i, L in enumerate(cfg["layers"]):
+        for role in ("norm1", "norm2"):
+            if "l%d.%s" % (i, role) in w:
+                w["l%d.%s" % (i, role)][:channels] = 0.0
+    x = rms_norm(np.asarray(w["embed"], np.float64), np.asarray(w["embed.norm"], np.float64), eps)
+    for i, L in enumerate(cfg["layers"]):
+        if L.get("mlp") and L["mlp"]["kind"] == "moe":
+            r = w["l%d.mlp.router" % i]
+            r[:, channels:] = 0.0
+            r[:, :channels] *= bf16_round(np.float32(math.sqrt(r.shape[1] / channels)))
+            w["l%d.mlp.router" % i] = bf16_round(r)
+            W = {k: np.asarray(w["l%d.mlp.%s" % (i, k)], np.float64) for k in ("router", "correction")}
+            s, _ = route(x, W, "", L["mlp"]["router"])
+            c, top = np.sort(s + W["correction"], axis=-1)[:, ::-1], L["mlp"]["router"]["top"]
+            if top < c.shape[1]:
+                good &= c[:, top - 1] - c[:, top] > margin
+    return np.flatnonzero(good).tolist()
+
+
 def write_model(folder, cfg, w):
     """config.json and model.safetensors (bfloat16) of (cfg, w) in `folder`."""
     import json
