@@ -190,7 +190,9 @@ int illm_wkv_step(const float* y, int splits, long long stride, int T, int ld, i
 // gemm_tc.cu, qk_prep.cu, moe.cu: further forms
 int illm_gemm_bf16_tc_grouped(const void* X, int x_rows, const void* W, const int* n, int n_groups, float* out, int M, int K, float* ws, int splits, int* err, void* stream, int skip_reduce);
 int illm_qk_prep_heads(const void* x, int x_dtype, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int d, int dv, const float* bq, const float* bk, const float* bv, const float* wq, const float* wk, float eps, const float* cos_sin, int rot, int pairs, int n_pos, const int* token_pos, const int* token_seq, const int* block_table, int max_pages, int page_size, void* q_out, void* kc, void* vc, int act_dtype, int T, int* err, float qt_coef, int qt_every, const float* v_first, int v_first_ld, const float* v_lambda, float* v_keep, int head_norm, void* stream);
-int illm_moe_combine_ex(const float* rows, const int* row_of_pair, const float* weight, const float* plus, const void* x, int x_dtype, float* out, int T, int D, int top, void* stream);
+int illm_moe_combine_ex(const float* rows, const int* row_of_pair, const float* weight, const float* plus, const void* x, int x_dtype, float* out, int T, int D, int top, int splits, long long slice_stride, void* stream);
+int illm_moe_down_splits(int T, int top, int E, int N, int K, int n_sms);
+int illm_moe_gemm_split(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated, int act, float act_limit, int bm, int tensor_cores, int splits, long long slice_stride, const int* pair_of_row, const int* tile_expert, const int* tile_row0, const int* tile_rows, void* stream);
 
 #ifdef __cplusplus
 }

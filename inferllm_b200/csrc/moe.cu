@@ -318,10 +318,13 @@ __device__ __forceinline__ void mm_mma(float* c, const unsigned* a, unsigned b0,
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+//
+// blockIdx.z: of a down product whose grid would not fill the GPU (single tokens), K may be cut into gridDim.z slices of k_per
+// slabs; slice z goes to its own rows, slice_stride elements behind the one before (moe_combine_kernel adds them in order).
 template <typename TY, int MODE>
 __global__ void __launch_bounds__(256)
-moe_gemm_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* __restrict__ y, int N, int K, int top, int act, float act_limit,
-                    const int* __restrict__ pair_of_row, const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
+moe_gemm_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* __restrict__ y, int N, int K, int top, int act, float act_limit, int k_per,
+                    long long slice_stride, const int* __restrict__ pair_of_row, const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
                     const int* __restrict__ tile_rows) {
     pdl_grid_sync();
     extern __shared__ __align__(16) unsigned char mm_raw[];
@@ -337,13 +340,15 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* 
     for (int m = tid; m < MM_BM; m += 256) src_row[m] = m < rows ? (MODE != MOE_DOWN ? pair_of_row[row0 + m] / top : row0 + m) : -1;
     __syncthreads();
     const bf16* wg = w + (size_t)e * N * K;
-    const int KT = (K + MM_BK - 1) / MM_BK;
+    const int kt0 = blockIdx.z * k_per, kt_all = (K + MM_BK - 1) / MM_BK;
+    const int KT = kt_all - kt0 < k_per ? kt_all - kt0 : k_per;
+    if (MODE == MOE_DOWN) y += (size_t)blockIdx.z * slice_stride;
     // what this thread copies per slab: one 16-byte piece of A, two of each B
     const int a_r = tid >> 2, a_c = (tid & 3) * 8;
     const int a_src = src_row[a_r];
     auto load = [&](int stage, int kt) {
         bf16* base = sm + (size_t)stage * STAGE_ELEMS;
-        const int k = kt * MM_BK + a_c;
+        const int k = (kt0 + kt) * MM_BK + a_c;
         {
             const bool ok = a_src >= 0 && k < K;
             mm_cp16(mm_smem(base + a_r * MM_LD + a_c), ok ? (const void*)(x + (size_t)a_src * K + k) : (const void*)x, ok ? 16 : 0);
@@ -424,7 +429,8 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* 
 // gives back (nullptr: there are none)
 template <typename TX>
 __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ row_of_pair, const float* __restrict__ weight,
-                                   const float* __restrict__ plus, const TX* __restrict__ x, float* __restrict__ out, int D, int top, long long n) {
+                                   const float* __restrict__ plus, const TX* __restrict__ x, float* __restrict__ out, int D, int top, long long n,
+                                   int splits, long long slice_stride) {
     pdl_grid_sync();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
@@ -433,44 +439,65 @@ __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __
     float acc = 0.f;
     for (int k = 0; k < top; k++) {
         const int row = row_of_pair[t * top + k];
-        const float v = row >= 0 ? rows[(size_t)row * D + c] : x ? to_f32(x[i]) : 0.f;
+        float v = row >= 0 ? rows[(size_t)row * D + c] : x ? to_f32(x[i]) : 0.f;
+        if (row >= 0)
+            for (int s = 1; s < splits; s++) v += rows[(size_t)s * slice_stride + (size_t)row * D + c];
         acc = fmaf(weight[t * top + k], v, acc);
     }
     out[i] = plus ? acc + plus[i] : acc;
 }
 
-// the same, four neighbouring channels per thread (D a multiple of four), a block per token
+// the same, four neighbouring channels per thread (D a multiple of four); grid (tokens, pieces of 1,024 channels)
 template <typename TX>
 __global__ void __launch_bounds__(256)
 moe_combine_vec_kernel(const float* __restrict__ rows, const int* __restrict__ row_of_pair, const float* __restrict__ weight, const float* __restrict__ plus,
-                       const TX* __restrict__ x, float* __restrict__ out, int D, int top) {
+                       const TX* __restrict__ x, float* __restrict__ out, int D, int top, int splits, long long slice_stride) {
     pdl_grid_sync();
-    const int t = blockIdx.x;
-    for (int c = threadIdx.x * 4; c < D; c += 1024) {
-        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int k = 0; k < top; k++) {
-            const int row = row_of_pair[t * top + k];
-            const float w = weight[t * top + k];
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (row >= 0) {
-                v = *reinterpret_cast<const float4*>(rows + (size_t)row * D + c);
-            } else if (x) {
-                const TX* xr = x + (size_t)t * D + c;
-                v = make_float4(to_f32(xr[0]), to_f32(xr[1]), to_f32(xr[2]), to_f32(xr[3]));
+    const int t = blockIdx.x, c = (blockIdx.y * 256 + threadIdx.x) * 4;
+    if (c >= D) return;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
+    for (int k = 0; k < top; k++) {
+        const int row = row_of_pair[t * top + k];
+        const float w = weight[t * top + k];
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (row >= 0) {
+            const float* r = rows + (size_t)row * D + c;
+            v = *reinterpret_cast<const float4*>(r);
+#pragma unroll 4
+            for (int s = 1; s < splits; s++) {
+                const float4 q = *reinterpret_cast<const float4*>(r + (size_t)s * slice_stride);
+                v.x += q.x, v.y += q.y, v.z += q.z, v.w += q.w;
             }
-            acc.x = fmaf(w, v.x, acc.x), acc.y = fmaf(w, v.y, acc.y), acc.z = fmaf(w, v.z, acc.z), acc.w = fmaf(w, v.w, acc.w);
+        } else if (x) {
+            const TX* xr = x + (size_t)t * D + c;
+            v = make_float4(to_f32(xr[0]), to_f32(xr[1]), to_f32(xr[2]), to_f32(xr[3]));
         }
-        if (plus) {
-            const float4 p = *reinterpret_cast<const float4*>(plus + (size_t)t * D + c);
-            acc.x += p.x, acc.y += p.y, acc.z += p.z, acc.w += p.w;
-        }
-        *reinterpret_cast<float4*>(out + (size_t)t * D + c) = acc;
+        acc.x = fmaf(w, v.x, acc.x), acc.y = fmaf(w, v.y, acc.y), acc.z = fmaf(w, v.z, acc.z), acc.w = fmaf(w, v.w, acc.w);
     }
+    if (plus) {
+        const float4 p = *reinterpret_cast<const float4*>(plus + (size_t)t * D + c);
+        acc.x += p.x, acc.y += p.y, acc.z += p.z, acc.w += p.w;
+    }
+    *reinterpret_cast<float4*>(out + (size_t)t * D + c) = acc;
 }
 
 extern "C" int illm_moe_max_tiles(int T, int top, int E, int bm) { return (int)(((long long)T * top + bm - 1) / bm) + E; }
 // rows per tile: the tensor-core kernel takes 64; the plain one 16 for steps of few tokens, else 64
 extern "C" int illm_moe_row_tile(int T, int top, int tensor_cores) { return tensor_cores || (long long)T * top > 1024 ? 64 : 16; }
+
+// In how many slices of K a tensor-core down product of few rows is cut: about four blocks per SM over the experts that the rows
+// can hit, no slice shorter than 16 slabs; and how many there then are.
+extern "C" int illm_moe_down_splits(int T, int top, int E, int N, int K, int n_sms) {
+    const long long P = (long long)T * top, hit = P < E ? P : E, blocks = (long long)((N + MM_BN - 1) / MM_BN) * (hit > 0 ? hit : 1);
+    const int k_tiles = (K + MM_BK - 1) / MM_BK;
+    long long splits = (4LL * n_sms + blocks - 1) / blocks;
+    if (splits > 8) splits = 8;
+    if (splits > k_tiles / 16) splits = k_tiles / 16;
+    if (splits <= 1) return 1;
+    const int k_per = (int)((k_tiles + splits - 1) / splits);
+    return (k_tiles + k_per - 1) / k_per;
+}
 
 // xs[row, :] = x[pair_of_row[row] / top, :], 16 bytes at a time (K a multiple of 8): the rows in the experts' order
 __global__ void moe_gather_rows_kernel(const bf16* __restrict__ x, bf16* __restrict__ xs, const int* __restrict__ pair_of_row, int K, int top) {
@@ -546,6 +573,9 @@ extern "C" int illm_moe_route_ex2(const float* logits, const float* bias, int T,
 extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated,
                                 int act, float act_limit, int bm, int tensor_cores, const int* pair_of_row, const int* tile_expert,
                                 const int* tile_row0, const int* tile_rows, void* stream);
+extern "C" int illm_moe_gemm_split(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated,
+                                   int act, float act_limit, int bm, int tensor_cores, int splits, long long slice_stride, const int* pair_of_row,
+                                   const int* tile_expert, const int* tile_row0, const int* tile_rows, void* stream);
 extern "C" int illm_moe_gemm(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated,
                              int act, int bm, int tensor_cores, const int* pair_of_row, const int* tile_expert, const int* tile_row0,
                              const int* tile_rows, void* stream) {
@@ -556,14 +586,23 @@ extern "C" int illm_moe_gemm(const void* x, int x_dtype, const void* w, int w_dt
 extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated,
                                 int act, float act_limit, int bm, int tensor_cores, const int* pair_of_row, const int* tile_expert,
                                 const int* tile_row0, const int* tile_rows, void* stream) {
+    return illm_moe_gemm_split(x, x_dtype, w, w_dtype, y, T, top, E, N, K, gated, act, act_limit, bm, tensor_cores, 1, 0, pair_of_row, tile_expert, tile_row0,
+                               tile_rows, stream);
+}
+// splits > 1 (tensor_cores and gated 0 only): K in so many slices, y [splits, T * top, N], slice_stride elements apart
+extern "C" int illm_moe_gemm_split(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int T, int top, int E, int N, int K, int gated,
+                                   int act, float act_limit, int bm, int tensor_cores, int splits, long long slice_stride, const int* pair_of_row,
+                                   const int* tile_expert, const int* tile_row0, const int* tile_rows, void* stream) {
     if (T <= 0) return 0;
+    if (splits < 1 || (splits > 1 && (gated || !tensor_cores || slice_stride < (long long)T * top * N))) return ILLM_ERR_BAD_ARG;
     if (N <= 0 || K <= 0 || x_dtype != w_dtype || (bm != 16 && bm != 64) || gated < 0 || gated > 2 || (gated == 1 && (N & 1))) return ILLM_ERR_BAD_ARG;
     const int tiles = illm_moe_max_tiles(T, top, E, bm);
     if (tiles > 65535) return ILLM_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     if (tensor_cores) {
         if (x_dtype != ILLM_BF16 || (K & 7) || bm != MM_BM || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return ILLM_ERR_BAD_ARG;
-        dim3 mgrid((N + MM_BN - 1) / MM_BN, tiles);
+        const int k_tiles = (K + MM_BK - 1) / MM_BK, k_per = (k_tiles + splits - 1) / splits;
+        dim3 mgrid((N + MM_BN - 1) / MM_BN, tiles, (k_tiles + k_per - 1) / k_per);
         const size_t smem = (size_t)MM_STAGES * (MM_BM + MM_BN) * MM_LD * sizeof(bf16);
         static bool raised = false;
         if (!raised) {
@@ -573,14 +612,14 @@ extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w
             raised = true;
         }
         if (gated == 1)
-            illm_launch(moe_gemm_mma_kernel<bf16, MOE_GATED>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (bf16*)y, N, K, top, act, act_limit,
-                        pair_of_row, tile_expert, tile_row0, tile_rows);
+            illm_launch(moe_gemm_mma_kernel<bf16, MOE_GATED>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (bf16*)y, N, K, top, act, act_limit, k_per,
+                        slice_stride, pair_of_row, tile_expert, tile_row0, tile_rows);
         else if (gated == 2)
-            illm_launch(moe_gemm_mma_kernel<bf16, MOE_PLAIN>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (bf16*)y, N, K, top, act, act_limit,
-                        pair_of_row, tile_expert, tile_row0, tile_rows);
+            illm_launch(moe_gemm_mma_kernel<bf16, MOE_PLAIN>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (bf16*)y, N, K, top, act, act_limit, k_per,
+                        slice_stride, pair_of_row, tile_expert, tile_row0, tile_rows);
         else
-            illm_launch(moe_gemm_mma_kernel<float, MOE_DOWN>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (float*)y, N, K, top, act, act_limit,
-                        pair_of_row, tile_expert, tile_row0, tile_rows);
+            illm_launch(moe_gemm_mma_kernel<float, MOE_DOWN>, mgrid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w, (float*)y, N, K, top, act, act_limit, k_per,
+                        slice_stride, pair_of_row, tile_expert, tile_row0, tile_rows);
         return illm_launch_status();
     }
     dim3 grid((N + MOE_BN - 1) / MOE_BN, tiles);
@@ -602,27 +641,30 @@ extern "C" int illm_moe_gemm_ex(const void* x, int x_dtype, const void* w, int w
     return illm_launch_status();
 }
 
-// x (x_dtype, [T, D]): the input rows, for pairs without a row (identity experts); nullptr: there are none
+// x (x_dtype, [T, D]): the input rows, for pairs without a row (identity experts); nullptr: there are none.  splits: the rows come
+// in so many slices, slice_stride elements apart
 extern "C" int illm_moe_combine_ex(const float* rows, const int* row_of_pair, const float* weight, const float* plus, const void* x, int x_dtype,
-                                   float* out, int T, int D, int top, void* stream) {
+                                   float* out, int T, int D, int top, int splits, long long slice_stride, void* stream) {
     if (T <= 0) return 0;
+    if (splits < 1) return ILLM_ERR_BAD_ARG;
     const long long n = (long long)T * D;
-    const dim3 grid((unsigned)((n + 255) / 256));
     cudaStream_t s = (cudaStream_t)stream;
-    if (!(D & 3) && !(((uintptr_t)rows | (uintptr_t)plus | (uintptr_t)out) & 15)) {
-        if (x && x_dtype == ILLM_BF16) illm_launch(moe_combine_vec_kernel<bf16>, dim3(T), dim3(256), 0, s, rows, row_of_pair, weight, plus, (const bf16*)x, out, D, top);
-        else if (!x || x_dtype == ILLM_F32) illm_launch(moe_combine_vec_kernel<float>, dim3(T), dim3(256), 0, s, rows, row_of_pair, weight, plus, (const float*)x, out, D, top);
-        else return ILLM_ERR_BAD_ARG;
+    const bool half = x && x_dtype == ILLM_BF16;
+    if (x && !half && x_dtype != ILLM_F32) return ILLM_ERR_BAD_ARG;
+    if (!(D & 3) && !(slice_stride & 3) && !(((uintptr_t)rows | (uintptr_t)plus | (uintptr_t)out) & 15)) {
+        const dim3 grid(T, (D + 1023) / 1024);
+        if (half) illm_launch(moe_combine_vec_kernel<bf16>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const bf16*)x, out, D, top, splits, slice_stride);
+        else illm_launch(moe_combine_vec_kernel<float>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const float*)x, out, D, top, splits, slice_stride);
         return illm_launch_status();
     }
-    if (x && x_dtype == ILLM_BF16) illm_launch(moe_combine_kernel<bf16>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const bf16*)x, out, D, top, n);
-    else if (!x || x_dtype == ILLM_F32) illm_launch(moe_combine_kernel<float>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const float*)x, out, D, top, n);
-    else return ILLM_ERR_BAD_ARG;
+    const dim3 grid((unsigned)((n + 255) / 256));
+    if (half) illm_launch(moe_combine_kernel<bf16>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const bf16*)x, out, D, top, n, splits, slice_stride);
+    else illm_launch(moe_combine_kernel<float>, grid, dim3(256), 0, s, rows, row_of_pair, weight, plus, (const float*)x, out, D, top, n, splits, slice_stride);
     return illm_launch_status();
 }
 extern "C" int illm_moe_combine_plus(const float* rows, const int* row_of_pair, const float* weight, const float* plus, float* out, int T, int D,
                                      int top, void* stream) {
-    return illm_moe_combine_ex(rows, row_of_pair, weight, plus, nullptr, 0, out, T, D, top, stream);
+    return illm_moe_combine_ex(rows, row_of_pair, weight, plus, nullptr, 0, out, T, D, top, 1, 0, stream);
 }
 extern "C" int illm_moe_combine(const float* rows, const int* row_of_pair, const float* weight, float* out, int T, int D, int top,
                                 void* stream) {

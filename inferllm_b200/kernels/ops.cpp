@@ -1253,7 +1253,10 @@ Mat moe_forward_ex(Device& dev, const Mat& h, const Mat& logits, const MoeRoutin
                                     r.weight_scale, expert, weight, row_of_pair, pair_of_row, tile_expert, tile_row0, tile_rows, dev.stream()),
                  "moe_route");
     const int code = code_of(h.dtype, "moe");
-    Mat hid = new_mat_exact(dev, P, F, h.dtype), rows = new_mat_exact(dev, P, D, DType::F32), out = new_mat_exact(dev, T, D, DType::F32);
+    // the down product of few rows in slices of K, which the combining kernel adds up
+    const int splits = tc && !tc5 ? illm_moe_down_splits((int)T, top, E, (int)D, (int)F, dev.n_sms()) : 1;
+    const long long slice = splits > 1 ? (P * D + 3) / 4 * 4 : 0;
+    Mat hid = new_mat_exact(dev, P, F, h.dtype), rows = new_mat_exact(dev, splits > 1 ? splits * (P + 1) : P, D, DType::F32), out = new_mat_exact(dev, T, D, DType::F32);
     if (tc5) {
         Mat xs = new_mat_exact(dev, P, D, DType::BF16);
         check_kernel(illm_moe_gather_rows(h.p, xs.p, pair_of_row, (int)P, (int)D, top, dev.stream()), "moe_gather_rows");
@@ -1267,12 +1270,12 @@ Mat moe_forward_ex(Device& dev, const Mat& h, const Mat& logits, const MoeRoutin
         check_kernel(illm_moe_gemm_ex(h.p, code, w_gu.p, code, hid.p, (int)T, top, E, (int)(per * F), (int)D, r.plain ? 2 : 1, act, r.act_limit, bm, tc, pair_of_row, tile_expert, tile_row0,
                                    tile_rows, dev.stream()),
                      "moe_gemm (gate/up)");
-        check_kernel(illm_moe_gemm(hid.p, code, w_down.p, code, rows.p, (int)T, top, E, (int)D, (int)F, 0, 0, bm, tc, pair_of_row, tile_expert, tile_row0,
-                                   tile_rows, dev.stream()),
+        check_kernel(illm_moe_gemm_split(hid.p, code, w_down.p, code, rows.p, (int)T, top, E, (int)D, (int)F, 0, 0, 0.f, bm, tc, splits, slice, pair_of_row,
+                                         tile_expert, tile_row0, tile_rows, dev.stream()),
                      "moe_gemm (down)");
     }
     check_kernel(illm_moe_combine_ex((const float*)rows.p, row_of_pair, weight, r.plus ? (const float*)r.plus->p : nullptr, r.identity ? h.p : nullptr, code,
-                                     (float*)out.p, (int)T, (int)D, top, dev.stream()),
+                                     (float*)out.p, (int)T, (int)D, top, splits, slice, dev.stream()),
                  "moe_combine");
     return out;
 }
